@@ -32,6 +32,7 @@ class KVRequest:
     window: Optional[int] = None
     v_head_dim: Optional[int] = None        # size of a value head when it differs from the key head's
     values_in_keys: bool = False            # the values are columns of the key rows: no value pages are kept
+    keep_first: int = 0                     # under a window: this many first keys of a sequence stay visible
 
 
 @dataclass(frozen=True)
@@ -72,15 +73,15 @@ def plan_groups(requests: Mapping[int, Sequence[object]]):
                 if seen_kv:
                     raise CacheError(f"cache entry {entry} asks for keys and values twice")
                 seen_kv = True
-                kv_keys.setdefault((r.n_kv_heads, r.head_dim, r.window, 0 if r.values_in_keys else r.v_head_dim or r.head_dim),
-                                   []).append(entry)
+                kv_keys.setdefault((r.n_kv_heads, r.head_dim, r.window, 0 if r.values_in_keys else r.v_head_dim or r.head_dim,
+                                    r.keep_first if r.window is not None else 0), []).append(entry)
             elif isinstance(r, StateRequest):
                 if r.dtype not in _TORCH:
                     raise CacheError(f"state '{r.name}': dtype {r.dtype} is not supported")
                 st_keys.setdefault((r.name, tuple(r.shape), r.dtype), []).append(entry)
             else:
                 raise CacheError(f"cache entry {entry}: unknown request {r!r}")
-    kv_groups = [KVGroupLayout(k[0], k[1], k[2], tuple(v), k[3]) for k, v in kv_keys.items()]     # v_head_dim 0: no value pages
+    kv_groups = [KVGroupLayout(k[0], k[1], k[2], tuple(v), k[3], k[4]) for k, v in kv_keys.items()]     # v_head_dim 0: no value pages
     st_groups = [StateGroupLayout(k[1], k[2], tuple(v), k[0]) for k, v in st_keys.items()]
     return kv_groups, st_groups
 

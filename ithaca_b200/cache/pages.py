@@ -7,7 +7,7 @@ of ``page_size`` positions drawn from a pool; a slot's block table maps
 position // page_size to a page.  Layers with different needs form groups with
 pools of their own: a group that keeps every key never releases a page before
 the slot is freed; a group with a window releases pages that no later query can
-reach.  Slots and pages go back to their pools when a sequence ends and are
+reach (those of a sequence's first ``keep_first`` keys stay).  Slots and pages go back to their pools when a sequence ends and are
 handed out again.
 """
 from __future__ import annotations
@@ -69,6 +69,7 @@ class KVGroupLayout:
     window: Optional[int]            # None: every key is kept
     cache_entries: tuple             # cache entries (of the schedule) stored in this group, in order
     v_head_dim: Optional[int] = None # size of a value head; None: as the key head; 0: the values lie in the key rows
+    keep_first: int = 0              # under a window: the first keys of a sequence that stay visible to every later query
 
 
 @dataclass(frozen=True)
@@ -193,11 +194,15 @@ class SlotTable:
             first_needed = max(0, new_len + 1 - grp.window)
             dead_cols = first_needed // self.page_size
             row = self.tables[g][slot]
-            for i in range(int(self._first_live[g][slot]), dead_cols):
+            for i in range(max(int(self._first_live[g][slot]), self._kept_cols(grp)), dead_cols):
                 if row[i] >= 0:
                     self.pools[g].give_back(int(row[i]))
                     row[i] = -1
             self._first_live[g][slot] = max(int(self._first_live[g][slot]), dead_cols)
+
+    def _kept_cols(self, grp: KVGroupLayout) -> int:
+        """Table columns that a windowed group never releases: the pages of its kept first keys."""
+        return -(-grp.keep_first // self.page_size)
 
     def truncate(self, slot: int, n: int) -> None:
         """Keeps the first ``n`` positions (the reference's ``rewind``, src/model.cpp:1047-1058).
@@ -220,7 +225,8 @@ class SlotTable:
         for g, grp in enumerate(self.kv_groups):
             if grp.window is not None and n < self.length[slot]:
                 first_needed = max(0, n + 1 - grp.window)
-                if first_needed // self.page_size < self._first_live[g][slot]:
+                # the released columns are those between the kept ones and the first live one
+                if max(first_needed // self.page_size, self._kept_cols(grp)) < self._first_live[g][slot]:
                     raise CacheError(f"slot {slot}: group {g} has released the pages a truncation to {n} would need")
         self.length[slot] = n
 

@@ -17,6 +17,7 @@ from .llama import LlamaConfig
 from .mimadra import MimadraConfig
 from .tiralix import TiralixConfig
 from .vebisun import VebisunConfig
+from .zomipel import ZomipelConfig
 
 
 @dataclass(frozen=True)
@@ -71,3 +72,4 @@ register_architecture(VebisunConfig.ARCHITECTURE, VebisunConfig)
 register_architecture(TiralixConfig.ARCHITECTURE, TiralixConfig)
 register_architecture(MimadraConfig.ARCHITECTURE, MimadraConfig)
 register_architecture(GunenexConfig.ARCHITECTURE, GunenexConfig)
+register_architecture(ZomipelConfig.ARCHITECTURE, ZomipelConfig)

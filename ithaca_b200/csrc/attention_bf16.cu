@@ -11,7 +11,8 @@
 //    group's query heads, one chunk of keys) and reads every key and value of its chunk
 //    exactly once for all its heads (the reference's k_attn_gqa, src/gpu_kernels.cpp:154-245),
 //    on the same mma.sync tiles as prefill with the heads as the tile's rows.
-//    Chunks start at absolute multiples of the chunk length; each block writes an
+//    Chunks are cut from the list of pages the query sees (without a window they start at absolute multiples of the chunk
+//    length); each block writes an
 //    unnormalised partial (max, sum, output) and a second kernel merges the partials of a
 //    head in chunk order (k_attn_comb, src/gpu_kernels.cpp:131-150).
 //
@@ -76,12 +77,17 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// The pages a tile of queries walks: those of the first `keep` keys, which stay visible behind a window, then those from the
+// first query's window on.  Page number i of the walk; n_kept = how many of the first kind come before page p_lo.
+__device__ __forceinline__ int kept_pages(int keep, int p_lo) { return min((keep + PAGE - 1) / PAGE, p_lo); }
+__device__ __forceinline__ int page_at(int i, int n_kept, int p_lo) { return i < n_kept ? i : p_lo + i - n_kept; }
+
 // ------------------------------------------------------------------------------------------ prefill
 template <int NW>
 __global__ void __launch_bounds__(32 * NW)
 attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                     bf16* __restrict__ out, const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
-                    const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window,
+                    const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window, int keep,
                     int sink, const float* __restrict__ sink_v, int n_pages, int* status) {
     ik_pdl_wait();
     ik_pdl_launch_dependents();
@@ -99,7 +105,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
     const int rows = min(BM, n_new - row0);
     const int pos_lo = start + row0, pos_hi = start + row0 + rows - 1;
     const int j_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
-    const int p_lo = j_lo / PAGE, p_hi = pos_hi / PAGE;
+    const int p_lo = j_lo / PAGE, n_kept = kept_pages(keep, p_lo), n_iter = n_kept + pos_hi / PAGE - p_lo + 1;
     const int kvh = h / (nh / nkv);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
 
@@ -122,7 +128,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
             cp16(vs + r * LD + c * 8, vg + r * HD + c * 8, true);
         }
     };
-    load_page(0, p_lo);
+    load_page(0, page_at(0, n_kept, p_lo));
     cp_commit();
 
     uint32_t qf[HD / 16][4];
@@ -139,13 +145,13 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
     const int my_pos[2] = {pos_lo + warp * 16 + g, pos_lo + warp * 16 + g + 8};
     const bool my_row[2] = {warp * 16 + g < rows, warp * 16 + g + 8 < rows};
 
-    for (int p = p_lo; p <= p_hi; p++) {
-        const int stage = (p - p_lo) & 1;
-        if (p + 1 <= p_hi) load_page(stage ^ 1, p + 1);
+    for (int it = 0; it < n_iter; it++) {
+        const int stage = it & 1, p = page_at(it, n_kept, p_lo);
+        if (it + 1 < n_iter) load_page(stage ^ 1, page_at(it + 1, n_kept, p_lo));
         cp_commit();
         cp_wait<1>();
         __syncthreads();
-        if (p == p_lo) {
+        if (it == 0) {
             #pragma unroll
             for (int ks = 0; ks < HD / 16; ks++)
                 ldsm4(qf[ks], Qs + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + ks * 16 + (lane >> 4) * 8);
@@ -175,7 +181,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
             #pragma unroll
             for (int e = 0; e < 4; e++) {
                 const int r = e >> 1, j = jbase + n * 8 + (e & 1);
-                const bool ok = my_row[r] && j <= my_pos[r] && (window <= 0 || j > my_pos[r] - window);
+                const bool ok = my_row[r] && j <= my_pos[r] && (window <= 0 || j > my_pos[r] - window || j < keep);
                 const float v = ok ? ik_capped(s[n][e], scale_log2e, cap_log2e) : -INFINITY;
                 s[n][e] = v;
                 mx[r] = fmaxf(mx[r], v);
@@ -272,7 +278,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                        const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
                        const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
                        const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e,
-                       int window, int sink, const float* __restrict__ sink_v, int n_pages, int* status) {
+                       int window, int keep, int sink, const float* __restrict__ sink_v, int n_pages, int* status) {
     extern __shared__ __align__(1024) unsigned char tc_smem[];
     ik_pdl_wait();
     ik_pdl_launch_dependents();
@@ -288,7 +294,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     const int rows = min(TC_BM, n_new - row0);
     const int pos_lo = start + row0, pos_hi = pos_lo + rows - 1;
     const int j_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
-    const int p_lo = j_lo / PAGE, n_iter = pos_hi / PAGE - p_lo + 1;
+    const int p_lo = j_lo / PAGE, n_kept = kept_pages(keep, p_lo), n_iter = n_kept + pos_hi / PAGE - p_lo + 1;
     const int kvh = h / (nh / nkv);
 
     // The swizzled tiles need 1024-byte alignment.  Dynamic shared memory of a kernel without static shared
@@ -344,7 +350,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             for (int bx = 0; bx < TC_BOXES; bx++)
                 tma_load_2d(Qs + bx * (TC_BM * 128), &map_q, h * HD + bx * 64, q_begin + row0, q_full);
             auto page_row = [&](int i) -> int {
-                int page = table[(size_t)b * table_stride + p_lo + i];
+                int page = table[(size_t)b * table_stride + page_at(i, n_kept, p_lo)];
                 if (page < 0 || page >= n_pages) { ik_set_status(status, IK_STATUS_READ_NO_PAGE); page = 0; }
                 return (page * nkv + kvh) * PAGE;
             };
@@ -412,7 +418,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         float m = sink ? (sink_v ? sink_v[h] * 1.4426950408889634f : 0.f) : -INFINITY, l = sink ? 1.f : 0.f;
         bool ok = true;
         for (int i = 0; i < n_iter && ok; i++) {
-            const int p = p_lo + i;
+            const int p = page_at(i, n_kept, p_lo);
             ok = mbar_wait(s_full + (i & 1), (i >> 1) & 1, abort_flag, status, IK_WAIT_LIMIT_NS, 17, i);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -425,7 +431,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 for (int c = 0; c < PAGE; c++) sc[c] = cap_log2e * ik_tanh_fast(sc[c] * scale_log2e);
             }
             const float mul = cap_log2e != 0.f ? 1.f : scale_log2e;
-            const bool need_mask = (p * PAGE + PAGE - 1 > pos_lo) || (window > 0 && p * PAGE < pos_hi + 1 - window);
+            const bool need_mask = (p * PAGE + PAGE - 1 > pos_lo) || (window > 0 && p * PAGE < pos_hi + 1 - window && p * PAGE + PAGE > keep);
             // Few instructions per score: the maximum is taken over the raw scores and scaled once (the scale is
             // positive), and the scaling of a score is folded into the subtraction of the reference below.  Four
             // independent chains for the maximum (and for the sum): a dependent chain's latency would show.  Rows
@@ -436,7 +442,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 #pragma unroll
                 for (int c = 0; c < PAGE; c++) {
                     const int j = p * PAGE + c;
-                    const bool in = row_valid && j <= pos_r && (window <= 0 || j > pos_r - window);
+                    const bool in = row_valid && j <= pos_r && (window <= 0 || j > pos_r - window || j < keep);
                     sc[c] = in ? sc[c] : -INFINITY;
                     mx4[c & 3] = fmaxf(mx4[c & 3], sc[c]);
                 }
@@ -546,7 +552,7 @@ template <int NS>
 __global__ void __launch_bounds__(128)
 attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                    float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ kv_lens,
-                   const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window,
+                   const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window, int keep,
                    int n_pages, int chunk_pages, int n_splits, int* status) {
     ik_pdl_wait();
     constexpr int CH = HD / 8;
@@ -560,9 +566,10 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
     const int kvh = blockIdx.y / n_hc, hc = blockIdx.y % n_hc;
     const int len = kv_lens[b], pos = len - 1;
     const int j0 = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
-    const int p_first = max(split * chunk_pages, j0 / PAGE);
-    const int p_last = min((split + 1) * chunk_pages - 1, pos / PAGE);
-    if (p_first > p_last) return;                                  // nothing of this chunk is visible
+    // chunks of the pages the query sees, in their order (without a window: of all pages)
+    const int p_lo = j0 / PAGE, n_kept = kept_pages(keep, p_lo), n_seen = n_kept + pos / PAGE - p_lo + 1;
+    const int i_first = split * chunk_pages, i_last = min((split + 1) * chunk_pages, n_seen) - 1;
+    if (i_first > i_last) return;                                  // there is no such chunk
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int h0 = kvh * G + hc * 16;                               // first query head of this block
@@ -588,7 +595,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
     };
     #pragma unroll
     for (int s = 0; s < NS; s++) {
-        if (p_first + s <= p_last) load_page(s, p_first + s);
+        if (i_first + s <= i_last) load_page(s, page_at(i_first + s, n_kept, p_lo));
         cp_commit();
     }
 
@@ -601,11 +608,11 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
     float m_i[2] = {-INFINITY, -INFINITY}, l_i[2] = {0.f, 0.f};
     const bool my_row[2] = {g < n_here, g + 8 < n_here};
 
-    for (int p = p_first; p <= p_last; p++) {
-        const int stage = (p - p_first) % NS;
+    for (int i = i_first; i <= i_last; i++) {
+        const int stage = (i - i_first) % NS, p = page_at(i, n_kept, p_lo);
         cp_wait<NS - 1>();
         __syncthreads();
-        if (p == p_first) {
+        if (i == i_first) {
             #pragma unroll
             for (int ks = 0; ks < HD / 16; ks++)
                 ldsm4(qf[ks], Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * LD + ks * 16 + (lane >> 4) * 8);
@@ -631,7 +638,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
             #pragma unroll
             for (int e = 0; e < 4; e++) {
                 const int r = e >> 1, j = jbase + n * 8 + (e & 1);
-                const bool ok = my_row[r] && j <= pos && j >= j0;
+                const bool ok = my_row[r] && j <= pos && (j >= j0 || j < keep);
                 const float v = ok ? ik_capped(s[n][e], scale_log2e, cap_log2e) : -INFINITY;
                 s[n][e] = v;
                 mx[r] = fmaxf(mx[r], v);
@@ -675,7 +682,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
             mma(o[2 * dp + 1], pa, bfr[2], bfr[3]);
         }
         __syncthreads();                                            // everyone is done with this stage
-        if (p + NS <= p_last) load_page(stage, p + NS);
+        if (i + NS <= i_last) load_page(stage, page_at(i + NS, n_kept, p_lo));
         cp_commit();
     }
     cp_wait<0>();
@@ -720,23 +727,23 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
 
 // Merges the partials of each (sequence, head) in chunk order and writes the normalised output.
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                    bf16* __restrict__ out, const int* __restrict__ kv_lens, int nh, int window,
+                                    bf16* __restrict__ out, const int* __restrict__ kv_lens, int nh, int window, int keep,
                                     int sink, const float* __restrict__ sink_v, int chunk_pages, int n_splits) {
     ik_pdl_wait();
     ik_pdl_launch_dependents();
     const int b = blockIdx.x, h = blockIdx.y;
     const int len = kv_lens[b], pos = len - 1;
     const int j0 = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
-    const int s_first = (j0 / PAGE) / chunk_pages, s_last = (pos / PAGE) / chunk_pages;
+    const int p_lo = j0 / PAGE, s_last = (kept_pages(keep, p_lo) + pos / PAGE - p_lo) / chunk_pages;
     const size_t base = ((size_t)b * nh + h) * n_splits;
     // a sink joins the merge as one more part: score 0 (or the head's own, in base-2 units), sum 1, no values
     const float m_sink = sink ? (sink_v ? sink_v[h] * 1.4426950408889634f : 0.f) : -INFINITY;
     float mm = m_sink;
-    for (int s = s_first; s <= s_last; s++) mm = fmaxf(mm, part_ml[(base + s) * 2]);
+    for (int s = 0; s <= s_last; s++) mm = fmaxf(mm, part_ml[(base + s) * 2]);
     const float m_use = mm == -INFINITY ? 0.f : mm;
     for (int x = threadIdx.x; x < HD; x += blockDim.x) {
         float acc = 0.f, ll = sink ? exp2f(m_sink - m_use) : 0.f;
-        for (int s = s_first; s <= s_last; s++) {
+        for (int s = 0; s <= s_last; s++) {
             const float a = exp2f(part_ml[(base + s) * 2] - m_use);
             acc += part_o[(base + s) * HD + x] * a;
             ll += part_ml[(base + s) * 2 + 1] * a;
@@ -756,7 +763,7 @@ IK_EXPORT int ik_attn_take_wait_record(int* out4) { return ik_take_wait_record(o
 
 IK_EXPORT int ik_attn_prefill(const void* q, const void* k_pages, const void* v_pages, void* out, const int* cu_seqlens,
                               const int* kv_lens, const int* table, int table_stride, int B, int max_new, int nh,
-                              int nkv, float scale, float softcap, int window, int sink, const float* sink_v, int page_size, int n_pages, int* status,
+                              int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, int page_size, int n_pages, int* status,
                               cudaStream_t stream) {
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     if (B <= 0 || max_new <= 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size != PAGE || B > 65535 || nh > 65535)
@@ -771,14 +778,14 @@ IK_EXPORT int ik_attn_prefill(const void* q, const void* k_pages, const void* v_
     dim3 grid((max_new + BM - 1) / BM, nh, B);
     IK_RETURN_IF_ERROR(ik_launch(kern, grid, 32 * NW, smem, stream, (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, (bf16*)out,
                                           cu_seqlens, kv_lens, table, table_stride, nh, nkv,
-                                          sc_a, sc_b, window, sink, sink_v, n_pages, status));
+                                          sc_a, sc_b, window, keep, sink, sink_v, n_pages, status));
     IK_LAUNCH_STATUS();
 }
 
 // The tcgen05 kernel (head sizes 64 and 128; IK_UNSUPPORTED otherwise).  T: rows of q.
 IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void* v_pages, void* out, const int* cu_seqlens,
                                  const int* kv_lens, const int* table, int table_stride, int T, int B, int max_new, int nh,
-                                 int nkv, float scale, float softcap, int window, int sink, const float* sink_v, int page_size, int n_pages, int* status,
+                                 int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, int page_size, int n_pages, int* status,
                                  cudaStream_t stream) {
 #if IK_HD == 64 || IK_HD == 128
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
@@ -799,7 +806,7 @@ IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void*
     if (e != cudaSuccess) return (int)e;
     dim3 grid((max_new + TC_BM - 1) / TC_BM, nh, B);
     IK_RETURN_IF_ERROR(ik_launch(kern, grid, 192, TC_SMEM, stream, mq, mk, mv, (bf16*)out, cu_seqlens, kv_lens, table,
-                                 table_stride, nh, nkv, sc_a, sc_b, window, sink, sink_v, n_pages, status));
+                                 table_stride, nh, nkv, sc_a, sc_b, window, keep, sink, sink_v, n_pages, status));
     IK_LAUNCH_STATUS();
 #else
     return IK_UNSUPPORTED;
@@ -807,10 +814,11 @@ IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void*
 }
 
 // part_o: [B, nh, n_splits, HD] floats, part_ml: [B, nh, n_splits, 2] floats, both owned by the caller.
-// n_splits must cover the longest sequence: n_splits * chunk_pages * 64 >= max kv length.
+// n_splits must cover the pages the longest sequence's query sees: n_splits * chunk_pages >= their number (without a window: all
+// its pages; with one: those of the first `keep` keys and those the window reaches into).
 IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_pages, void* out, float* part_o,
                              float* part_ml, const int* kv_lens, const int* table, int table_stride, int B, int nh,
-                             int nkv, float scale, float softcap, int window, int sink, const float* sink_v, int page_size, int n_pages, int chunk_pages,
+                             int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, int page_size, int n_pages, int chunk_pages,
                              int n_splits, int ring_kb, int* status, cudaStream_t stream) {
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     if (B <= 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size != PAGE || chunk_pages <= 0 || n_splits <= 0 ||
@@ -833,7 +841,7 @@ IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_p
             if (e0 != cudaSuccess) return (int)e0;                                                                   \
         }                                                                                                            \
         IK_RETURN_IF_ERROR(ik_launch(kern, grid, 128, smem, stream, (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, part_o, part_ml, \
-                                          kv_lens, table, table_stride, nh, nkv, sc_a, sc_b, window, \
+                                          kv_lens, table, table_stride, nh, nkv, sc_a, sc_b, window, keep, \
                                           n_pages, chunk_pages, n_splits, status));                                   \
     }
     if (ns == 2) IK_DEC(2) else if (ns == 3) IK_DEC(3) else IK_DEC(4)
@@ -841,7 +849,7 @@ IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_p
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
     dim3 grid2(B, nh);
-    IK_RETURN_IF_ERROR(ik_launch_family(IK_FAMILY_ATTENTION_MERGE, attn_combine_kernel, grid2, HD < 128 ? HD : 128, 0, stream, part_o, part_ml, (bf16*)out, kv_lens, nh, window,
+    IK_RETURN_IF_ERROR(ik_launch_family(IK_FAMILY_ATTENTION_MERGE, attn_combine_kernel, grid2, HD < 128 ? HD : 128, 0, stream, part_o, part_ml, (bf16*)out, kv_lens, nh, window, keep,
                                                                     sink, sink_v, chunk_pages, n_splits));
     IK_LAUNCH_STATUS();
 }

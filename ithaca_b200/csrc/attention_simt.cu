@@ -2,14 +2,15 @@
 //
 // One block per (query token, head).  Keys run from j0 to the token's own position
 // (causal by loop bound; j0 > 0 only under a window), in tiles of 128 that start at
-// absolute multiples of 128, so the order in which a query's keys are reduced depends
+// absolute multiples of 128 (the tiles of the first `keep` keys, which stay visible behind the window, come first), so the order in which a query's keys are reduced depends
 // only on its position, not on how the tokens were cut into steps or batched.
 // Scores, the running maximum, the sum and the output are float; exp is the accurate
 // function.  This is the 32-bit path's attention and the fallback for head sizes the
 // tensor-core kernels do not take.  Options: a cap on the scores, s <- cap * tanh(s / cap) after the scale
 // (cap 0 = none), value heads of another size than the key heads (hdv), values that are the leading hdv columns of the
 // key rows themselves (v_pages = k_pages with ldv = hd: a latent that serves as key and value), and a sink: one more
-// key of score 0 that carries no value, so that the weights are exp(s_j) / (1 + sum exp(s_j)).
+// key of score 0 that carries no value, so that the weights are exp(s_j) / (1 + sum exp(s_j)).  Under a window the first
+// `keep` keys of the sequence may stay visible to every later query.
 #include <math.h>
 #define IK_FAMILY 4
 #include "common.cuh"
@@ -24,7 +25,7 @@ __global__ void __launch_bounds__(TILE)
 attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pages, const TC* __restrict__ v_pages,
                       TO* __restrict__ out, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                       const int* __restrict__ table, int table_stride, int nh, int nkv, int hd, int hdv, int ldv, float scale,
-                      float softcap, int window, int sink, const float* __restrict__ sink_v, int page_size, int n_pages, int* status) {
+                      float softcap, int window, int keep, int sink, const float* __restrict__ sink_v, int page_size, int n_pages, int* status) {
     ik_pdl_wait();
     ik_pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smem[];
@@ -48,9 +49,11 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pages, 
     for (int r = 0; r < MAX_R; r++) o[r] = 0.f;
     __syncthreads();
 
-    for (int base = (j0 / TILE) * TILE; base <= pos; base += TILE) {
-        const int j = base + tid;
-        const bool valid = j >= j0 && j <= pos;
+    // every tile visited holds at least one visible key
+    const int kept_tiles = (keep + TILE - 1) / TILE;
+    for (int tile = keep > 0 ? 0 : j0 / TILE; tile * TILE <= pos; tile = tile + 1 >= kept_tiles ? max(tile + 1, j0 / TILE) : tile + 1) {
+        const int base = tile * TILE, j = base + tid;
+        const bool valid = (j >= j0 || j < keep) && j <= pos;
         float s = -INFINITY;
         size_t off = 0;
         if (valid) {
@@ -104,17 +107,17 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pages, 
 
 IK_EXPORT int ik_attention_simt(const void* q, int q_dtype, const void* k_pages, const void* v_pages, int cache_dtype,
                                 void* out, int out_dtype, const int* token_seq, const int* token_pos, const int* table,
-                                int table_stride, int T, int nh, int nkv, int hd, int hdv, int ldv, float scale, float softcap, int window,
+                                int table_stride, int T, int nh, int nkv, int hd, int hdv, int ldv, float scale, float softcap, int window, int keep,
                                 int sink, const float* sink_v, int page_size, int n_pages, int* status, cudaStream_t stream) {
     if (ldv < hdv) return IK_BAD_ARGUMENT;
-    if (T < 0 || nh <= 0 || nkv <= 0 || nh % nkv || hd <= 0 || hdv <= 0 || hdv > TILE * MAX_R || page_size <= 0 || softcap < 0.f) return IK_BAD_ARGUMENT;
+    if (T < 0 || nh <= 0 || nkv <= 0 || nh % nkv || hd <= 0 || hdv <= 0 || hdv > TILE * MAX_R || page_size <= 0 || softcap < 0.f || keep < 0) return IK_BAD_ARGUMENT;
     if (q_dtype != out_dtype) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
     dim3 grid(T, nh);
     const size_t smem = (size_t)(hd + TILE + 32) * sizeof(float) + TILE * sizeof(size_t);
 #define IK_ATT(TQ, TC)                                                                                                \
     IK_RETURN_IF_ERROR(ik_launch(attention_simt_kernel<TQ, TC, TQ>, grid, TILE, smem, stream, (const TQ*)q, (const TC*)k_pages, (const TC*)v_pages, \
-        (TQ*)out, token_seq, token_pos, table, table_stride, nh, nkv, hd, hdv, ldv, scale, softcap, window, sink, sink_v, page_size, n_pages, status))
+        (TQ*)out, token_seq, token_pos, table, table_stride, nh, nkv, hd, hdv, ldv, scale, softcap, window, keep, sink, sink_v, page_size, n_pages, status))
     if (q_dtype == IK_F32 && cache_dtype == IK_F32) IK_ATT(float, float);
     else if (q_dtype == IK_BF16 && cache_dtype == IK_BF16) IK_ATT(__nv_bfloat16, __nv_bfloat16);
     else if (q_dtype == IK_F32 && cache_dtype == IK_BF16) IK_ATT(float, __nv_bfloat16);

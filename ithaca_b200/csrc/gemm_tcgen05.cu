@@ -524,6 +524,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             bf16* const kv_base = (rotated ? rope.k_pages : rope.v_pages) +
                                   (size_t)(head - rope.nh - (rotated ? 0 : rope.nkv)) * rope.page_size * rope.hd + r0;
             const float2* const cs_base = reinterpret_cast<const float2*>(rope.cos_sin) + (r0 >> 1);
+            const bool biased = fused_rope && rope.bias && feature < N;
+            const float bias0 = biased ? rope.bias[f0] : 0.f, bias1 = biased ? rope.bias[f0 + 1] : 0.f;
             // The plain epilogue (whole sums of this block, to Y or added to Y): 32 columns a turn, both halves of the
             // accumulator asked for before either is waited for.
             if (!fused_rope && !swiglu && !slice_sums && !CL && c_hi == c_lo) {
@@ -571,7 +573,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                     #pragma unroll
                     for (int c = 0; c < 8; c++) {
                         const float other = __shfl_xor_sync(0xffffffffu, odd ? v[c] : v[c + 8], 1);
-                        const float a = odd ? other : v[c], b = odd ? v[c + 8] : other;
+                        const float a = (odd ? other : v[c]) + bias0, b = (odd ? v[c + 8] : other) + bias1;
                         packed[c] = __floats2bfloat162_rn(a * cs[c].x - b * cs[c].y, a * cs[c].y + b * cs[c].x);
                     }
                     if (feature < N) {

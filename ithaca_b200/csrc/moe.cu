@@ -6,7 +6,9 @@
 //             score = 1 the sigmoid of every logit by itself.  Experts form `n_groups` equal groups of
 //             neighbours; a group counts by its best score, only experts of the `keep` best groups can be chosen
 //             (n_groups <= 1: all can), and the `top` best of them are.  The weights are the chosen experts' scores as
-//             they are, or divided by their sum (renorm).  Equal scores: the lower index wins.
+//             they are, or divided by their sum (renorm).  Equal scores: the lower index wins.  A bias may join the
+//             logits (`bias` [E]), and the router may have one row more, whose sigmoid goes to `gate` [T] (the weight of an
+//             expert that every token uses).
 //   sort      a counting sort of the A = T * top assignments by expert: sorted[] lists assignment ids (t * top + k)
 //             expert by expert; tiles[] cuts every expert's run into row tiles of MOE_BM for the products.
 //   gemm      for every row tile, rows of X (chosen through `sorted`) times the tile's expert's matrix.  Mode 0:
@@ -14,7 +16,8 @@
 //             sorted place.  Mode 1: X = h at the sorted place, W = down, result at the assignment's own row a.
 //             CUDA cores, float accumulation in ascending k per output element: a row's result does not depend on
 //             its place in a tile nor on what else is in the step.
-//   combine   y[t] = sum_k weight[t, k] * out[t * top + k], ascending k.
+//   combine   y[t] = sum_k weight[t, k] * out[t * top + k], ascending k, plus extra_weight[t] * extra[t] when there is one more
+//             result per token; stored or added to y.
 //
 // The bfloat16 path runs the two products on the tcgen05 product's grouped mode instead (gemm_tcgen05.cu).  For that
 // the sort lays the assignments out in padded order: every expert's rows start at a multiple of the token tile's
@@ -89,8 +92,8 @@ __device__ __forceinline__ void route_token(float* sc, float* gb, int lane, int*
 
 // From ready-made logits: one warp per token.  smem: scores [E] then group bests [n_groups] per warp.
 __global__ void __launch_bounds__(128)
-moe_route_kernel(const float* __restrict__ logits, int* __restrict__ chosen, float* __restrict__ weight, int T, int E,
-                 int top, int n_groups, int keep, int renorm, int score) {
+moe_route_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ bias, int* __restrict__ chosen,
+                 float* __restrict__ weight, float* __restrict__ gate, int T, int E, int top, int n_groups, int keep, int renorm, int score) {
     ik_pdl_wait();
     IK_AFTER_WAIT(logits);
     ik_pdl_launch_dependents();
@@ -100,7 +103,8 @@ moe_route_kernel(const float* __restrict__ logits, int* __restrict__ chosen, flo
     if (t >= T) return;
     const int ng = n_groups > 1 ? n_groups : 0;
     float* sc = sm + (size_t)warp * (E + ng);
-    for (int e = lane; e < E; e += 32) sc[e] = logits[(size_t)t * E + e];
+    for (int e = lane; e < E; e += 32) sc[e] = logits[(size_t)t * ldl + e] + (bias ? bias[e] : 0.f);
+    if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-logits[(size_t)t * ldl + E]));
     __syncwarp();
     route_token(sc, sc + E, lane, chosen + (size_t)t * top, weight + (size_t)t * top, E, top, ng, keep, renorm, score);
 }
@@ -113,8 +117,8 @@ moe_route_kernel(const float* __restrict__ logits, int* __restrict__ chosen, flo
 // Few tokens (decode): one token a block and 32 warps, so that a token's experts are spread over many warps.
 template <int TOK, int THREADS, typename TX>
 __global__ void __launch_bounds__(THREADS)
-moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, int* __restrict__ chosen, float* __restrict__ weight,
-                  int T, int K, int E, int top, int n_groups, int keep, int renorm, int score, int ldx) {
+moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, const float* __restrict__ bias, int* __restrict__ chosen,
+                  float* __restrict__ weight, float* __restrict__ gate, int T, int K, int E, int top, int n_groups, int keep, int renorm, int score, int ldx) {
     ik_pdl_wait();
     IK_AFTER_WAIT(x);
     ik_pdl_launch_dependents();
@@ -122,6 +126,7 @@ moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, int* _
     const int ng = n_groups > 1 ? n_groups : 0;
     float* xs = sm;                                   // [TOK][K]
     float* lg = sm + (size_t)TOK * K;                 // [TOK][E + ng]
+    const int ER = E + (gate ? 1 : 0);                // rows of the router
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * TOK;
     constexpr int V = 16 / (int)sizeof(TX);            // activations per 16-byte load
@@ -152,10 +157,10 @@ moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, int* _
     const float4* xs4 = reinterpret_cast<const float4*>(xs);
     // four experts a pass: an activation read from shared memory serves four products
     constexpr int EB = 4, NW = THREADS / 32;
-    for (int e0 = warp; e0 < E; e0 += NW * EB) {
+    for (int e0 = warp; e0 < ER; e0 += NW * EB) {
         const float4* w4[EB];
         #pragma unroll
-        for (int j = 0; j < EB; j++) w4[j] = reinterpret_cast<const float4*>(wr + (size_t)min(e0 + j * NW, E - 1) * K);
+        for (int j = 0; j < EB; j++) w4[j] = reinterpret_cast<const float4*>(wr + (size_t)min(e0 + j * NW, ER - 1) * K);
         float acc[EB][TOK];
         #pragma unroll
         for (int j = 0; j < EB; j++)
@@ -165,7 +170,7 @@ moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, int* _
         for (int k = lane; k < K4; k += 32) {
             float4 wv[EB];
             #pragma unroll
-            for (int j = 0; j < EB; j++) wv[j] = (j == 0 || e0 + j * NW < E) ? __ldg(w4[j] + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int j = 0; j < EB; j++) wv[j] = (j == 0 || e0 + j * NW < ER) ? __ldg(w4[j] + k) : make_float4(0.f, 0.f, 0.f, 0.f);
             #pragma unroll
             for (int i = 0; i < TOK; i++) {
                 const float4 xv = xs4[i * K4 + k];
@@ -177,12 +182,14 @@ moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, int* _
         #pragma unroll
         for (int j = 0; j < EB; j++) {
             const int e = e0 + j * NW;
-            if (e >= E) break;
+            if (e >= ER) break;
             #pragma unroll
             for (int i = 0; i < TOK; i++) {
                 float v = acc[j][i];
                 for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-                if (lane == 0) lg[i * (E + ng) + e] = v;
+                if (lane != 0) continue;
+                if (e < E) lg[i * (E + ng) + e] = bias ? v + bias[e] : v;
+                else if (t0 + i < T) gate[t0 + i] = 1.0f / (1.0f + expf(-v));
             }
         }
     }
@@ -396,11 +403,14 @@ __global__ void moe_gather_scaled_kernel(const __nv_bfloat16* __restrict__ x, co
 
 // ------------------------------------------------------------------------------------------ combine
 __global__ void moe_combine_kernel(const float* __restrict__ parts, const float* __restrict__ weight, const int* __restrict__ row_of,
-                                   float* __restrict__ y, int T, int top, int d) {
+                                   const float* __restrict__ extra, const float* __restrict__ extra_weight, float* __restrict__ y, int T,
+                                   int top, int d, int accumulate) {
     ik_pdl_wait();
     IK_AFTER_WAIT(parts);
     IK_AFTER_WAIT(weight);
     IK_AFTER_WAIT(row_of);
+    IK_AFTER_WAIT(extra);
+    IK_AFTER_WAIT(extra_weight);
     ik_pdl_launch_dependents();
     const size_t total = (size_t)T * d, stride = (size_t)gridDim.x * blockDim.x;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += stride) {
@@ -408,7 +418,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ parts, const float*
         const int i = (int)(idx - t * d);
         float acc = 0.f;
         for (int k = 0; k < top; k++) acc = fmaf(weight ? weight[t * top + k] : 1.0f, parts[(size_t)(row_of ? row_of[t * top + k] : t * top + k) * d + i], acc);
-        y[idx] = acc;
+        if (extra) acc = fmaf(extra_weight ? extra_weight[t] : 1.0f, extra[idx], acc);
+        y[idx] = accumulate ? y[idx] + acc : acc;
     }
 }
 
@@ -435,19 +446,20 @@ int launch_gemm(const void* X, int x_dtype, const void* W, int w_dtype, void* Y,
 
 IK_EXPORT int ik_moe_tile_rows() { return MOE_BM; }
 
-IK_EXPORT int ik_moe_route(const float* logits, int* chosen, float* weight, int T, int E, int top, int n_groups, int keep,
-                           int renorm, int score, cudaStream_t stream) {
-    if (T < 0 || E <= 0 || top <= 0 || top > E) return IK_BAD_ARGUMENT;
+// logits [T, E] (rows ldl apart; with `gate` one column more)
+IK_EXPORT int ik_moe_route(const float* logits, int ldl, const float* bias, int* chosen, float* weight, float* gate, int T, int E, int top,
+                           int n_groups, int keep, int renorm, int score, cudaStream_t stream) {
+    if (T < 0 || E <= 0 || top <= 0 || top > E || ldl < E + (gate ? 1 : 0)) return IK_BAD_ARGUMENT;
     if (n_groups > 1 && (E % n_groups || keep <= 0 || keep > n_groups || top > keep * (E / n_groups))) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
     const size_t smem = 4 * (size_t)(E + (n_groups > 1 ? n_groups : 0)) * sizeof(float);
     if (smem > 48 * 1024) return IK_UNSUPPORTED;
-    IK_RETURN_IF_ERROR(ik_launch(moe_route_kernel, (T + 3) / 4, 128, smem, stream, logits, chosen, weight, T, E, top, n_groups, keep, renorm, score));
+    IK_RETURN_IF_ERROR(ik_launch(moe_route_kernel, (T + 3) / 4, 128, smem, stream, logits, ldl, bias, chosen, weight, gate, T, E, top, n_groups, keep, renorm, score));
     IK_LAUNCH_STATUS();
 }
 
-// x [T, K] (float or bfloat16, rows ldx apart), wr [E, K] float -> chosen, weight [T, top]
-IK_EXPORT int ik_moe_router(const void* x, int x_dtype, const float* wr, int* chosen, float* weight, int T, int K, int E, int top,
+// x [T, K] (float or bfloat16, rows ldx apart), wr [E, K] float (with `gate` [E + 1, K]) -> chosen, weight [T, top], gate [T]
+IK_EXPORT int ik_moe_router(const void* x, int x_dtype, const float* wr, const float* bias, int* chosen, float* weight, float* gate, int T, int K, int E, int top,
                             int n_groups, int keep, int renorm, int score, int ldx, cudaStream_t stream) {
     if (T < 0 || E <= 0 || K <= 0 || top <= 0 || top > E || ldx < K) return IK_BAD_ARGUMENT;
     if (n_groups > 1 && (E % n_groups || keep <= 0 || keep > n_groups || top > keep * (E / n_groups))) return IK_BAD_ARGUMENT;
@@ -467,7 +479,7 @@ IK_EXPORT int ik_moe_router(const void* x, int x_dtype, const float* wr, int* ch
             cudaError_t e0 = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
             if (e0 != cudaSuccess) return (int)e0;                                                                         \
         }                                                                                                                  \
-        IK_RETURN_IF_ERROR(ik_launch(kern, (T + TOK - 1) / TOK, THREADS, smem, stream, (const TX*)x, wr, chosen, weight, T, K, E, top, \
+        IK_RETURN_IF_ERROR(ik_launch(kern, (T + TOK - 1) / TOK, THREADS, smem, stream, (const TX*)x, wr, bias, chosen, weight, gate, T, K, E, top, \
                                      n_groups, keep, renorm, score, ldx));                                                        \
     }
     if (x_dtype == IK_F32) { if (tok == 1) IK_ROUTER(1, float) else if (tok == 4) IK_ROUTER(4, float) else IK_ROUTER(8, float) }
@@ -528,11 +540,13 @@ IK_EXPORT int ik_moe_gather_scaled(const void* x, const int* src_token, const in
     IK_LAUNCH_STATUS();
 }
 
-// row_of: where assignment a's result lies in `parts` (nullptr: at row a); weight nullptr: every weight is 1
-IK_EXPORT int ik_moe_combine(const float* parts, const float* weight, const int* row_of, float* y, int T, int top, int d, cudaStream_t stream) {
+// row_of: where assignment a's result lies in `parts` (nullptr: at row a); weight nullptr: every weight is 1; extra [T, d] (or
+// nullptr) joins times extra_weight [T] (nullptr: 1)
+IK_EXPORT int ik_moe_combine(const float* parts, const float* weight, const int* row_of, const float* extra, const float* extra_weight, float* y,
+                             int T, int top, int d, int accumulate, cudaStream_t stream) {
     if (T < 0 || top <= 0 || d <= 0) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
     const size_t total = (size_t)T * d, want = (total + 255) / 256, cap = (size_t)ik_sm_count() * 16;
-    IK_RETURN_IF_ERROR(ik_launch(moe_combine_kernel, (int)(want < cap ? want : cap), 256, 0, stream, parts, weight, row_of, y, T, top, d));
+    IK_RETURN_IF_ERROR(ik_launch(moe_combine_kernel, (int)(want < cap ? want : cap), 256, 0, stream, parts, weight, row_of, extra, extra_weight, y, T, top, d, accumulate));
     IK_LAUNCH_STATUS();
 }

@@ -85,7 +85,7 @@ _SIGNATURES = {
     "ik_rope_table": [_vp, _vp, _vp, _i, _i, _vp],
     "ik_gemm_qkv_rope_mma": [_vp, _vp, _i, _i, _i, _i, _i, _vp, _vp],
     "ik_gemm_qkv_rope_tcgen05": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp],
-    "ik_attention_simt": [_vp, _i, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _vp, _i, _i, _vp, _vp],
+    "ik_attention_simt": [_vp, _i, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _i, _i, _vp, _vp],
     "ik_gemm_simt_batched": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _u64, _u64, _u64, _vp],
     "ik_scale_add_norm": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _vp],
     "ik_plain_act": [_vp, _vp, _i, _u64, _i, _vp],
@@ -99,11 +99,11 @@ _SIGNATURES = {
     "ik_conv_rope_append": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i,
                             _i, _i, _i, _i, _i, _vp, _vp],
     "ik_moe_tile_rows": [],
-    "ik_moe_route": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
-    "ik_moe_router": [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "ik_moe_route": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "ik_moe_router": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
     "ik_moe_sort": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "ik_moe_gemm": [_i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp],
-    "ik_moe_combine": [_vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "ik_moe_combine": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
     "ik_moe_sort_padded": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp],
     "ik_moe_gather": [_vp, _vp, _vp, _i, _i, _vp],
     "ik_moe_gather_scaled": [_vp, _vp, _vp, _vp, _vp, _i, _i, _vp],
@@ -120,6 +120,9 @@ _SIGNATURES = {
     "ik_glu_act": [_vp, _vp, _i, _i, _i, _i, _f, _f, _f, _vp],
     "ik_causal_conv": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "ik_selective_scan": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "ik_ssd": [_i, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "ik_ssd_decode": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "ik_gated_group_norm": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _f, _vp],
     "ik_decay_attention": [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "ik_norm_rope_append": [_vp, _i, _i, _i, _i, _vp, _vp, _f, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _f, _i, _i, _i, _i,
                             _i, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp],
@@ -543,7 +546,7 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] =
 class RopeStore(ctypes.Structure):
     """Mirror of IkRopeStore (rope_store.cuh): where the fused q/k/v product puts its results."""
     _fields_ = [("q_out", _vp), ("k_pages", _vp), ("v_pages", _vp), ("cos_sin", _vp), ("token_seq", _vp),
-                ("token_pos", _vp), ("table", _vp), ("status", _vp), ("table_stride", _i), ("nh", _i), ("nkv", _i),
+                ("token_pos", _vp), ("table", _vp), ("status", _vp), ("bias", _vp), ("table_stride", _i), ("nh", _i), ("nkv", _i),
                 ("hd", _i), ("page_size", _i), ("n_pages", _i), ("write_cache", _i)]
 
 
@@ -561,8 +564,8 @@ def rope_table(token_pos: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
 def gemm_qkv_rope(x: torch.Tensor, w: torch.Tensor, q_out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                   cos_sin: torch.Tensor, token_seq: torch.Tensor, token_pos: torch.Tensor, table: torch.Tensor,
                   n_heads: int, n_kv_heads: int, head_dim: int, write_cache: bool, status: Optional[torch.Tensor],
-                  skinny_max: int = 16, splits: Optional[int] = None) -> bool:
-    """q, k, v = x W^T with rotary pairs in adjacent rows of W; rotated q to ``q_out``, rotated k and v into
+                  skinny_max: int = 16, splits: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> bool:
+    """q, k, v = x W^T (+ ``bias``, a float vector over W's rows) with rotary pairs in adjacent rows of W; rotated q to ``q_out``, rotated k and v into
     the pages.  Returns False when the kernels do not take these sizes (the caller then runs the steps apart)."""
     _need(x, "x", torch.bfloat16, contiguous=False)
     _need(w, "w", torch.bfloat16, contiguous=False)
@@ -575,13 +578,14 @@ def gemm_qkv_rope(x: torch.Tensor, w: torch.Tensor, q_out: torch.Tensor, k_pages
     N = w.shape[0]
     n_pages, nkv, page_size, hd = k_pages.shape
     if (N != (n_heads + 2 * n_kv_heads) * head_dim or nkv != n_kv_heads or hd != head_dim or head_dim % 2
-            or cos_sin.shape != (M, head_dim // 2, 2) or q_out.shape != (M, n_heads * head_dim)):
+            or cos_sin.shape != (M, head_dim // 2, 2) or q_out.shape != (M, n_heads * head_dim)
+            or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != N or not bias.is_contiguous()))):
         raise KernelError("gemm_qkv_rope: the sizes do not fit together")
     if K % 8 or x.stride(0) % 8 or w.stride(0) % 8 or x.data_ptr() % 16 or w.data_ptr() % 16 or x.stride(1) != 1 \
             or w.stride(1) != 1:
         return False
     rs = RopeStore(_ptr(q_out), _ptr(k_pages), _ptr(v_pages), _ptr(cos_sin), _ptr(token_seq), _ptr(token_pos),
-                   _ptr(table), _ptr(status), table.stride(0), n_heads, n_kv_heads, head_dim, page_size, n_pages,
+                   _ptr(table), _ptr(status), _ptr(bias), table.stride(0), n_heads, n_kv_heads, head_dim, page_size, n_pages,
                    1 if write_cache else 0)
     _work(f"gemm_{'skinny' if M <= skinny_max else 'tcgen05'} +rope+cache {M}x{N}x{K}", 2 * (M * K + N * K + M * N), 2 * M * N * K)
     if M <= skinny_max:
@@ -624,12 +628,13 @@ def sink_values(sink, n_heads: int) -> Optional[torch.Tensor]:
 def attention_simt(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, token_seq: torch.Tensor,
                    token_pos: torch.Tensor, table: torch.Tensor, n_heads: int, scale: float, window: int,
                    status: Optional[torch.Tensor], out: Optional[torch.Tensor] = None, softcap: float = 0.0, sink=False,
-                   values_in_keys: int = 0) -> torch.Tensor:
+                   values_in_keys: int = 0, keep: int = 0) -> torch.Tensor:
     """``softcap``: scores become cap * tanh(score / cap) after the scale (0 = no cap).  The value pages may
     have a head size of their own; the output is then [T, n_heads * that size].  ``sink``: one more key of score 0
     that carries no value (the weights are exp(s_j) / (1 + sum exp(s_j))); a float32 tensor [n_heads] instead of True gives
     every head's sink a score of its own (not scaled).  ``values_in_keys`` = n > 0: a key row's
-    leading n columns are its value (``v_pages`` is not read)."""
+    leading n columns are its value (``v_pages`` is not read).  ``keep``: under a window the first ``keep`` keys stay
+    visible to every later query."""
     _need(q, "q")
     _need(k_pages, "k_pages")
     _need(table, "table", torch.int32)
@@ -649,7 +654,7 @@ def attention_simt(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor
     _work(f"attention_simt {T}x{n_heads}", _nbytes(q, out))
     _check(lib().ik_attention_simt(_ptr(q), _code(q), _ptr(k_pages), _ptr(v_pages), _code(k_pages), _ptr(out),
                                    _code(out), _ptr(token_seq), _ptr(token_pos), _ptr(table), table.stride(0), T,
-                                   n_heads, nkv, hd, hdv, ldv, scale, softcap, window, sink_flag(sink), _ptr(sink_values(sink, n_heads)),
+                                   n_heads, nkv, hd, hdv, ldv, scale, softcap, window, keep, sink_flag(sink), _ptr(sink_values(sink, n_heads)),
                                    page_size, n_pages, _ptr(status), _stream()),
            "attention_simt")
     return out
@@ -732,34 +737,49 @@ def conv_rope_append(qkv: torch.Tensor, conv_w: Optional[torch.Tensor], ring: Op
 MOE_SCORES = {"softmax": 0, "sigmoid": 1}
 
 
-def moe_route(logits: torch.Tensor, top: int, n_groups: int = 0, keep: int = 0, renorm: bool = False, score: str = "softmax"):
+def _router_extras(T: int, E: int, bias: Optional[torch.Tensor], gate: Optional[torch.Tensor]) -> None:
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+    if gate is not None:
+        _need(gate, "gate", torch.float32)
+    if (bias is not None and bias.numel() != E) or (gate is not None and gate.numel() != T):
+        raise KernelError("moe router: the bias needs one number per expert, the gate one per token")
+
+
+def moe_route(logits: torch.Tensor, top: int, n_groups: int = 0, keep: int = 0, renorm: bool = False, score: str = "softmax",
+              bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
     """Scores over the experts (``score``: the softmax over all logits, or the sigmoid of each by itself) and the ``top`` best among the ``keep`` best of ``n_groups`` groups of
-    neighbours (0 groups: among all).  Returns (chosen int32 [T, top], weights float [T, top])."""
+    neighbours (0 groups: among all).  ``bias`` [E] float is added to the logits.  ``gate`` [T] float: the logits have one
+    column more, whose sigmoid is written there.  Returns (chosen int32 [T, top], weights float [T, top])."""
     _need(logits, "logits", torch.float32)
     T, E = logits.shape
+    E -= gate is not None
+    _router_extras(T, E, bias, gate)
     chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     weight = torch.empty((T, top), dtype=torch.float32, device=logits.device)
     _work(f"moe_route {T}x{E}", _nbytes(logits, chosen, weight))
-    _check(lib().ik_moe_route(_ptr(logits), _ptr(chosen), _ptr(weight), T, E, top, n_groups, keep, 1 if renorm else 0,
+    _check(lib().ik_moe_route(_ptr(logits), logits.shape[1], _ptr(bias), _ptr(chosen), _ptr(weight), _ptr(gate), T, E, top, n_groups, keep, 1 if renorm else 0,
                               MOE_SCORES[score], _stream()), "moe_route")
     return chosen, weight
 
 
 def moe_router(x: torch.Tensor, router: torch.Tensor, top: int, n_groups: int = 0, keep: int = 0, renorm: bool = False,
-               score: str = "softmax"):
+               score: str = "softmax", bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
     """The router's logits ``x router^T`` (float products and sums, whatever type ``x`` has) and the routing of
     ``moe_route``, in one kernel.  Returns (chosen int32 [T, top], weights float [T, top]), or None when the kernel does
-    not take these sizes (the caller forms the logits with a product and routes them)."""
+    not take these sizes (the caller forms the logits with a product and routes them).  ``bias`` [E] float is added to the
+    logits.  ``gate`` [T] float: ``router`` has one row more, and the sigmoid of its product is written there."""
     _need(x, "x", contiguous=False)
     _need(router, "router", torch.float32)
     T, K = x.shape
-    E = router.shape[0]
+    E = router.shape[0] - (gate is not None)
+    _router_extras(T, E, bias, gate)
     if router.shape[1] != K or x.stride(1) != 1:
         raise KernelError("moe_router: the sizes do not fit together")
     chosen = torch.empty((T, top), dtype=torch.int32, device=x.device)
     weight = torch.empty((T, top), dtype=torch.float32, device=x.device)
     _work(f"moe_router {T}x{E}x{K}", T * K * x.element_size() + E * K * 4 + 8 * T * top, 2 * T * E * K)
-    st = lib().ik_moe_router(_ptr(x), _code(x), _ptr(router), _ptr(chosen), _ptr(weight), T, K, E, top, n_groups, keep,
+    st = lib().ik_moe_router(_ptr(x), _code(x), _ptr(router), _ptr(bias), _ptr(chosen), _ptr(weight), _ptr(gate), T, K, E, top, n_groups, keep,
                              1 if renorm else 0, MOE_SCORES[score], x.stride(0), _stream())
     if st == -2:
         return None
@@ -878,9 +898,11 @@ def gemm_tcgen05_grouped(x: torch.Tensor, w: torch.Tensor, plan: MoEPaddedPlan, 
 
 
 def moe_combine(parts: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None,
-                row_of: Optional[torch.Tensor] = None, unweighted: bool = False) -> torch.Tensor:
-    """y[t] = sum_k weight[t, k] * parts[row_of[t * top + k]] (``row_of`` None: row t * top + k).  ``unweighted``: a plain sum
-    (``weight`` then only gives the shape)."""
+                row_of: Optional[torch.Tensor] = None, unweighted: bool = False, extra: Optional[torch.Tensor] = None,
+                extra_weight: Optional[torch.Tensor] = None, accumulate: bool = False) -> torch.Tensor:
+    """y[t] (+)= sum_k weight[t, k] * parts[row_of[t * top + k]] (``row_of`` None: row t * top + k).  ``unweighted``: a plain sum
+    (``weight`` then only gives the shape).  ``extra`` [T, d] float: one more result for every token, times ``extra_weight``
+    [T] (None: as it is)."""
     _need(parts, "parts", torch.float32)
     _need(weight, "weight", torch.float32)
     T, top = weight.shape
@@ -888,10 +910,16 @@ def moe_combine(parts: torch.Tensor, weight: torch.Tensor, out: Optional[torch.T
     if row_of is None and parts.shape[0] != T * top:
         raise KernelError("moe_combine: one row per (token, choice) is needed")
     if out is None:
+        if accumulate:
+            raise KernelError("moe_combine: accumulate needs an output to add to")
         out = torch.empty((T, d), dtype=torch.float32, device=parts.device)
-    _work(f"moe_combine {T}x{d}", _nbytes(parts, out))
-    _check(lib().ik_moe_combine(_ptr(parts), 0 if unweighted else _ptr(weight), _ptr(row_of), _ptr(out), T, top, d, _stream()),
-           "moe_combine")
+    _need(out, "out", torch.float32)
+    if out.shape != (T, d) or (extra is not None and (extra.shape != (T, d) or extra.dtype != torch.float32 or not extra.is_contiguous())) \
+            or (extra_weight is not None and (extra_weight.numel() != T or extra_weight.dtype != torch.float32)):
+        raise KernelError("moe_combine: the sizes do not fit together")
+    _work(f"moe_combine {T}x{d}", _nbytes(extra, out) + (_nbytes(out) if accumulate else 0) + T * top * d * 4)
+    _check(lib().ik_moe_combine(_ptr(parts), 0 if unweighted else _ptr(weight), _ptr(row_of), _ptr(extra), _ptr(extra_weight), _ptr(out),
+                                T, top, d, 1 if accumulate else 0, _stream()), "moe_combine")
     return out
 
 
@@ -1556,4 +1584,97 @@ def row_decay(rule: str, u: torch.Tensor, x1_off: int, k_off: int, v_off: int, d
                             _ptr(ctx.slots), _ptr(ctx.cu_seqlens), _ptr(ctx.kv_lens), _ptr(out), T, ctx.n_seqs, H, G, dk, dv,
                             1 if ctx.is_decode else 0, _stream())
     _check(st, "row_decay")
+    return out
+
+
+# ---------------------------------------------------------------------------------------------
+# State-space duality: a matrix state per head with one decay per token and head
+def _ssd_sizes(state: torch.Tensor, A: torch.Tensor, D: torch.Tensor, dt_bias: torch.Tensor, n_groups: int):
+    _need(state, "state", torch.float32)
+    _, two, H, N, P = state.shape
+    for name, v in (("A", A), ("D", D), ("dt_bias", dt_bias)):
+        _need(v, name, torch.float32)
+        if v.numel() != H:
+            raise KernelError(f"ssd: {name} needs one number per head")
+    if two != 2 or H % n_groups:
+        raise KernelError("ssd: the sizes do not fit together")
+    return H, N, P
+
+
+def ssd(u: torch.Tensor, p: torch.Tensor, dt_off: int, dt_bias: torch.Tensor, A: torch.Tensor, D: torch.Tensor, state: torch.Tensor,
+        ctx, n_groups: int, chunks: Optional[bool] = None) -> torch.Tensor:
+    """S <- exp(A dt) S + dt B x^T;  y = S^T C + D x per head, over the step's tokens, with dt = softplus(raw + dt_bias).
+    ``u`` [T, H P + 2 G N]: x, B, C behind their convolution; the raw steps are columns ``dt_off``.. of ``p`` (float);
+    ``A`` [H] negative; ``state`` [slots, 2, H, N, P] float.  ``chunks``: True = the tensor-core kernel that takes 64 tokens at
+    a time (bfloat16 ``u``), False = token by token, None = chunks where they apply and a sequence may bring several
+    tokens.  Returns y [T, H P] float."""
+    _need(u, "u")
+    _need(p, "p", torch.float32, contiguous=False)
+    H, N, P = _ssd_sizes(state, A, D, dt_bias, n_groups)
+    T = u.shape[0]
+    if u.shape[1] != H * P + 2 * n_groups * N or p.stride(1) != 1 or dt_off + H > p.shape[1] or p.shape[0] != T:
+        raise KernelError("ssd: the sizes do not fit together")
+    out = torch.empty((T, H * P), dtype=torch.float32, device=u.device)
+    nbytes = T * (u.shape[1] * u.element_size() + 4 * H * (P + 1)) + 8 * ctx.n_seqs * H * N * P
+    exact = u.dtype == torch.float32
+    must = bool(chunks)
+    if chunks is None:
+        chunks = u.dtype == torch.bfloat16 and not ctx.is_decode
+
+    def run(kind):
+        return lib().ik_ssd(kind, _ptr(u), _code(u), u.stride(0), _ptr(p), p.stride(0), dt_off, _ptr(dt_bias), _ptr(A), _ptr(D), _ptr(state),
+                            _ptr(ctx.slots), _ptr(ctx.cu_seqlens), _ptr(ctx.kv_lens), _ptr(out), T, ctx.n_seqs, H, n_groups, N, P,
+                            1 if exact else 0, _stream())
+    if chunks:
+        _work(f"ssd chunks {T}x{H}x{N}x{P}", nbytes, T * H * (4 * N * P + 64 * (N + P)))
+        st = run(1)
+        if st != -2 or must:
+            _check(st, "ssd")
+            return out
+    _work(f"ssd {T}x{H}x{N}x{P}", nbytes, 5 * T * H * N * P)
+    _check(run(0), "ssd")
+    return out
+
+
+def ssd_decode(p: torch.Tensor, x_off: int, conv_w: torch.Tensor, conv_b: torch.Tensor, ring: Optional[torch.Tensor], dt_bias: torch.Tensor,
+               A: torch.Tensor, D: torch.Tensor, state: torch.Tensor, ctx, n_groups: int) -> Optional[torch.Tensor]:
+    """One token per sequence: the short convolution (``conv_w`` [taps, channels] tap-major, ``ring`` [slots, taps, channels]) with
+    silu and the step of ``ssd`` in one kernel.  ``p`` [B, ...] float: x, B, C from ``x_off``, then the raw steps.  Returns None when
+    the kernel does not take these sizes."""
+    _need(p, "p", torch.float32, contiguous=False)
+    _need(conv_w, "conv_w", torch.float32)
+    _need(conv_b, "conv_b", torch.float32)
+    H, N, P = _ssd_sizes(state, A, D, dt_bias, n_groups)
+    B, C = p.shape[0], H * P + 2 * n_groups * N
+    taps = conv_w.shape[0]
+    if conv_w.shape[1] != C or conv_b.numel() != C or p.stride(1) != 1 or x_off + C + H > p.shape[1] or B != ctx.n_seqs or not ctx.is_decode:
+        raise KernelError("ssd_decode: the sizes do not fit together")
+    if taps > 1:
+        _need(ring, "ring", torch.float32)
+        if tuple(ring.shape[1:]) != (taps, C):
+            raise KernelError("ssd_decode: the ring has the wrong shape")
+    out = torch.empty((B, H * P), dtype=torch.float32, device=p.device)
+    _work(f"ssd decode {B}x{H}x{N}x{P}", B * (8 * H * N * P + 4 * C * (taps + 1) + 4 * H * P), 5 * B * H * N * P)
+    st = lib().ik_ssd_decode(_ptr(p), p.stride(0), x_off, _ptr(conv_w), _ptr(conv_b), _ptr(ring) if taps > 1 else 0, _ptr(dt_bias), _ptr(A),
+                             _ptr(D), _ptr(state), _ptr(ctx.slots), _ptr(ctx.cu_seqlens), _ptr(ctx.kv_lens), _ptr(out), B, H, n_groups,
+                             N, P, taps, _stream())
+    if st == -2:
+        return None
+    _check(st, "ssd_decode")
+    return out
+
+
+def gated_group_norm(x: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """g = x * silu(z), every one of ``groups`` equal parts of a row divided by its own root mean square (``eps`` inside the
+    root), times ``weight``.  ``z`` may be a column range of a wider float matrix."""
+    _need(x, "x", torch.float32)
+    _need(z, "z", torch.float32, contiguous=False)
+    _need(weight, "weight", torch.float32)
+    T, d = x.shape
+    if z.shape != x.shape or z.stride(1) != 1 or weight.numel() != d or d % groups:
+        raise KernelError("gated_group_norm: the sizes do not fit together")
+    out = torch.empty((T, d), dtype=out_dtype, device=x.device)
+    _work(f"gated_group_norm {T}x{d}", T * d * (8 + out.element_size()))
+    _check(lib().ik_gated_group_norm(_ptr(x), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), _code(out), T, groups, d // groups, eps, _stream()),
+           "gated_group_norm")
     return out

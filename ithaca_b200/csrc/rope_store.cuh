@@ -5,7 +5,8 @@
 // are (i, i + head_dim / 2) has the rows of its q and k weights reordered when it is loaded; scores do not
 // change, since q and k are reordered alike).  For token m and pair i the cosine and sine of
 // float(pos_m) * inv_freq_i come from a table made once per step.  Rotated q goes to q_out, rotated k and plain
-// v go to the token's place in the paged cache; the [tokens, features] intermediate is never written.
+// v go to the token's place in the paged cache; the [tokens, features] intermediate is never written.  A bias over the
+// features (in the order of the rows) may join the product first.
 #pragma once
 #include "common.cuh"
 
@@ -18,6 +19,7 @@ struct IkRopeStore {
     const int* token_pos;          // [M] absolute position
     const int* table;              // block table [sequences][table_stride]
     int* status;
+    const float* bias;             // [features] added to the product before the rotation, or null
     int table_stride, nh, nkv, hd, page_size, n_pages, write_cache;
 };
 
@@ -37,6 +39,7 @@ __device__ __forceinline__ int ik_rope_cache_row(const IkRopeStore& e, int m, in
 // (a, b): the product's values at features (f0, f0 + 1) of token m, f0 even.
 __device__ __forceinline__ void ik_rope_store_pair(const IkRopeStore& e, int m, int f0, float a, float b) {
     const int head = f0 / e.hd, r0 = f0 - head * e.hd;
+    if (e.bias) { a += e.bias[f0]; b += e.bias[f0 + 1]; }
     float o0 = a, o1 = b;
     if (head < e.nh + e.nkv) {
         const float2 cs = *reinterpret_cast<const float2*>(e.cos_sin + ((size_t)m * (e.hd >> 1) + (r0 >> 1)) * 2);

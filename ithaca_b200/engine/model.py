@@ -96,7 +96,9 @@ class DecoderModel:
                     continue
                 for n, have in enumerate(out[e.cache]):
                     if isinstance(have, KVRequest) and have.window is not None and (r.window is None or r.window > have.window):
-                        out[e.cache][n] = dataclasses.replace(have, window=r.window)
+                        have = out[e.cache][n] = dataclasses.replace(have, window=r.window)
+                    if isinstance(have, KVRequest) and r.keep_first > have.keep_first:
+                        out[e.cache][n] = dataclasses.replace(have, keep_first=r.keep_first)
         return out
 
     def forward(self, ctx, cache: SequenceCache) -> Optional[torch.Tensor]:

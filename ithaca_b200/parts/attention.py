@@ -29,11 +29,15 @@ Options a spec may give (all off by default):
 * ``sink``: the softmax's denominator counts one more key of score 0 that carries no value: the weights are
   exp(s_j) / (1 + sum exp(s_j)), so a query may attend to nothing.  ``sink: "learned"`` with the tensor ``sink`` [n_heads]:
   every head's sink has a score of its own (not scaled), the denominator's extra term is exp(sink_h).
-* ``bias`` with the tensors ``q_bias``, ``k_bias``, ``v_bias``, ``o_bias``: the four projections add a vector.
+* ``bias`` with the tensors ``q_bias``, ``k_bias``, ``v_bias``, ``o_bias``: the four projections add a vector.  ``bias: "qkv"``: the
+  first three do, and the output projection has none.
+* ``keep_first``: under a window the first ``keep_first`` keys of a sequence stay visible to every later query, at their true
+  positions; the cache never releases their pages.
 * ``v_norm``: every value head is divided by its root mean square (``norm_eps`` inside the root, no weight) and cached so.
 * a position part whose cos and sin carry a constant factor (``magnitude``).
 
-With any of these but the first three the mixer runs "wide": one product gives [q | k | v | g] in float, one kernel norms, rotates
+With ``qk_norm``, ``head_gate``, ``sink``, ``v_norm``, an output bias or a magnitude (and with ``bias: "qkv"`` where the product's own
+epilogue cannot rotate and append) the mixer runs "wide": one product gives [q | k | v | g] in float, one kernel norms, rotates
 and appends, the attention kernel runs, and the gate kernel writes the output projection's operand.  A wide mixer can
 also serve as a branch of a composite (``parts/parallel.py``): ``branch_in()`` / ``branch_out()`` hand out its matrices
 so that the composite stacks them with other branches' into one product each, and ``core`` works on column ranges of
@@ -74,7 +78,9 @@ class Attention:
             out[w["sink"]] = TensorReq((nh,), std=1.0)
         if spec.get("bias"):
             out[w["q_bias"]], out[w["k_bias"]] = TensorReq((nh * hd,)), TensorReq((nkv * hd,))
-            out[w["v_bias"]], out[w["o_bias"]] = TensorReq((nkv * hdv,)), TensorReq((d,))
+            out[w["v_bias"]] = TensorReq((nkv * hdv,))
+            if spec.get("bias") != "qkv":
+                out[w["o_bias"]] = TensorReq((d,))
         taps = spec.get("conv_taps") or 0
         if taps:
             # taps around 1/taps: the convolution keeps the projections' scale
@@ -98,6 +104,10 @@ class Attention:
         self.window = spec.get("window")
         if self.window is not None and self.window <= 0:
             raise ValueError(f"attention: window must be positive, found {self.window}")
+        # without a window every key is visible anyway
+        self.keep_first = int(spec.get("keep_first") or 0) if self.window is not None else 0
+        if self.keep_first < 0:
+            raise ValueError(f"attention: keep_first cannot be negative, found {self.keep_first}")
         scale = spec.get("scale")
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(self.head_dim)
         self.position = position
@@ -117,11 +127,11 @@ class Attention:
         # what the kernels get: False, True (a key of score 0) or every head's score
         self.sink_arg = as_float32(tensors[w["sink"]], runtime) if spec.get("sink") == "learned" else self.sink
         self.v_norm = bool(spec.get("v_norm"))
+        if spec.get("bias") not in (None, False, True, "qkv"):
+            raise ValueError(f"attention: bias {spec.get('bias')!r} is not supported (true, qkv)")
         self.biased = bool(spec.get("bias"))
-        self.wide = bool(qk_norm or self.head_gate or self.sink or self.v_norm or self.biased or (position is not None and getattr(position, "magnitude", 1.0) != 1.0)
-                         or not standalone)
-        if self.wide and self.conv_taps:
-            raise ValueError("attention: a short convolution and the wide arrangement (qk_norm, head_gate) do not go together")
+        self.wide = bool(qk_norm or self.head_gate or self.sink or self.v_norm or (self.biased and spec.get("bias") != "qkv")
+                         or (position is not None and getattr(position, "magnitude", 1.0) != 1.0) or not standalone)
         self.norm_eps = float(spec.get("norm_eps") or 0.0)
         self.q_norm_w = as_float32(tensors[w["q_norm"]], runtime) if qk_norm else None
         self.k_norm_w = as_float32(tensors[w["k_norm"]], runtime) if qk_norm else None
@@ -132,12 +142,19 @@ class Attention:
         self.pairing = position.pairing if position is not None else 0
         self.fused_rope = (runtime.dtype == "bfloat16" and position is not None and position.rotary_dim == self.head_dim
                            and self.head_dim % 2 == 0 and not self.conv_taps and self.v_head_dim == self.head_dim
-                           and not self.wide)
+                           and not self.wide and not (self.biased and self.hidden % 8))
+        if self.biased and not self.fused_rope:
+            self.wide = True
+        if self.wide and self.conv_taps:
+            raise ValueError("attention: a short convolution and the wide arrangement do not go together")
+        bq, bk = (tensors[w["q_bias"]], tensors[w["k_bias"]]) if self.biased else (None, None)
         if self.fused_rope and self.pairing == 0:
             half = self.head_dim // 2
             order = torch.stack((torch.arange(half), torch.arange(half) + half), dim=1).reshape(-1)
             wq = wq.view(self.n_heads, self.head_dim, -1)[:, order].reshape(wq.shape)
             wk = wk.view(self.n_kv_heads, self.head_dim, -1)[:, order].reshape(wk.shape)
+            if self.biased:
+                bq, bk = bq.view(self.n_heads, -1)[:, order].reshape(-1), bk.view(self.n_kv_heads, -1)[:, order].reshape(-1)
             self.pairing = 1                                       # pairs are (2i, 2i + 1) from here on
         self._in = [wq, wk, tensors[w["v"]]] + ([tensors[w["g"]]] if self.head_gate else [])
         self._out = tensors[w["o"]]
@@ -151,8 +168,9 @@ class Attention:
         self._out_bias = None
         if self.biased:
             zeros = torch.zeros(self.n_in - self.g_off, dtype=torch.float32)
-            self.in_bias = torch.cat([tensors[w[r]].to(torch.float32).cpu() for r in ("q_bias", "k_bias", "v_bias")] + [zeros]).to(runtime.device).contiguous()
-            self._out_bias = as_float32(tensors[w["o_bias"]], runtime)
+            self.in_bias = torch.cat([b.to(torch.float32).cpu() for b in (bq, bk, tensors[w["v_bias"]])] + [zeros]).to(runtime.device).contiguous()
+            if spec.get("bias") != "qkv":
+                self._out_bias = as_float32(tensors[w["o_bias"]], runtime)
         if standalone:
             self.qkv = Linear(self._in, runtime)
             self.o = Linear([self._out], runtime)
@@ -178,9 +196,8 @@ class Attention:
         """The vector the output projection adds (float32), or None."""
         return self._out_bias
 
-    def core(self, p: torch.Tensor, mid: torch.Tensor, ctx, cache: LayerCache, writes_cache: bool = True, mult: float = 1.0) -> None:
-        """``p`` [T, n_in] float: [q | k | v | g] (a column range of a wider matrix may be given); ``mid`` [T, n_mid] in the
-        activation type receives ``mult`` times the gated heads, the operand of the output projection."""
+    def _attend_wide(self, p: torch.Tensor, ctx, cache: LayerCache, writes_cache: bool) -> torch.Tensor:
+        """Norms, rotation and append, then the attention itself: the heads' results before their gate."""
         rt, pos = self.runtime, self.position
         q = torch.empty((p.shape[0], self.n_heads * self.head_dim), dtype=rt.act_dtype, device=p.device)
         table = ctx.tables[cache.kv_group]
@@ -188,12 +205,18 @@ class Attention:
                              cache.v_pages, ctx.token_seq, ctx.token_pos, table, pos.inv_freq if pos is not None else None,
                              getattr(pos, "magnitude", 1.0), self.n_heads, pos.rotary_dim if pos is not None else 0,
                              self.pairing, writes_cache, rt.status, per_head=self.norm_per_head, bias=self.in_bias, v_norm=self.v_norm)
-        att = attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, sink=self.sink_arg)
+        return attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, sink=self.sink_arg,
+                      keep=self.keep_first)
+
+    def core(self, p: torch.Tensor, mid: torch.Tensor, ctx, cache: LayerCache, writes_cache: bool = True, mult: float = 1.0) -> None:
+        """``p`` [T, n_in] float: [q | k | v | g] (a column range of a wider matrix may be given); ``mid`` [T, n_mid] in the
+        activation type receives ``mult`` times the gated heads, the operand of the output projection."""
+        att = self._attend_wide(p, ctx, cache, writes_cache)
         ops.head_gate(att, p if self.head_gate else None, self.g_off, mid, self.n_heads, mult, wide=self.gate_wide)
 
     def cache_requests(self) -> List[object]:
         v = self.v_head_dim if self.v_head_dim != self.head_dim else None
-        out: List[object] = [KVRequest(self.n_kv_heads, self.head_dim, self.window, v)]
+        out: List[object] = [KVRequest(self.n_kv_heads, self.head_dim, self.window, v, keep_first=self.keep_first)]
         if self.conv_taps > 1:
             out.append(StateRequest("conv_ring", (self.conv_taps, self.channels), "float32"))
         return out
@@ -205,8 +228,11 @@ class Attention:
         T = x.shape[0]
         if self.wide:
             p = self.qkv(x, out_dtype=torch.float32)
-            mid = torch.empty((T, self.n_mid), dtype=rt.act_dtype, device=x.device)
-            self.core(p, mid, ctx, cache, writes_cache)
+            if self.head_gate:
+                mid = torch.empty((T, self.n_mid), dtype=rt.act_dtype, device=x.device)
+                self.core(p, mid, ctx, cache, writes_cache)
+            else:
+                mid = self._attend_wide(p, ctx, cache, writes_cache)
             self.o(mid, out=residual, accumulate=accumulate)
             if self._out_bias is not None:
                 ops.add_rows_(residual, self._out_bias)
@@ -222,7 +248,9 @@ class Attention:
                 cos_sin = ctx.shared[key] = ops.rope_table(ctx.token_pos, pos.inv_freq)
             done = ops.gemm_qkv_rope(x, self.qkv.weight, q, cache.k_pages, cache.v_pages, cos_sin, ctx.token_seq,
                                      ctx.token_pos, table, self.n_heads, self.n_kv_heads, self.head_dim, writes_cache,
-                                     rt.status)
+                                     rt.status, bias=self.in_bias)
+            if not done and self.biased:
+                raise ValueError("attention: the fused q/k/v product did not take these sizes, and the plain path adds no biases")
         if self.plain_append:
             qkv = self.qkv(x, out_dtype=torch.float32)
             ring = cache.state("conv_ring") if self.conv_taps > 1 else None
@@ -235,22 +263,22 @@ class Attention:
             ops.rope_append(qkv, q, cache.k_pages, cache.v_pages, ctx.token_seq, ctx.token_pos, table,
                             pos.inv_freq if pos is not None else None, self.n_heads, self.n_kv_heads, self.head_dim,
                             pos.rotary_dim if pos is not None else 0, self.pairing, writes_cache, rt.status)
-        att = attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap)
+        att = attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, keep=self.keep_first)
         self.o(att, out=residual, accumulate=accumulate)
 
 
 def attend(q: torch.Tensor, cache: LayerCache, ctx, table: torch.Tensor, n_heads: int, scale: float, window: int,
-           rt: Runtime, softcap: float = 0.0, sink=False) -> torch.Tensor:
+           rt: Runtime, softcap: float = 0.0, sink=False, keep: int = 0) -> torch.Tensor:
     """Chooses the attention kernel: tensor-core kernels for bfloat16 when they take the
     head sizes, else the CUDA-core kernel (always for float32)."""
     if q.dtype == torch.bfloat16 and cache.v_pages.shape[3] == cache.k_pages.shape[3]:
         from ..csrc import attention_bf16
         out = attention_bf16.attend(q, cache.k_pages, cache.v_pages, ctx, table, n_heads, scale, window, rt.status,
-                                    softcap=softcap, sink=sink)
+                                    softcap=softcap, sink=sink, keep=keep)
         if out is not None:
             return out
     return ops.attention_simt(q, cache.k_pages, cache.v_pages, ctx.token_seq, ctx.token_pos, table, n_heads, scale,
-                              window, rt.status, softcap=softcap, sink=sink)
+                              window, rt.status, softcap=softcap, sink=sink, keep=keep)
 
 
 register_mixer("attention", Attention)

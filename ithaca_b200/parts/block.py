@@ -8,6 +8,9 @@ a vector of the layer before it joins the stream: x += s1 * mixer(norm(x)); x +=
 then writes into a float32 buffer of its own, and one kernel adds s1 times it to the stream and forms the feed-forward's
 norm of the new stream in the same pass.  Such a layer may have no feed-forward.
 
+``parallel``: one norm in front of both sublayers, x += mixer(norm(x)) + feed_forward(norm(x)).  The normed row is formed once,
+and both sublayers add into the float stream.  The feed-forward may be absent.
+
 ``sandwich``: a norm in front of and behind each sublayer, and a constant on what joins the
 stream: x += m * norm_out(mixer(norm(x))); x += m * norm_out'(feed_forward(norm'(x))).  The
 sublayer writes into a float32 buffer of its own (the stream is not what it adds to); the norm
@@ -110,6 +113,44 @@ class PreNormBlock:
         xn = ops.scale_add_norm(y, self.mixer_scale, residual, self.ff_norm.weight, self.ff_norm.eps, self.runtime.act_dtype)
         self.feed_forward.forward(xn, ctx, y, accumulate=False)
         ops.scale_add_norm(y, self.ff_scale, residual)
+
+
+class ParallelBlock:
+    @classmethod
+    def manifest(cls, spec: BlockSpec) -> Dict[str, TensorReq]:
+        out: Dict[str, TensorReq] = {}
+        _merge(out, MIXERS.get(spec.mixer.kind).manifest(spec.mixer))
+        if spec.feed_forward is not None:
+            _merge(out, FEED_FORWARDS.get(spec.feed_forward.kind).manifest(spec.feed_forward))
+        _merge(out, NORMS.get(spec.norms["mixer"].kind).manifest(spec.norms["mixer"]))
+        if spec.position is not None:
+            _merge(out, POSITIONS.get(spec.position.kind).manifest(spec.position))
+        return out
+
+    def __init__(self, spec: BlockSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
+        if set(spec.norms) != {"mixer"}:
+            raise ValueError("parallel block: the spec needs one norm, 'mixer', which both sublayers read")
+        position = None
+        if spec.position is not None:
+            position = POSITIONS.get(spec.position.kind)(spec.position, tensors, runtime)
+        mixer_cls = MIXERS.get(spec.mixer.kind)
+        if "position" in inspect.signature(mixer_cls.__init__).parameters:
+            self.mixer = mixer_cls(spec.mixer, tensors, runtime, position=position)
+        else:
+            self.mixer = mixer_cls(spec.mixer, tensors, runtime)
+        self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.feed_forward = FEED_FORWARDS.get(spec.feed_forward.kind)(spec.feed_forward, tensors, runtime)
+        self.norm = NORMS.get(spec.norms["mixer"].kind)(spec.norms["mixer"], tensors, runtime)
+
+    def cache_requests(self) -> List[object]:
+        return list(self.mixer.cache_requests())
+
+    def forward(self, residual: torch.Tensor, ctx, cache: LayerCache, writes_cache: bool = True) -> None:
+        xn = self.norm.forward(residual)                   # before either sublayer adds to the stream
+        self.mixer.forward(xn, ctx, cache, residual, writes_cache)
+        if self.feed_forward is not None:
+            self.feed_forward.forward(xn, ctx, residual)
 
 
 class SandwichBlock:
@@ -315,5 +356,6 @@ class HyperBlock:
 
 register_block("prenorm", PreNormBlock)
 register_block("hyper", HyperBlock)
+register_block("parallel", ParallelBlock)
 register_block("sandwich", SandwichBlock)
 register_block("outnorm", OutNormBlock)

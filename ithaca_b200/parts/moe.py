@@ -1,19 +1,25 @@
 """Mixture of experts: a router and small feed-forwards, of which each token uses a few.
 
 Router: z = Wr x in float32 (x may be the activations' 16-bit rounding), scores = softmax(z)
-over all experts (``score: "sigmoid"``: the sigmoid of every logit by itself).  Experts may form equal groups of neighbours: a group counts by its best
+over all experts (``score: "sigmoid"``: the sigmoid of every logit by itself).  With the tensor ``router_bias`` [experts] a
+bias joins the logits.  Experts may form equal groups of neighbours: a group counts by its best
 score, and only experts of the ``group_keep`` best groups can be chosen.  The ``top`` best of
-them are; their weights are their scores (``renormalize``: divided by their sum).  An expert is
+them are; their weights are their scores (``renormalize``: divided by their sum; with softmax scores that is the softmax over
+the chosen experts' logits).  An expert is
 y = Wd (silu(Wg x) * (Wu x)); the layer's output is the weighted sum of the chosen experts'.
 
 ``expert: "plain"``: an expert is ungated, y = Wd act(Wu x) with ``activation`` ``relu2`` or ``gelu_tanh`` (no ``gate`` tensors).
 ``weight_on: "input"``: the weight multiplies what the expert reads instead of what it gives, y = sum_e expert_e(w_e x); the
 scaled rows are formed (in float, rounded once to the operands' type) while the tokens are gathered into expert order.
 
+``shared: n`` with the tensors ``shared_gate``, ``shared_up``, ``shared_down``: one more gated expert, n wide, that every token
+uses; with the tensor ``shared_weight`` [1, hidden] its result is multiplied by the sigmoid of one number per token, a
+projection that the router's kernel forms as one row more.
+
 On the device: one kernel forms the router's logits and picks experts and weights per token; a counting sort groups the
 (token, choice) pairs by expert; two grouped products run every expert over its rows (the first
 with silu(g) * u as its epilogue, so the [rows, 2 ff] intermediate is never written); a last kernel
-adds a token's choices in the order they were chosen.  Nothing is read back by the host: grids are
+adds a token's choices in the order they were chosen, then the shared expert's result, straight into the stream.  Nothing is read back by the host: grids are
 sized from upper bounds, so a captured step can be replayed.
 
 The bfloat16 path's products are the tcgen05 product in its grouped mode: the pairs are laid out so
@@ -32,7 +38,8 @@ import torch
 from ..config.spec import PartSpec
 from ..csrc import ops
 from ..weights.loader import TensorReq
-from .base import Runtime, register_feed_forward, to_device
+from .base import Runtime, as_float32, register_feed_forward, to_device
+from .feed_forward import GatedMLP
 
 
 class MoEFeedForward:
@@ -55,6 +62,13 @@ class MoEFeedForward:
             out[u], out[dn] = TensorReq((ff, d)), TensorReq((d, ff))
             if g is not None:
                 out[g] = TensorReq((ff, d))
+        w, n = spec.weights, spec.get("shared") or 0
+        if "router_bias" in w:
+            out[w["router_bias"]] = TensorReq((spec["n_experts"],))
+        if n:
+            out[w["shared_gate"]], out[w["shared_up"]], out[w["shared_down"]] = TensorReq((n, d)), TensorReq((n, d)), TensorReq((d, n))
+            if "shared_weight" in w:
+                out[w["shared_weight"]] = TensorReq((1, d))
         return out
 
     def __init__(self, spec: PartSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
@@ -96,6 +110,15 @@ class MoEFeedForward:
         wt = torch.bfloat16 if runtime.dtype == "bfloat16" else None
         # the router stays float32 whatever the path: its products are formed and added in 32 bits
         self.router = to_device(tensors[router], runtime).to(torch.float32).contiguous()
+        w = spec.weights
+        self.router_bias = as_float32(tensors[w["router_bias"]], runtime) if "router_bias" in w else None
+        # a gated expert for every token, and, as the router's last row, the projection behind its weight
+        self.shared = int(spec.get("shared") or 0)
+        self.shared_weighted = bool(self.shared) and "shared_weight" in w
+        if self.shared_weighted:
+            self.router = torch.cat([self.router, as_float32(tensors[w["shared_weight"]], runtime)], dim=0).contiguous()
+        self.shared_expert = GatedMLP(PartSpec("gated_mlp", {"hidden_size": self.hidden, "intermediate_size": self.shared},
+                                               {r: w["shared_" + r] for r in ("gate", "up", "down")}), tensors, runtime) if self.shared else None
 
         def stack(mats):
             t = torch.stack([to_device(m, runtime) for m in mats], dim=0)
@@ -118,10 +141,12 @@ class MoEFeedForward:
 
     def forward(self, x: torch.Tensor, ctx, residual: torch.Tensor, accumulate: bool = True) -> None:
         rt = self.runtime
-        routed = ops.moe_router(x, self.router, self.top, self.n_groups, self.group_keep, self.renormalize, self.score)
+        sg = torch.empty((x.shape[0],), dtype=torch.float32, device=x.device) if self.shared_weighted else None
+        extras = {"bias": self.router_bias, "gate": sg}
+        routed = ops.moe_router(x, self.router, self.top, self.n_groups, self.group_keep, self.renormalize, self.score, **extras)
         if routed is None:                                   # sizes beyond the fused kernel's shared memory
             logits = ops.gemm_simt(x, self.router, out_dtype=torch.float32)
-            routed = ops.moe_route(logits, self.top, self.n_groups, self.group_keep, self.renormalize, self.score)
+            routed = ops.moe_route(logits, self.top, self.n_groups, self.group_keep, self.renormalize, self.score, **extras)
         chosen, weight = routed
         parts = row_of = None
         on_input = self.weight_on_input
@@ -144,10 +169,11 @@ class MoEFeedForward:
                 h = ops.moe_gemm(2, x, self.up, plan, rt.act_dtype, row_scale=weight if on_input else None, act=self.act)
             parts = ops.moe_gemm(1, h, self.down, plan, torch.float32)
             row_of = None
-        if accumulate:
-            ops.add_(residual, ops.moe_combine(parts, weight, row_of=row_of, unweighted=on_input))
-        else:
-            ops.moe_combine(parts, weight, out=residual, row_of=row_of, unweighted=on_input)
+        every = None
+        if self.shared_expert is not None:
+            every = torch.empty((x.shape[0], self.hidden), dtype=torch.float32, device=x.device)
+            self.shared_expert.forward(x, ctx, every, accumulate=False)
+        ops.moe_combine(parts, weight, out=residual, row_of=row_of, unweighted=on_input, extra=every, extra_weight=sg, accumulate=accumulate)
 
 
 register_feed_forward("moe", MoEFeedForward)

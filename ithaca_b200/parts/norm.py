@@ -5,7 +5,8 @@ Layer norm: y = (x - mean) / sqrt(var + eps) * w + b with var the mean of the sq
 deviations, in float32.  A norm may also stand behind a sublayer: ``add_into`` then adds
 ``mult * y`` to the residual stream in the same kernel.  The RMS norm may carry a second vector
 (``scale``, a per-channel "layer scale") that multiplies what it adds to the stream.  With ``scalar_weight`` the RMS
-norm's weight is ONE number for all coordinates (stored as a tensor without dimensions); the kernels get it spread out."""
+norm's weight is ONE number for all coordinates (stored as a tensor without dimensions); the kernels get it spread out.
+With ``unit_offset`` the stored weight is the distance from one: y = x / rms(x) * (1 + w), the sum formed in float at load."""
 from __future__ import annotations
 
 from typing import Dict, Mapping, Optional
@@ -21,7 +22,8 @@ from .base import Runtime, as_float32, register_norm
 class RMSNorm:
     @classmethod
     def manifest(cls, spec: PartSpec) -> Dict[str, TensorReq]:
-        out = {spec.weights["weight"]: TensorReq(() if spec.get("scalar_weight") else (spec["size"],), init="ones")}
+        kind = {"init": "normal", "std": 0.01} if spec.get("unit_offset") else {"init": "ones"}
+        out = {spec.weights["weight"]: TensorReq(() if spec.get("scalar_weight") else (spec["size"],), **kind)}
         if "scale" in spec.weights:
             out[spec.weights["scale"]] = TensorReq((spec["size"],), init="ones")
         return out
@@ -30,6 +32,8 @@ class RMSNorm:
         self.size = int(spec["size"])
         self.eps = float(spec["eps"])
         self.weight = as_float32(tensors[spec.weights["weight"]], runtime)
+        if spec.get("unit_offset"):
+            self.weight = self.weight + 1.0
         if spec.get("scalar_weight"):
             self.weight = self.weight.reshape(1).expand(self.size).contiguous()
         self.scale = as_float32(tensors[spec.weights["scale"]], runtime) if "scale" in spec.weights else None
