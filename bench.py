@@ -17,6 +17,10 @@
                                                                 first one's rows; attention with a learned sink beside token-shift time
                                                                 mixing; routed plain experts) beside a Mimadra of equal width, heads,
                                                                 feed-forward and depth (its closest relative here), in the same form
+    python bench.py --only zomipel [--batch B]                  the Zomipel decoder (parallel layers; state-space duality mixers; windowed
+                                                                attention that keeps the first keys; routed experts beside one that
+                                                                every token uses; a looped span of layers) beside a Tiralix of equal
+                                                                width, heads, active feed-forward and layer runs, in the same form
     python bench.py --config 1b-unequal|13b-long                the other two workloads alone, through Engine.generate
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at the given batch with every
@@ -639,6 +643,41 @@ def gunenex_pair(size, vocab=32000):
     return gun, mim, len(kinds)
 
 
+ZOMIPEL_SIZES = [
+    # name, width, heads, kv heads, head size, ssd heads, ssd values, states, groups, experts, chosen, expert width, shared width,
+    # window, kept, layers, (loop start, stop, times)
+    ("2048 wide, 16 heads of 128, 64 ssd heads of 64 x 128, 16 experts of 1024", 2048, 16, 4, 128, 64, 64, 128, 8, 16, 4, 1024, 4096, 2048, 64,
+     ("mamba2", "attention", "mamba2", "mamba2"), (1, 3, 2)),
+    ("4096 wide, 32 heads of 128, 128 ssd heads of 64 x 128, 8 experts of 3584", 4096, 32, 8, 128, 128, 64, 128, 8, 8, 2, 3584, 7168, 2048, 64,
+     ("mamba2", "attention", "mamba2", "mamba2"), (1, 3, 2)),
+]
+
+
+def zomipel_pair(size, vocab=32000):
+    """The Zomipel configuration of a size and the Tiralix next to it: the same width, attention heads and head size, inner
+    channels of the recurrent layers, as many layers as the Zomipel model has layer runs, a feed-forward as wide as what a
+    token uses of the routed one.  Where Zomipel has its attention Tiralix has its parallel layer (attention beside linear
+    attention), where Zomipel has state-space duality Tiralix has its selective scan of 16 states."""
+    _, d, nh, nkv, hd, H, Pv, N, G, E, top, ff, shared, window, keep, kinds, loop = size
+    ssd = {"heads": H, "vdim": Pv, "state": N, "groups": G, "conv": 4, "norm_groups": G}
+    att = {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "rot": {"base": 500000.0, "dims": hd},
+           "mask": {"size": window, "keep_first": keep}}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": E, "top": top}, "shared": {"ff": shared}}
+    layers = [{"type": k, "mixer": ssd if k == "mamba2" else att, "mlp": {"kind": "dense", "ff": top * ff + shared} if i == 0 else moe}
+              for i, k in enumerate(kinds)]
+    zom = {"architecture": "Zomipel", "vocab": vocab, "width": d, "norm": {"eps": 1e-6}, "layers": layers,
+           "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]}}
+    lo, hi, times = loop
+    runs = list(kinds[:lo]) + list(kinds[lo:hi]) * times + list(kinds[hi:])
+    tiralix, _, _ = tiralix_pair(("", d, nh, nkv, hd, top * ff + shared, H * Pv, 16, d // 16, tuple("mamba1" if k == "mamba2" else "parallel" for k in runs)),
+                                 vocab)
+    return zom, tiralix, len(runs)
+
+
+def zomipel_run(pk, batch, steps, warmup, context=2048, prompt=4096):
+    return vebisun_run(pk, batch, steps, warmup, context, prompt, sizes=ZOMIPEL_SIZES, pair=zomipel_pair, name="zomipel", partner="tiralix")
+
+
 def gunenex_run(pk, batch, steps, warmup, context=2048, prompt=4096):
     return vebisun_run(pk, batch, steps, warmup, context, prompt, sizes=GUNENEX_SIZES, pair=gunenex_pair, name="gunenex", partner="mimadra")
 
@@ -743,7 +782,7 @@ def main():
                     help="with --only decode / prefill: another context length (decode) or prompt length (prefill) than the default run's")
     ap.add_argument("--config", default=None, choices=["1b-unequal", "13b-long"],
                     help="run one of the other workloads alone and print its figures")
-    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "attention", "products", "marginal", "issue-rate", "vebisun", "tiralix", "mimadra", "gunenex"],
+    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "attention", "products", "marginal", "issue-rate", "vebisun", "tiralix", "mimadra", "gunenex", "zomipel"],
                     help="run one part only and print its figures (for profiling a small case)")
     args = ap.parse_args()
 
@@ -779,6 +818,9 @@ def main():
     if args.only == "gunenex":
         print(json.dumps({"only": "gunenex", "peaks": pk, "sizes": gunenex_run(pk, args.batch, min(args.steps, 64), args.warmup)}))
         return 0
+    if args.only == "zomipel":
+        print(json.dumps({"only": "zomipel", "peaks": pk, "sizes": zomipel_run(pk, args.batch, min(args.steps, 64), args.warmup)}))
+        return
     if args.only == "issue-rate":
         # what the thread that issues tensor-core products costs: cycles per instruction, one or two issuing threads
         from ithaca_b200.csrc import ops

@@ -175,7 +175,7 @@ __device__ __forceinline__ float sd_hi(uint32_t w) { return __uint_as_float(w & 
 
 template <int NP, int NW>                                  // states padded to NP (a multiple of 16), warps
 constexpr size_t ssd_chunk_smem() {
-    return (size_t)2 * (2 * Q * (NP + 8) + Q * (16 * NW + 8)) * sizeof(bf16) + (size_t)2 * Q * (Q + 8) * sizeof(bf16) + (size_t)NW * 2 * Q * sizeof(float);
+    return (size_t)2 * (2 * Q * (NP + 8) + Q * (16 * NW + 8)) * sizeof(bf16) + (size_t)2 * Q * (Q + 8) * sizeof(bf16) + (size_t)NW * 3 * Q * sizeof(float);
 }
 
 template <int NP, int NW>
@@ -190,7 +190,7 @@ ssd_chunk_kernel(const bf16* __restrict__ u, int ldu, const float* __restrict__ 
     bf16* Xs = Bs + 2 * Q * LN;                            // [2][Q][LP]
     bf16* Mh = Xs + 2 * Q * LP;                            // [Q][LM] decayed scores, leading part: row i, column j
     bf16* Ml = Mh + Q * LM;                                // ... and the rest
-    float* cw_all = (float*)(Ml + Q * LM);                 // [NW][2][Q]: c_i and dt_i, a copy per warp
+    float* cw_all = (float*)(Ml + Q * LM);                 // [NW][3][Q]: c_i in two parts and dt_i, a copy per warp
     ik_pdl_wait();
     IK_AFTER_WAIT(u);
     IK_AFTER_WAIT(p);
@@ -207,8 +207,12 @@ ssd_chunk_kernel(const bf16* __restrict__ u, int ldu, const float* __restrict__ 
     const float* st_in = state + ((size_t)slots[b] * 2 + ((start - 1) & 1)) * per + (size_t)h * N * P;
     float* st_out = state + ((size_t)slots[b] * 2 + ((end - 1) & 1)) * per + (size_t)h * N * P;
     const float rate = A[h], bias = dt_bias[h], skip = Dv[h];
-    float* cw = cw_all + warp * 2 * Q;
-    float* dw = cw + Q;
+    float* cw = cw_all + warp * 3 * Q;
+    float* cl = cw + Q;
+    float* dw = cl + Q;
+    // exp(c_i - c_j): c may be large (a token that forgets everything) where the difference is small, so c is kept as the sum of
+    // two floats
+    auto decay = [&](int i, int j) -> float { return __expf((cw[i] - cw[j]) + (cl[i] - cl[j])); };
 
     auto load = [&](int t0, int buf) {
         bf16* cs = Cs + buf * Q * LN;
@@ -247,15 +251,16 @@ ssd_chunk_kernel(const bf16* __restrict__ u, int ldu, const float* __restrict__ 
         // steps and their running sums: every warp for itself, lane l the tokens l and l + 32
         {
             const float d0 = t0 + lane < hi ? ik_softplusf(raw0 + bias) : 0.f, d1 = t0 + lane + 32 < hi ? ik_softplusf(raw1 + bias) : 0.f;
-            float s0 = rate * d0, s1 = rate * d1;
+            double s0 = (double)rate * d0, s1 = (double)rate * d1;
             #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
-                const float q0 = __shfl_up_sync(0xffffffffu, s0, o), q1 = __shfl_up_sync(0xffffffffu, s1, o);
+                const double q0 = __shfl_up_sync(0xffffffffu, s0, o), q1 = __shfl_up_sync(0xffffffffu, s1, o);
                 if (lane >= o) { s0 += q0; s1 += q1; }
             }
             s1 += __shfl_sync(0xffffffffu, s0, 31);
             __syncwarp();
-            cw[lane] = s0; cw[lane + 32] = s1;
+            cw[lane] = (float)s0; cw[lane + 32] = (float)s1;
+            cl[lane] = (float)(s0 - (double)(float)s0); cl[lane + 32] = (float)(s1 - (double)(float)s1);
             dw[lane] = d0; dw[lane + 32] = d1;
             __syncwarp();
         }
@@ -294,13 +299,12 @@ ssd_chunk_kernel(const bf16* __restrict__ u, int ldu, const float* __restrict__ 
             for (int n = 0; n < Q / 8; n++) {
                 if (n > 2 * it + 1) break;
                 const int j = n * 8 + 2 * t;
-                const float c0 = cw[j], c1 = cw[j + 1], d0 = dw[j], d1 = dw[j + 1];
+                const float d0 = dw[j], d1 = dw[j + 1];
                 #pragma unroll
                 for (int r = 0; r < 2; r++) {
                     const int i = it * 16 + g + 8 * r;
-                    const float ci = cw[i];
-                    float m0 = j <= i ? sc[n][2 * r] * (__expf(ci - c0) * d0) : 0.f;
-                    float m1 = j + 1 <= i ? sc[n][2 * r + 1] * (__expf(ci - c1) * d1) : 0.f;
+                    float m0 = j <= i ? sc[n][2 * r] * (decay(i, j) * d0) : 0.f;
+                    float m1 = j + 1 <= i ? sc[n][2 * r + 1] * (decay(i, j + 1) * d1) : 0.f;
                     *reinterpret_cast<uint32_t*>(Mh + i * LM + j) = sd_take(m0, m1);
                     *reinterpret_cast<uint32_t*>(Ml + i * LM + j) = sd_take(m0, m1);
                 }
@@ -341,7 +345,7 @@ ssd_chunk_kernel(const bf16* __restrict__ u, int ldu, const float* __restrict__ 
         }
         __syncthreads();                                   // the scores are written
         // 3. the chunk's own tokens, and 4. the state behind them: both read x^T, 16 tokens at a time
-        const float c_last = cw[Q - 1], keep = __expf(c_last);
+        const float keep = __expf(cw[Q - 1]);
         #pragma unroll
         for (int n = 0; n < 2 * KN; n++)
             #pragma unroll
@@ -366,7 +370,7 @@ ssd_chunk_kernel(const bf16* __restrict__ u, int ldu, const float* __restrict__ 
             #pragma unroll
             for (int e = 0; e < 4; e++) {                  // elements e: tokens j = 16 k + 2t, + 1 (e < 2) or + 8, + 9
                 const int j = k * 16 + 2 * t + (e >> 1) * 8;
-                float v0 = sd_lo(xf[e]) * (__expf(c_last - cw[j]) * dw[j]), v1 = sd_hi(xf[e]) * (__expf(c_last - cw[j + 1]) * dw[j + 1]);
+                float v0 = sd_lo(xf[e]) * (decay(Q - 1, j) * dw[j]), v1 = sd_hi(xf[e]) * (decay(Q - 1, j + 1) * dw[j + 1]);
                 wh[e] = sd_take(v0, v1);
                 wl[e] = sd_take(v0, v1);
             }
