@@ -121,6 +121,8 @@ _SIGNATURES = {
     "ik_causal_conv": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "ik_selective_scan": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "ik_ssd": [_i, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "ik_ssd_tcgen05": [_vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp],
+    "ik_ssd_take_wait_record": [_vp],
     "ik_ssd_decode": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "ik_gated_group_norm": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _f, _vp],
     "ik_decay_attention": [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
@@ -928,7 +930,7 @@ def wait_records() -> str:
     error message, empty if none did."""
     found = []
     rec = (ctypes.c_int * 4)()
-    takers = [("matrix product", lib().ik_gemm_tcgen05_take_wait_record)]
+    takers = [("matrix product", lib().ik_gemm_tcgen05_take_wait_record), ("state-space duality", lib().ik_ssd_take_wait_record)]
     from . import attention_bf16
     for hd, m in attention_bf16._modules.items():
         takers.append((f"attention (head size {hd})", m.ik_attn_take_wait_record))
@@ -1601,38 +1603,47 @@ def _ssd_sizes(state: torch.Tensor, A: torch.Tensor, D: torch.Tensor, dt_bias: t
     return H, N, P
 
 
+SSD_KINDS = ("auto", "scan", "mma", "tcgen05")
+
+
 def ssd(u: torch.Tensor, p: torch.Tensor, dt_off: int, dt_bias: torch.Tensor, A: torch.Tensor, D: torch.Tensor, state: torch.Tensor,
-        ctx, n_groups: int, chunks: Optional[bool] = None) -> torch.Tensor:
+        ctx, n_groups: int, kind: str = "auto", status: Optional[torch.Tensor] = None) -> torch.Tensor:
     """S <- exp(A dt) S + dt B x^T;  y = S^T C + D x per head, over the step's tokens, with dt = softplus(raw + dt_bias).
     ``u`` [T, H P + 2 G N]: x, B, C behind their convolution; the raw steps are columns ``dt_off``.. of ``p`` (float);
-    ``A`` [H] negative; ``state`` [slots, 2, H, N, P] float.  ``chunks``: True = the tensor-core kernel that takes 64 tokens at
-    a time (bfloat16 ``u``), False = token by token, None = chunks where they apply and a sequence may bring several
-    tokens.  Returns y [T, H P] float."""
+    ``A`` [H] negative; ``state`` [slots, 2, H, N, P] float.  Returns y [T, H P] float.
+
+    ``kind``: ``scan`` = token by token on the CUDA cores (any sizes, both types); ``mma`` and ``tcgen05`` = chunks of 64 and of
+    128 tokens on the tensor cores, bfloat16 ``u`` only (N <= 128 with N and P multiples of 8; N 64 or 128 with P a multiple of
+    64); ``auto`` = the last of these that takes the sizes, when a sequence may bring several tokens."""
     _need(u, "u")
     _need(p, "p", torch.float32, contiguous=False)
     H, N, P = _ssd_sizes(state, A, D, dt_bias, n_groups)
     T = u.shape[0]
     if u.shape[1] != H * P + 2 * n_groups * N or p.stride(1) != 1 or dt_off + H > p.shape[1] or p.shape[0] != T:
         raise KernelError("ssd: the sizes do not fit together")
+    if kind not in SSD_KINDS:
+        raise KernelError(f"ssd: kind {kind!r} is not known ({', '.join(SSD_KINDS)})")
     out = torch.empty((T, H * P), dtype=torch.float32, device=u.device)
     nbytes = T * (u.shape[1] * u.element_size() + 4 * H * (P + 1)) + 8 * ctx.n_seqs * H * N * P
-    exact = u.dtype == torch.float32
-    must = bool(chunks)
-    if chunks is None:
-        chunks = u.dtype == torch.bfloat16 and not ctx.is_decode
-
-    def run(kind):
-        return lib().ik_ssd(kind, _ptr(u), _code(u), u.stride(0), _ptr(p), p.stride(0), dt_off, _ptr(dt_bias), _ptr(A), _ptr(D), _ptr(state),
-                            _ptr(ctx.slots), _ptr(ctx.cu_seqlens), _ptr(ctx.kv_lens), _ptr(out), T, ctx.n_seqs, H, n_groups, N, P,
-                            1 if exact else 0, _stream())
-    if chunks:
-        _work(f"ssd chunks {T}x{H}x{N}x{P}", nbytes, T * H * (4 * N * P + 64 * (N + P)))
-        st = run(1)
-        if st != -2 or must:
-            _check(st, "ssd")
+    where = (_ptr(p), p.stride(0), dt_off, _ptr(dt_bias), _ptr(A), _ptr(D), _ptr(state), _ptr(ctx.slots), _ptr(ctx.cu_seqlens),
+             _ptr(ctx.kv_lens), _ptr(out), T, ctx.n_seqs, H, n_groups, N, P)
+    several = u.dtype == torch.bfloat16 and not ctx.is_decode
+    if kind == "tcgen05" or (kind == "auto" and several):
+        if u.dtype != torch.bfloat16:
+            raise KernelError("ssd: the tensor-core kernels take bfloat16 inputs")
+        _work(f"ssd tcgen05 {T}x{H}x{N}x{P}", nbytes, T * H * (4 * N * P + 128 * (N + P)))
+        st = lib().ik_ssd_tcgen05(_ptr(u), u.stride(0), *where, _ptr(status), _stream())
+        if st != -2 or kind == "tcgen05":
+            _check(st, "ssd (tcgen05)")
             return out
-    _work(f"ssd {T}x{H}x{N}x{P}", nbytes, 5 * T * H * N * P)
-    _check(run(0), "ssd")
+    if kind == "mma" or (kind == "auto" and several):
+        _work(f"ssd mma {T}x{H}x{N}x{P}", nbytes, T * H * (4 * N * P + 64 * (N + P)))
+        st = lib().ik_ssd(1, _ptr(u), _code(u), u.stride(0), *where, 0, _stream())
+        if st != -2 or kind == "mma":
+            _check(st, "ssd (mma)")
+            return out
+    _work(f"ssd scan {T}x{H}x{N}x{P}", nbytes, 5 * T * H * N * P)
+    _check(lib().ik_ssd(0, _ptr(u), _code(u), u.stride(0), *where, 1 if u.dtype == torch.float32 else 0, _stream()), "ssd")
     return out
 
 

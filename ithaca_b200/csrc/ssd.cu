@@ -15,7 +15,8 @@
 // Three kernels:
 //   ssd_scan     one token after the other on the CUDA cores, any sizes; the float32 path's kernel for prompts and single
 //                tokens alike (a token gives the same bits however a prompt is cut).
-//   ssd_chunk    bfloat16 inputs, prompts: chunks of 64 tokens on the tensor cores.
+//   ssd_chunk    bfloat16 inputs, prompts: chunks of 64 tokens on the warp-level tensor path (ssd_tcgen05.cu has the form for
+//                tcgen05, which takes fewer sizes and is several times faster).
 //   ssd_decode   bfloat16 path, one token per sequence: convolution, step, decay, update and read-out in one pass over the
 //                state.
 #include "common.cuh"

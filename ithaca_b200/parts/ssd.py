@@ -16,7 +16,8 @@ belongs to, so that a decode step never overwrites what it read) and a ring of t
 convolution, float32.  Steps, decays, the state, its sums, the skip, the gate and the norm are float32 on both paths; the
 projections' operands and, for a prompt, the convolution's output are 16-bit on the bfloat16 path.
 
-A prompt on the bfloat16 path runs convolution, then chunks of 64 tokens on the tensor cores (``csrc/ssd.cu``); a decode step
+A prompt on the bfloat16 path runs convolution, then chunks of 128 tokens on tcgen05 (``csrc/ssd_tcgen05.cu``) or, for sizes that
+kernel does not take, of 64 tokens on the warp-level tensor path (``csrc/ssd.cu``); a decode step
 runs convolution, step, decay, update and read-out in one kernel; the float32 path runs the convolution and the recurrence
 token by token, for prompts and single tokens alike.
 """
@@ -98,7 +99,8 @@ class StateSpaceDuality:
             y = ops.ssd_decode(p, self.inner, self.conv_w, self.conv_b, ring, self.dt_bias, self.A, self.D, state, ctx, self.n_groups)
         if y is None:
             u = ops.causal_conv(p[:, self.inner:self.inner + self.channels], self.conv_w, self.conv_b, ring, ctx, rt.act_dtype, act=True)
-            y = ops.ssd(u, p, self.inner + self.channels, self.dt_bias, self.A, self.D, state, ctx, self.n_groups)
+            y = ops.ssd(u, p, self.inner + self.channels, self.dt_bias, self.A, self.D, state, ctx, self.n_groups,
+                        status=rt.status)
         mid = ops.gated_group_norm(y, p[:, :self.inner], self.norm_w, self.norm_groups, self.norm_eps, rt.act_dtype)
         self.o(mid, out=residual, accumulate=accumulate)
 

@@ -198,14 +198,15 @@ def _ssd_plain(u, raw, dt_bias, A_log, D, H, G, N, Pv, state):
 
 
 @pytest.mark.parametrize("slow", [False, True])
-@pytest.mark.parametrize("kind,dtype", [("scan", torch.float32), ("scan", torch.bfloat16), ("chunks", torch.bfloat16)])
+@pytest.mark.parametrize("kind,dtype", [("scan", torch.float32), ("scan", torch.bfloat16), ("mma", torch.bfloat16), ("tcgen05", torch.bfloat16)])
 @pytest.mark.parametrize("H,G,N,Pv", [(4, 2, 16, 24), (3, 3, 40, 8), (2, 1, 128, 64), (6, 1, 24, 16), (1, 1, 64, 136), (4, 4, 8, 32), (5, 1, 12, 10),
-                                      (2, 2, 200, 33)])
+                                      (2, 2, 200, 33), (4, 2, 64, 64), (3, 3, 128, 192), (8, 2, 128, 64)])
 def test_state_space_kernels(kind, dtype, H, G, N, Pv, slow):
     """A prompt, portions and single tokens behind it, three sequences in scattered slots with leftovers in their states; the
     state in both its places and every y."""
     from ithaca_b200.csrc import ops
-    takes_chunks = N <= 128 and N % 8 == 0 and Pv % 8 == 0
+    takes = {"scan": True, "mma": N <= 128 and N % 8 == 0 and Pv % 8 == 0, "tcgen05": N in (64, 128) and Pv % 64 == 0}[kind]
+    status = torch.zeros(1, dtype=torch.int32, device=DEV)
     slots = [3, 0, 2]
     state = torch.randn(4, 2, H, N, Pv, device=DEV)                   # leftovers: a sequence starts from zeros all the same
     plain = {b: None for b in range(3)}
@@ -221,11 +222,12 @@ def test_state_space_kernels(kind, dtype, H, G, N, Pv, slow):
         p = torch.full((u.shape[0], H + 7), 9.0)
         p[:, 5:5 + H] = raw
         args = (u, p.to(DEV), 5, dt_bias.to(DEV), A, D.to(DEV), state, ctx, G)
-        if kind == "chunks" and not takes_chunks:
+        if not takes:
             with pytest.raises(ops.KernelError):
-                ops.ssd(*args, chunks=True)
+                ops.ssd(*args, kind=kind)
             return
-        y = ops.ssd(*args, chunks=kind == "chunks").cpu().double()
+        y = ops.ssd(*args, kind=kind, status=status).cpu().double()
+        assert status.item() == 0
         at = 0
         for b in range(3):
             n = hi[b] - lo[b]
@@ -239,10 +241,32 @@ def test_state_space_kernels(kind, dtype, H, G, N, Pv, slow):
     assert worst < (3e-6 if kind == "scan" and dtype == torch.float32 else 2e-5), worst
 
 
+@pytest.mark.parametrize("kind", ["mma", "tcgen05"])
+def test_long_prompts_in_chunks_against_token_by_token(kind):
+    """Prompts of several chunks with a ragged end, two sequences, a portion behind each: both tensor-core kernels against the
+    token-by-token kernel on the same values, many heads at once."""
+    from ithaca_b200.csrc import ops
+    H, G, N, Pv = 24, 4, 128, 64
+    status = torch.zeros(1, dtype=torch.int32, device=DEV)
+    ends = [1000, 389]
+    data = [_ssd_case(H, G, N, Pv, 20 + b, torch.bfloat16, ends[b], b == 0) for b in range(2)]
+    dt_bias, A, D = data[0][2].to(DEV), -torch.exp(data[0][3].double()).float().to(DEV), data[0][4].to(DEV)
+    states = [torch.randn(2, 2, H, N, Pv, generator=torch.Generator().manual_seed(1)).to(DEV) for _ in range(2)]
+    for lo, hi in (([0, 0], [700, 256]), ([700, 256], [1000, 389])):
+        ctx = _ctx(lo, hi, [1, 0])
+        u = torch.cat([data[b][0][lo[b]:hi[b]] for b in range(2)]).to(DEV)
+        raw = torch.cat([data[b][1][lo[b]:hi[b]] for b in range(2)]).to(DEV).contiguous()
+        got, want = (ops.ssd(u, raw, 0, dt_bias, A, D, st, ctx, G, kind=k, status=status) for st, k in zip(states, (kind, "scan")))
+        assert status.item() == 0 and rel_err(got.cpu().numpy(), want.cpu().numpy()) < 2e-5
+        for b in range(2):
+            a, w = (st[[1, 0][b], (hi[b] - 1) & 1].cpu().numpy() for st in states)
+            assert rel_err(a, w) < 2e-5
+
+
 def test_state_space_scan_gives_the_same_bits_however_it_is_cut():
     from ithaca_b200.csrc import ops
     H, G, N, Pv, n = 4, 2, 24, 40, 90
-    u, raw, dt_bias, A_log, D = (x.to(DEV) for x in _ssd_case(H, G, N, Pv, 3, torch.float32, n, False))
+    u, raw, dt_bias, A_log, D = (v.to(DEV) for v in _ssd_case(H, G, N, Pv, 3, torch.float32, n, False))
     A = -torch.exp(A_log)
 
     def run(cuts):
