@@ -9,13 +9,15 @@
 //   gain    D  = W x,  W_nj = exp(c_last - c_j) dt_j B_jn  [states x 64]    W as two bfloat16 terms in TMEM
 //   y_i = exp(c_i) Yi_i + Yp_i + skip x_i,      S <- exp(c_last) S + D.
 // x, B and C are bfloat16 as they come; a float operand is handed over as the sum of two bfloat16 numbers (relative error
-// 2^-17; the state three: 2^-25), each with a product of its own, and all sums are float.  The state itself stays in
-// registers as floats, one row (64 columns) per thread.
+// 2^-17; the state three: 2^-25), each with a product of its own, and all sums are float.  The state itself stays in registers as floats, one row (64
+// columns) per thread.
 //   warp 0        TMA: C, B, x of a chunk into one of two stages.
-//   warp 1        tcgen05.mma.
+//   warps 1, 3    tcgen05.mma: scores and own tokens; gain and carry.  Issuing a product costs its thread more than the tensor
+//                 core takes for one this narrow, so two threads issue.
 //   warp 2        steps, running sums (in double, so that a difference of two sums is exact where the sums are large) and the
 //                 factors made of them, a chunk ahead.
-//   warps 4..7    a token per thread: P from the scores, y from the two results.  For columns j outside a warp's own 32 x 32
+//   warps 4..7    a token per thread: P from the scores, y from the two results (to global memory by whole rows, through shared
+//                 memory, while the products of the next chunk run).  For columns j outside a warp's own 32 x 32
 //                 diagonal block exp(c_i - c_j) is the product of two factors, of the row and of the column, both at most 1
 //                 (c at the block's first row lies between the two), so only the diagonal block needs an exponential per element.
 //   warps 8..11   a state per thread: W from B and the factors, S from D.
@@ -45,7 +47,9 @@ struct Factors {                                           // what the decays of
 };
 
 template <int NS> constexpr int stage_bytes() { return (2 * (NS / 64) + 1) * TILE_BYTES; }      // C, B, x
-template <int NS> constexpr int smem_bytes() { return 2 * stage_bytes<NS>() + 3 * NS * 128 + 2 * (int)sizeof(Factors) + 256; }
+// y on its way out: over the chunk's C, or (64 states: C is too small, and there is room) in two places of its own
+template <int NS> constexpr int y_bytes() { return NS == 64 ? 2 * Q * PC * 4 : 0; }
+template <int NS> constexpr int smem_bytes() { return 2 * stage_bytes<NS>() + 3 * NS * 128 + y_bytes<NS>() + 2 * (int)sizeof(Factors) + 256; }
 
 // the leading bfloat16 parts of two floats, packed; the floats become what is left of them
 __device__ __forceinline__ uint32_t take2(float& a, float& b) {
@@ -82,9 +86,9 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
     }
     const int n_chunks = (hi - lo + Q - 1) / Q;
     unsigned char* Ss = smem + 2 * SB;                     // [3][NS rows][64 columns], swizzled like x
-    Factors* fac = (Factors*)(Ss + 3 * NS * 128);          // [2]
+    Factors* fac = (Factors*)(Ss + 3 * NS * 128 + y_bytes<NS>());      // [2]
     uint64_t* full = (uint64_t*)(fac + 2);                 // [2] a stage's tiles are there
-    uint64_t* freed = full + 2;                            // [2] ... and have been read: the products, 128 + 128 threads
+    uint64_t* freed = full + 2;                            // [2] ... and have been read: two issuers' products, 128 + 128 threads
     uint64_t* fac_full = freed + 2;                        // [2]
     uint64_t* fac_free = fac_full + 2;                     // [2]
     uint64_t* sc_full = fac_free + 2;
@@ -92,14 +96,16 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
     uint64_t* w_ready = p_ready + 1;
     uint64_t* d_full = w_ready + 1;
     uint64_t* s_ready = d_full + 1;                        // the state before chunk c, as three terms
-    uint64_t* y_full = s_ready + 1;
-    uint32_t* tmem_slot = (uint32_t*)(y_full + 1);
+    uint64_t* yi_full = s_ready + 1;
+    uint64_t* yp_full = yi_full + 1;
+    uint64_t* y_read = yp_full + 1;                        // both have been read
+    uint32_t* tmem_slot = (uint32_t*)(y_read + 1);
     volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
         for (int s = 0; s < 2; s++) {
             mbar_init(full + s, 1);
-            mbar_init(freed + s, 257);
+            mbar_init(freed + s, 258);
             mbar_init(fac_full + s, 32);
             mbar_init(fac_free + s, 256);
         }
@@ -108,7 +114,9 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
         mbar_init(w_ready, 128);
         mbar_init(d_full, 1);
         mbar_init(s_ready, 128);
-        mbar_init(y_full, 1);
+        mbar_init(yi_full, 1);
+        mbar_init(yp_full, 1);
+        mbar_init(y_read, 128);
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("prefetch.tensormap [%0];" :: "l"(&map_u) : "memory");
@@ -140,13 +148,10 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
     } else if (warp == 1) {
         if (lane == 0) {
             const uint32_t id_sc = umma_idesc(Q), id_v = umma_idesc(PC, 1);
-            bool ok = true;
-            for (int c = 0; c < n_chunks && ok; c++) {
+            for (int c = 0; c < n_chunks; c++) {
                 const int s = c & 1;
                 const uint32_t c_addr = smem_u32(smem + s * SB), b_addr = c_addr + BOXES * TILE_BYTES, x_addr = b_addr + BOXES * TILE_BYTES;
-                const uint32_t s_addr = smem_u32(Ss);
-                ok = mbar_wait(full + s, (c >> 1) & 1, abort_flag, status, lim, 32, c);
-                if (!ok) break;
+                if (!mbar_wait(full + s, (c >> 1) & 1, abort_flag, status, lim, 32, c)) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 // the scores overwrite the P of the chunk before, whose products were issued before these
                 #pragma unroll
@@ -154,8 +159,36 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
                     umma(tmem + COL_SC, umma_desc(c_addr + (j / 4) * TILE_BYTES + (j % 4) * 32), umma_desc(b_addr + (j / 4) * TILE_BYTES + (j % 4) * 32),
                          id_sc, j != 0);
                 umma_commit(sc_full);
-                ok = mbar_wait(w_ready, c & 1, abort_flag, status, lim, 33, c);
-                if (!ok) break;
+                if (!mbar_wait(p_ready, c & 1, abort_flag, status, lim, 34, c)) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                #pragma unroll
+                for (int j = 0; j < Q / 16; j++) {
+                    const uint64_t xd = umma_desc_mn(x_addr + j * 2048, TILE_BYTES);
+                    umma_ts(tmem + COL_YP, tmem + COL_PL + j * 8, xd, id_v, j != 0);
+                    umma_ts(tmem + COL_YP, tmem + COL_SC + j * 8, xd, id_v, 1);
+                }
+                umma_commit(yp_full);
+                if (c + 2 < n_chunks) umma_commit(freed + s);          // (nobody waits for the last two)
+            }
+        }
+    } else if (warp == 3) {
+        if (lane == 0) {
+            const uint32_t id_v = umma_idesc(PC, 1), s_addr = smem_u32(Ss);
+            for (int c = 0; c < n_chunks; c++) {
+                const int s = c & 1;
+                const uint32_t c_addr = smem_u32(smem + s * SB), x_addr = c_addr + 2 * BOXES * TILE_BYTES;
+                if (!mbar_wait(full + s, (c >> 1) & 1, abort_flag, status, lim, 32, c)) break;
+                // the state's terms, and the carry of the chunk before read from its accumulator
+                if (!mbar_wait(s_ready, c & 1, abort_flag, status, lim, 35, c) || !mbar_wait(y_read, (c & 1) ^ 1, abort_flag, status, lim, 45, c)) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                #pragma unroll
+                for (int e = 2; e >= 0; e--)
+                    #pragma unroll
+                    for (int j = 0; j < NS / 16; j++)
+                        umma(tmem + COL_YI, umma_desc(c_addr + (j / 4) * TILE_BYTES + (j % 4) * 32), umma_desc_mn(s_addr + e * NS * 128 + j * 2048, NS * 128),
+                             id_v, e != 2 || j != 0);
+                umma_commit(yi_full);
+                if (!mbar_wait(w_ready, c & 1, abort_flag, status, lim, 33, c)) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 #pragma unroll
                 for (int j = 0; j < Q / 16; j++) {
@@ -164,23 +197,7 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
                     umma_ts(tmem + COL_D, tmem + COL_WH + j * 8, xd, id_v, 1);
                 }
                 umma_commit(d_full);
-                ok = mbar_wait(p_ready, c & 1, abort_flag, status, lim, 34, c) && mbar_wait(s_ready, c & 1, abort_flag, status, lim, 35, c);
-                if (!ok) break;
-                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                #pragma unroll
-                for (int e = 2; e >= 0; e--)
-                    #pragma unroll
-                    for (int j = 0; j < NS / 16; j++)
-                        umma(tmem + COL_YI, umma_desc(c_addr + (j / 4) * TILE_BYTES + (j % 4) * 32), umma_desc_mn(s_addr + e * NS * 128 + j * 2048, NS * 128),
-                             id_v, e != 2 || j != 0);
-                #pragma unroll
-                for (int j = 0; j < Q / 16; j++) {
-                    const uint64_t xd = umma_desc_mn(x_addr + j * 2048, TILE_BYTES);
-                    umma_ts(tmem + COL_YP, tmem + COL_PL + j * 8, xd, id_v, j != 0);
-                    umma_ts(tmem + COL_YP, tmem + COL_SC + j * 8, xd, id_v, 1);
-                }
-                umma_commit(freed + s);
-                umma_commit(y_full);
+                if (c + 2 < n_chunks) umma_commit(freed + s);          // (nobody waits for the last two)
             }
         }
     } else if (warp == 2) {
@@ -245,9 +262,25 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
         const int quarter = warp & 3, i = quarter * 32 + lane;
         const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16);
         const float skip = Dv[h];
+        auto y_place = [&](int c) -> unsigned char* { return NS == 64 ? Ss + 3 * NS * 128 + (c & 1) * Q * PC * 4 : smem + (c & 1) * SB; };
+        // the warp's 32 rows of 64 floats to global memory, two rows a turn; then their chunk's stage may be filled again
+        auto store_rows = [&](int c) {
+            const int t0 = lo + c * Q + 32 * quarter, half = lane >> 4, piece = lane & 15;
+            const unsigned char* ybase = y_place(c) + 32 * quarter * 256;
+            #pragma unroll 8
+            for (int k = 0; k < 16; k++) {
+                const int r = 2 * k + half;
+                const float4 v = *reinterpret_cast<const float4*>(ybase + r * 256 + ((piece ^ (r & 7)) << 4));
+                if (t0 + r < hi) *reinterpret_cast<float4*>(out + (size_t)(t0 + r) * H * P + h * P + p0 + 4 * piece) = v;
+            }
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // the next tiles come here by TMA
+            mbar_arrive(freed + (c & 1));
+        };
+        bool ok = true;
         for (int c = 0; c < n_chunks; c++) {
             const int s = c & 1;
-            if (!mbar_wait(fac_full + s, (c >> 1) & 1, abort_flag, status, lim, 37, c) || !mbar_wait(sc_full, c & 1, abort_flag, status, lim, 38, c)) break;
+            ok = mbar_wait(fac_full + s, (c >> 1) & 1, abort_flag, status, lim, 37, c) && mbar_wait(sc_full, c & 1, abort_flag, status, lim, 38, c);
+            if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const Factors& F = fac[s];
             const float my_er = F.er[i], my_ei = F.ei[i];
@@ -271,10 +304,16 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
                         }
                     } else {
                         const float ch = F.ch[i], cl = F.cl[i];
+                        const float4* ch4 = reinterpret_cast<const float4*>(F.ch + 32 * k);
+                        const float4* cl4 = reinterpret_cast<const float4*>(F.cl + 32 * k);
+                        const float4* dt4 = reinterpret_cast<const float4*>(F.dt + 32 * k);
                         #pragma unroll
-                        for (int e = 0; e < 32; e++) {
-                            const int j = 32 * k + e;
-                            v[e] = e <= lane ? v[e] * (ik_ex2((ch - F.ch[j]) + (cl - F.cl[j])) * F.dt[j]) : 0.f;
+                        for (int e = 0; e < 8; e++) {
+                            const float4 a = ch4[e], q = cl4[e], d = dt4[e];
+                            const float aa[4] = {a.x, a.y, a.z, a.w}, qq[4] = {q.x, q.y, q.z, q.w}, dd[4] = {d.x, d.y, d.z, d.w};
+                            #pragma unroll
+                            for (int r = 0; r < 4; r++)
+                                v[4 * e + r] = 4 * e + r <= lane ? v[4 * e + r] * (ik_ex2((ch - aa[r]) + (cl - qq[r])) * dd[r]) : 0.f;
                         }
                     }
                     #pragma unroll
@@ -289,12 +328,15 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
             tmem_st_wait();
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             mbar_arrive(fac_free + s);
-            mbar_arrive(p_ready);                          // (after y_full of the chunk before: this thread has read its y)
-            if (!mbar_wait(y_full, c & 1, abort_flag, status, lim, 39, c) || !mbar_wait(full + s, (c >> 1) & 1, abort_flag, status, lim, 40, c)) break;
+            mbar_arrive(p_ready);                          // (this thread has read the y of the chunk before)
+            if (c > 0) store_rows(c - 1);
+            ok = mbar_wait(yi_full, c & 1, abort_flag, status, lim, 39, c) && mbar_wait(yp_full, c & 1, abort_flag, status, lim, 39, c) &&
+                 mbar_wait(full + s, (c >> 1) & 1, abort_flag, status, lim, 40, c);
+            if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const int t = lo + c * Q + i;
             const unsigned char* xrow = smem + s * SB + 2 * BOXES * TILE_BYTES + i * 128;
-            float* orow = out + (size_t)t * H * P + h * P + p0;
+            // 16-byte pieces swizzled within eight rows; both products that read C are done
+            unsigned char* yrow = y_place(c) + i * 256;
             #pragma unroll
             for (int k = 0; k < 4; k++) {                  // 16 columns a turn
                 float yi[16], yp[16];
@@ -311,12 +353,17 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
                         yp[a] = fmaf(my_ei, yi[a], fmaf(skip, __uint_as_float(xw[q] << 16), yp[a]));
                         yp[a + 1] = fmaf(my_ei, yi[a + 1], fmaf(skip, __uint_as_float(xw[q] & 0xffff0000u), yp[a + 1]));
                     }
-                    if (t < hi) store8(orow + 16 * k + 8 * e, yp + 8 * e);
+                    #pragma unroll
+                    for (int q = 0; q < 2; q++)
+                        *reinterpret_cast<float4*>(yrow + (((4 * k + 2 * e + q) ^ (i & 7)) << 4)) =
+                            make_float4(yp[8 * e + 4 * q], yp[8 * e + 4 * q + 1], yp[8 * e + 4 * q + 2], yp[8 * e + 4 * q + 3]);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-            mbar_arrive(freed + s);
+            mbar_arrive(y_read);
+            __syncwarp();
         }
+        if (ok) store_rows(n_chunks - 1);
     } else if (warp >= 8) {
         const int quarter = warp & 3, n = quarter * 32 + lane;
         const bool live = n < NS;
@@ -403,7 +450,7 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
             mbar_arrive(fac_free + s);
             mbar_arrive(w_ready);                          // (after d_full of the chunk before: this thread has read its D)
             // D, and the carry's product, which still reads the terms of the state before
-            ok = mbar_wait(d_full, c & 1, abort_flag, status, lim, 43, c) && mbar_wait(y_full, c & 1, abort_flag, status, lim, 44, c);
+            ok = mbar_wait(d_full, c & 1, abort_flag, status, lim, 43, c) && mbar_wait(yi_full, c & 1, abort_flag, status, lim, 44, c);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             if (quarter * 32 < NS) {
@@ -449,7 +496,8 @@ int launch(const CUtensorMap& map, const float* p, int ldp, int dt_off, const fl
 
 }  // namespace
 
-// Sites of this module's waits: 31 loader for a free stage; 32 issuer for a stage, 33 W, 34 P, 35 the state's terms; 36 factors
+// Sites of this module's waits: 31 loader for a free stage; 32 issuers for a stage, 33 W, 34 P, 35 the state's terms, 45 the
+// carry's accumulator; 36 factors
 // for a free place; 37..40 token threads for factors, scores, results, the stage; 41..44 state threads for factors, the stage,
 // D, results.
 IK_EXPORT int ik_ssd_take_wait_record(int* out4) { return ik_take_wait_record(out4); }
