@@ -16,11 +16,12 @@
 //                 core takes for one this narrow, so two threads issue.
 //   warp 2        steps, running sums (in double, so that a difference of two sums is exact where the sums are large) and the
 //                 factors made of them, a chunk ahead.
-//   warps 4..7    a token per thread: P from the scores, y from the two results (to global memory by whole rows, through shared
-//                 memory, while the products of the next chunk run).  For columns j outside a warp's own 32 x 32
+//   warps 4..7    a token per thread: P from the scores, y from the two results (to global memory by pieces of rows, through
+//                 shared memory).  For columns j outside a warp's own 32 x 32
 //                 diagonal block exp(c_i - c_j) is the product of two factors, of the row and of the column, both at most 1
 //                 (c at the block's first row lies between the two), so only the diagonal block needs an exponential per element.
-//   warps 8..11   a state per thread: W from B and the factors, S from D.
+//   warps 8..11   a state per thread: S from D, and S as three terms.
+//   warps 12..15  a state per thread: W from B and the factors.
 // Every mbarrier here completes one phase per chunk (per use of a stage), and no phase can complete before every waiter has
 // seen the one before it: see the notes at the arrivals.  All waits are bounded (tc_common.cuh); on a timeout the status word
 // is set, the block leaves its loops and frees its TMEM.
@@ -47,17 +48,30 @@ struct Factors {                                           // what the decays of
 };
 
 template <int NS> constexpr int stage_bytes() { return (2 * (NS / 64) + 1) * TILE_BYTES; }      // C, B, x
-// y on its way out: over the chunk's C, or (64 states: C is too small, and there is room) in two places of its own
-template <int NS> constexpr int y_bytes() { return NS == 64 ? 2 * Q * PC * 4 : 0; }
-template <int NS> constexpr int smem_bytes() { return 2 * stage_bytes<NS>() + 3 * NS * 128 + y_bytes<NS>() + 2 * (int)sizeof(Factors) + 256; }
+constexpr int Y_BYTES = Q * 16 * 4;                         // y on its way out, 16 columns at a time
+template <int NS> constexpr int smem_bytes() { return 2 * stage_bytes<NS>() + 3 * NS * 128 + Y_BYTES + 2 * (int)sizeof(Factors) + 256; }
 
 // the leading bfloat16 parts of two floats, packed; the floats become what is left of them
 __device__ __forceinline__ uint32_t take2(float& a, float& b) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
     const uint32_t w = *reinterpret_cast<const uint32_t*>(&v);
-    a -= __uint_as_float(w << 16);
-    b -= __uint_as_float(w & 0xffff0000u);
+    asm("{\n\t.reg .b64 x, y, m;\n\t"
+        "mov.b64 x, {%0, %1};\n\t"
+        "mov.b64 y, {%2, %3};\n\t"
+        "mov.b64 m, {%4, %4};\n\t"
+        "fma.rn.f32x2 x, y, m, x;\n\t"
+        "mov.b64 {%0, %1}, x;\n\t}"
+        : "+f"(a), "+f"(b) : "f"(__uint_as_float(w << 16)), "f"(__uint_as_float(w & 0xffff0000u)), "f"(-1.0f));
     return w;
+}
+// (a, b) *= (c, d)
+__device__ __forceinline__ void mul2(float& a, float& b, float c, float d) {
+    asm("{\n\t.reg .b64 x, y;\n\t"
+        "mov.b64 x, {%0, %1};\n\t"
+        "mov.b64 y, {%2, %3};\n\t"
+        "mul.rn.f32x2 x, x, y;\n\t"
+        "mov.b64 {%0, %1}, x;\n\t}"
+        : "+f"(a), "+f"(b) : "f"(c), "f"(d));
 }
 __device__ __forceinline__ void store8(float* p, const float* v) {
     reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
@@ -65,7 +79,7 @@ __device__ __forceinline__ void store8(float* p, const float* v) {
 }
 
 template <int NS>
-__global__ void __launch_bounds__(384, 1)
+__global__ void __launch_bounds__(512, 1)
 ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict__ p, int ldp, int dt_off, const float* __restrict__ dt_bias,
               const float* __restrict__ A, const float* __restrict__ Dv, float* __restrict__ state, const int* __restrict__ slots,
               const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens, float* __restrict__ out, int H, int G, int P, int* status) {
@@ -86,7 +100,8 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
     }
     const int n_chunks = (hi - lo + Q - 1) / Q;
     unsigned char* Ss = smem + 2 * SB;                     // [3][NS rows][64 columns], swizzled like x
-    Factors* fac = (Factors*)(Ss + 3 * NS * 128 + y_bytes<NS>());      // [2]
+    unsigned char* Ys = Ss + 3 * NS * 128;
+    Factors* fac = (Factors*)(Ys + Y_BYTES);               // [2]
     uint64_t* full = (uint64_t*)(fac + 2);                 // [2] a stage's tiles are there
     uint64_t* freed = full + 2;                            // [2] ... and have been read: two issuers' products, 128 + 128 threads
     uint64_t* fac_full = freed + 2;                        // [2]
@@ -99,7 +114,8 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
     uint64_t* yi_full = s_ready + 1;
     uint64_t* yp_full = yi_full + 1;
     uint64_t* y_read = yp_full + 1;                        // both have been read
-    uint32_t* tmem_slot = (uint32_t*)(y_read + 1);
+    uint64_t* d_read = y_read + 1;
+    uint32_t* tmem_slot = (uint32_t*)(d_read + 1);
     volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
@@ -107,7 +123,7 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
             mbar_init(full + s, 1);
             mbar_init(freed + s, 258);
             mbar_init(fac_full + s, 32);
-            mbar_init(fac_free + s, 256);
+            mbar_init(fac_free + s, 384);
         }
         mbar_init(sc_full, 1);
         mbar_init(p_ready, 128);
@@ -117,6 +133,7 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
         mbar_init(yi_full, 1);
         mbar_init(yp_full, 1);
         mbar_init(y_read, 128);
+        mbar_init(d_read, 128);
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("prefetch.tensormap [%0];" :: "l"(&map_u) : "memory");
@@ -188,7 +205,7 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
                         umma(tmem + COL_YI, umma_desc(c_addr + (j / 4) * TILE_BYTES + (j % 4) * 32), umma_desc_mn(s_addr + e * NS * 128 + j * 2048, NS * 128),
                              id_v, e != 2 || j != 0);
                 umma_commit(yi_full);
-                if (!mbar_wait(w_ready, c & 1, abort_flag, status, lim, 33, c)) break;
+                if (!mbar_wait(w_ready, c & 1, abort_flag, status, lim, 33, c) || !mbar_wait(d_read, (c & 1) ^ 1, abort_flag, status, lim, 48, c)) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 #pragma unroll
                 for (int j = 0; j < Q / 16; j++) {
@@ -262,20 +279,7 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
         const int quarter = warp & 3, i = quarter * 32 + lane;
         const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16);
         const float skip = Dv[h];
-        auto y_place = [&](int c) -> unsigned char* { return NS == 64 ? Ss + 3 * NS * 128 + (c & 1) * Q * PC * 4 : smem + (c & 1) * SB; };
-        // the warp's 32 rows of 64 floats to global memory, two rows a turn; then their chunk's stage may be filled again
-        auto store_rows = [&](int c) {
-            const int t0 = lo + c * Q + 32 * quarter, half = lane >> 4, piece = lane & 15;
-            const unsigned char* ybase = y_place(c) + 32 * quarter * 256;
-            #pragma unroll 8
-            for (int k = 0; k < 16; k++) {
-                const int r = 2 * k + half;
-                const float4 v = *reinterpret_cast<const float4*>(ybase + r * 256 + ((piece ^ (r & 7)) << 4));
-                if (t0 + r < hi) *reinterpret_cast<float4*>(out + (size_t)(t0 + r) * H * P + h * P + p0 + 4 * piece) = v;
-            }
-            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // the next tiles come here by TMA
-            mbar_arrive(freed + (c & 1));
-        };
+        unsigned char* ys = Ys + quarter * 2048;             // 32 rows of 16 floats, 16-byte pieces swizzled within eight rows
         bool ok = true;
         for (int c = 0; c < n_chunks; c++) {
             const int s = c & 1;
@@ -300,7 +304,10 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
                         #pragma unroll
                         for (int e = 0; e < 8; e++) {
                             const float4 q = f[e];
-                            v[4 * e] *= q.x * my_er; v[4 * e + 1] *= q.y * my_er; v[4 * e + 2] *= q.z * my_er; v[4 * e + 3] *= q.w * my_er;
+                            mul2(v[4 * e], v[4 * e + 1], q.x, q.y);
+                            mul2(v[4 * e + 2], v[4 * e + 3], q.z, q.w);
+                            mul2(v[4 * e], v[4 * e + 1], my_er, my_er);
+                            mul2(v[4 * e + 2], v[4 * e + 3], my_er, my_er);
                         }
                     } else {
                         const float ch = F.ch[i], cl = F.cl[i];
@@ -329,14 +336,12 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             mbar_arrive(fac_free + s);
             mbar_arrive(p_ready);                          // (this thread has read the y of the chunk before)
-            if (c > 0) store_rows(c - 1);
             ok = mbar_wait(yi_full, c & 1, abort_flag, status, lim, 39, c) && mbar_wait(yp_full, c & 1, abort_flag, status, lim, 39, c) &&
                  mbar_wait(full + s, (c >> 1) & 1, abort_flag, status, lim, 40, c);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const unsigned char* xrow = smem + s * SB + 2 * BOXES * TILE_BYTES + i * 128;
-            // 16-byte pieces swizzled within eight rows; both products that read C are done
-            unsigned char* yrow = y_place(c) + i * 256;
+            const int t0 = lo + c * Q + 32 * quarter;
             #pragma unroll
             for (int k = 0; k < 4; k++) {                  // 16 columns a turn
                 float yi[16], yp[16];
@@ -355,16 +360,25 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
                     }
                     #pragma unroll
                     for (int q = 0; q < 2; q++)
-                        *reinterpret_cast<float4*>(yrow + (((4 * k + 2 * e + q) ^ (i & 7)) << 4)) =
+                        *reinterpret_cast<float4*>(ys + lane * 64 + (((2 * e + q) ^ ((lane >> 1) & 3)) << 4)) =
                             make_float4(yp[8 * e + 4 * q], yp[8 * e + 4 * q + 1], yp[8 * e + 4 * q + 2], yp[8 * e + 4 * q + 3]);
                 }
+                if (k == 3) {                              // all of this chunk's results and x have been read
+                    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+                    mbar_arrive(y_read);
+                    mbar_arrive(freed + s);
+                }
+                __syncwarp();
+                #pragma unroll
+                for (int r8 = 0; r8 < 4; r8++) {           // eight rows of 64 bytes an instruction
+                    const int r = 8 * r8 + (lane >> 2), piece = lane & 3;
+                    const float4 v = *reinterpret_cast<const float4*>(ys + r * 64 + ((piece ^ ((r >> 1) & 3)) << 4));
+                    if (t0 + r < hi) *reinterpret_cast<float4*>(out + (size_t)(t0 + r) * H * P + h * P + p0 + 16 * k + 4 * piece) = v;
+                }
+                __syncwarp();
             }
-            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-            mbar_arrive(y_read);
-            __syncwarp();
         }
-        if (ok) store_rows(n_chunks - 1);
-    } else if (warp >= 8) {
+    } else if (warp >= 8 && warp < 12) {
         const int quarter = warp & 3, n = quarter * 32 + lane;
         const bool live = n < NS;
         const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16);
@@ -401,54 +415,13 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
             mbar_arrive(s_ready);
         };
         publish();
-        if (!live) {                                       // rows of W beyond the states: zeros for good
-            const uint32_t z[16] = {};
-            for (int k = 0; k < 4; k++) {
-                tmem_st16_bits(base + COL_WH + 16 * k, z);
-                tmem_st16_bits(base + COL_WL + 16 * k, z);
-            }
-            tmem_st_wait();
-        }
         bool ok = true;
         for (int c = 0; c < n_chunks; c++) {
             const int s = c & 1;
-            ok = mbar_wait(fac_full + s, (c >> 1) & 1, abort_flag, status, lim, 41, c) && mbar_wait(full + s, (c >> 1) & 1, abort_flag, status, lim, 42, c);
+            ok = mbar_wait(fac_full + s, (c >> 1) & 1, abort_flag, status, lim, 41, c);
             if (!ok) break;
-            const Factors& F = fac[s];
-            const float keep = F.keep;
-            if (quarter * 32 < NS) {
-                const unsigned char* bt = smem + s * SB + (BOXES + n / 64) * TILE_BYTES;      // 128 tokens x 64 states
-                const int piece = (n & 63) >> 3, in = (n & 7) * 2;
-                #pragma unroll 1
-                for (int k = 0; k < 4; k++) {              // 32 tokens a turn
-                    float v[32];
-                    const float4* w4 = reinterpret_cast<const float4*>(F.w + 32 * k);
-                    #pragma unroll
-                    for (int e = 0; e < 8; e++) {
-                        const float4 q = w4[e];
-                        const float wq[4] = {q.x, q.y, q.z, q.w};
-                        #pragma unroll
-                        for (int r = 0; r < 4; r++) {
-                            const int j = 32 * k + 4 * e + r;      // j & 7 is known: 32 k is a multiple of eight
-                            const unsigned short raw = *reinterpret_cast<const unsigned short*>(bt + j * 128 + ((piece ^ ((4 * e + r) & 7)) << 4) + in);
-                            v[4 * e + r] = __uint_as_float((uint32_t)raw << 16) * wq[r];
-                        }
-                    }
-                    uint32_t wh[16], wl[16];
-                    #pragma unroll
-                    for (int e = 0; e < 16; e++) {
-                        wh[e] = take2(v[2 * e], v[2 * e + 1]);
-                        wl[e] = take2(v[2 * e], v[2 * e + 1]);
-                    }
-                    tmem_st16_bits(base + COL_WH + 16 * k, wh);
-                    tmem_st16_bits(base + COL_WL + 16 * k, wl);
-                }
-                tmem_st_wait();
-            }
-            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-            mbar_arrive(freed + s);
+            const float keep = fac[s].keep;
             mbar_arrive(fac_free + s);
-            mbar_arrive(w_ready);                          // (after d_full of the chunk before: this thread has read its D)
             // D, and the carry's product, which still reads the terms of the state before
             ok = mbar_wait(d_full, c & 1, abort_flag, status, lim, 43, c) && mbar_wait(yi_full, c & 1, abort_flag, status, lim, 44, c);
             if (!ok) break;
@@ -465,11 +438,66 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            mbar_arrive(d_read);
             if (c + 1 < n_chunks) publish();
         }
         if (ok && live) {
             #pragma unroll
             for (int k = 0; k < PC / 8; k++) store8(st_out + 8 * k, S + 8 * k);
+        }
+    } else if (warp >= 12) {
+        const int quarter = warp & 3, n = quarter * 32 + lane;
+        const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16);
+        if (n >= NS) {                                     // rows of W beyond the states: zeros for good
+            const uint32_t z[16] = {};
+            for (int k = 0; k < 4; k++) {
+                tmem_st16_bits(base + COL_WH + 16 * k, z);
+                tmem_st16_bits(base + COL_WL + 16 * k, z);
+            }
+            tmem_st_wait();
+        }
+        for (int c = 0; c < n_chunks; c++) {
+            const int s = c & 1;
+            // (the gain's product of the chunk before has read its W)
+            if (!mbar_wait(fac_full + s, (c >> 1) & 1, abort_flag, status, lim, 46, c) || !mbar_wait(full + s, (c >> 1) & 1, abort_flag, status, lim, 42, c) ||
+                (c > 0 && !mbar_wait(d_full, (c - 1) & 1, abort_flag, status, lim, 47, c)))
+                break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const Factors& F = fac[s];
+            if (quarter * 32 < NS) {
+                const unsigned char* bt = smem + s * SB + (BOXES + n / 64) * TILE_BYTES;      // 128 tokens x 64 states
+                const int piece = (n & 63) >> 3, in = (n & 7) * 2;
+                #pragma unroll 1
+                for (int k = 0; k < 4; k++) {              // 32 tokens a turn
+                    float v[32];
+                    const float4* w4 = reinterpret_cast<const float4*>(F.w + 32 * k);
+                    #pragma unroll
+                    for (int e = 0; e < 8; e++) {
+                        const float4 q = w4[e];
+                        #pragma unroll
+                        for (int r = 0; r < 4; r++) {
+                            const int j = 32 * k + 4 * e + r;      // j & 7 is known: 32 k is a multiple of eight
+                            const unsigned short raw = *reinterpret_cast<const unsigned short*>(bt + j * 128 + ((piece ^ ((4 * e + r) & 7)) << 4) + in);
+                            v[4 * e + r] = __uint_as_float((uint32_t)raw << 16);
+                        }
+                        mul2(v[4 * e], v[4 * e + 1], q.x, q.y);
+                        mul2(v[4 * e + 2], v[4 * e + 3], q.z, q.w);
+                    }
+                    uint32_t wh[16], wl[16];
+                    #pragma unroll
+                    for (int e = 0; e < 16; e++) {
+                        wh[e] = take2(v[2 * e], v[2 * e + 1]);
+                        wl[e] = take2(v[2 * e], v[2 * e + 1]);
+                    }
+                    tmem_st16_bits(base + COL_WH + 16 * k, wh);
+                    tmem_st16_bits(base + COL_WL + 16 * k, wl);
+                }
+                tmem_st_wait();
+            }
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            mbar_arrive(freed + s);
+            mbar_arrive(fac_free + s);
+            mbar_arrive(w_ready);
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -489,7 +517,7 @@ int launch(const CUtensorMap& map, const float* p, int ldp, int dt_off, const fl
         IK_RETURN_IF_ERROR(cudaFuncSetAttribute(ssd_tc_kernel<NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
         raised = true;
     }
-    IK_RETURN_IF_ERROR(ik_launch(ssd_tc_kernel<NS>, dim3(H, B, P / PC), 384, smem, stream, map, p, ldp, dt_off, dt_bias, A, Dv, state, slots,
+    IK_RETURN_IF_ERROR(ik_launch(ssd_tc_kernel<NS>, dim3(H, B, P / PC), 512, smem, stream, map, p, ldp, dt_off, dt_bias, A, Dv, state, slots,
                                  cu_seqlens, kv_lens, out, H, G, P, status));
     IK_LAUNCH_STATUS();
 }
@@ -497,9 +525,9 @@ int launch(const CUtensorMap& map, const float* p, int ldp, int dt_off, const fl
 }  // namespace
 
 // Sites of this module's waits: 31 loader for a free stage; 32 issuers for a stage, 33 W, 34 P, 35 the state's terms, 45 the
-// carry's accumulator; 36 factors
-// for a free place; 37..40 token threads for factors, scores, results, the stage; 41..44 state threads for factors, the stage,
-// D, results.
+// carry's accumulator, 48 the gain's; 36 factors
+// for a free place; 37..40 token threads for factors, scores, results, the stage; 41, 43, 44 state threads for factors, the gain, the
+// carry; 42, 46, 47 W threads for the stage, factors, the gain before.
 IK_EXPORT int ik_ssd_take_wait_record(int* out4) { return ik_take_wait_record(out4); }
 
 // Arguments as ik_ssd's (ssd.cu); bfloat16 u, N 64 or 128, P a multiple of 64, 16-byte aligned rows.
