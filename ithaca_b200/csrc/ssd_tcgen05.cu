@@ -342,12 +342,19 @@ ssd_tc_kernel(const __grid_constant__ CUtensorMap map_u, const float* __restrict
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const unsigned char* xrow = smem + s * SB + 2 * BOXES * TILE_BYTES + i * 128;
             const int t0 = lo + c * Q + 32 * quarter;
+            float ahead[2][16];                            // the next turn's results are asked for a turn early
+            tmem_ld16_issue(base + COL_YI, ahead[0]);
+            tmem_ld16_issue(base + COL_YP, ahead[1]);
             #pragma unroll
             for (int k = 0; k < 4; k++) {                  // 16 columns a turn
                 float yi[16], yp[16];
-                tmem_ld16_issue(base + COL_YI + 16 * k, yi);
-                tmem_ld16_issue(base + COL_YP + 16 * k, yp);
                 tmem_ld_wait();
+                #pragma unroll
+                for (int e = 0; e < 16; e++) { yi[e] = ahead[0][e]; yp[e] = ahead[1][e]; }
+                if (k < 3) {
+                    tmem_ld16_issue(base + COL_YI + 16 * (k + 1), ahead[0]);
+                    tmem_ld16_issue(base + COL_YP + 16 * (k + 1), ahead[1]);
+                }
                 #pragma unroll
                 for (int e = 0; e < 2; e++) {
                     const uint4 xv = *reinterpret_cast<const uint4*>(xrow + (((2 * k + e) ^ (i & 7)) << 4));
