@@ -17,6 +17,11 @@
 #include "common.cuh"
 
 __device__ __forceinline__ float ik_silu(float x) { return x / (1.0f + expf(-x)); }
+// ... as a result of the given type: what is rounded to 16 bits anyway takes the hardware's approximate exponential and quotient
+// (relative error near 1e-6)
+template <typename TO> __device__ __forceinline__ float ik_silu_for(float x) {
+    return sizeof(TO) == 2 ? __fdividef(x, 1.0f + __expf(-x)) : ik_silu(x);
+}
 __device__ __forceinline__ float ik_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float ik_softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
@@ -53,7 +58,7 @@ causal_conv_kernel(const float* __restrict__ x, int ldx, const float* __restrict
         acc = fmaf(w[(size_t)j * C + c], u, acc);
     }
     if (inline_ring && ring) ring[((size_t)slots[b] * taps + pos % taps) * C + c] = x[(size_t)t * ldx + c];
-    ik_st(out, idx, act ? ik_silu(acc) : acc);
+    ik_st(out, idx, act ? ik_silu_for<TO>(acc) : acc);
 }
 
 // The same for four neighbouring channels per thread (channel counts and row distances that are multiples of four,
@@ -84,8 +89,62 @@ causal_conv4_kernel(const float* __restrict__ x, int ldx, const float* __restric
         acc.x = fmaf(wj.x, u.x, acc.x); acc.y = fmaf(wj.y, u.y, acc.y); acc.z = fmaf(wj.z, u.z, acc.z); acc.w = fmaf(wj.w, u.w, acc.w);
     }
     if (inline_ring && ring) ik_st4(ring, ((size_t)slots[b] * taps + pos % taps) * C + c, ik_ld4(x, (size_t)t * ldx + c));
-    if (act) { acc.x = ik_silu(acc.x); acc.y = ik_silu(acc.y); acc.z = ik_silu(acc.z); acc.w = ik_silu(acc.w); }
+    if (act) { acc.x = ik_silu_for<TO>(acc.x); acc.y = ik_silu_for<TO>(acc.y); acc.z = ik_silu_for<TO>(acc.z); acc.w = ik_silu_for<TO>(acc.w); }
     ik_st4(out, (size_t)t * C + c, acc);
+}
+
+// The same for prompts: a thread takes RUN neighbouring tokens of its four channels and keeps the inputs behind the current
+// one in registers, so an input is read once (and TAPS - 1 more at the run's start and where a sequence begins) instead of TAPS
+// times.  The sum of a token runs in the same order as above.
+template <typename TO, int TAPS, int RUN>
+__global__ void __launch_bounds__(256)
+causal_conv4_run_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                        const float* __restrict__ ring, const int* __restrict__ slots, const int* __restrict__ cu_seqlens,
+                        const int* __restrict__ token_seq, const int* __restrict__ token_pos, TO* __restrict__ out, int T, int C, int act) {
+    ik_pdl_wait();
+    IK_AFTER_WAIT(x);
+    IK_AFTER_WAIT(ring);
+    IK_AFTER_WAIT(slots);
+    IK_AFTER_WAIT(cu_seqlens);
+    IK_AFTER_WAIT(token_seq);
+    IK_AFTER_WAIT(token_pos);
+    ik_pdl_launch_dependents();
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4, t0 = blockIdx.x * RUN;
+    if (c >= C) return;
+    float4 now[RUN], wj[TAPS], past[TAPS - 1];
+    #pragma unroll
+    for (int r = 0; r < RUN; r++) now[r] = t0 + r < T ? ik_ld4(x, (size_t)(t0 + r) * ldx + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    #pragma unroll
+    for (int j = 0; j < TAPS; j++) wj[j] = ik_ld4(w, (size_t)j * C + c);
+    const float4 b4 = bias ? ik_ld4(bias, c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    int seq = -1;
+    #pragma unroll
+    for (int r = 0; r < RUN; r++) {
+        const int t = t0 + r;
+        if (t >= T) break;
+        const int b = token_seq[t];
+        if (r == 0 || b != seq) {                          // the inputs behind this token: of this step, older ones, or none
+            const int pos = token_pos[t], first = cu_seqlens[b];
+            seq = b;
+            #pragma unroll
+            for (int j = 0; j < TAPS - 1; j++) {
+                const int back = TAPS - 1 - j;
+                past[j] = back > pos ? make_float4(0.f, 0.f, 0.f, 0.f)
+                        : t - back >= first ? ik_ld4(x, (size_t)(t - back) * ldx + c)
+                                            : ik_ld4(ring, ((size_t)slots[b] * TAPS + (pos - back) % TAPS) * C + c);
+            }
+        }
+        float4 acc = b4;
+        #pragma unroll
+        for (int j = 0; j < TAPS; j++) {
+            const float4 u = j < TAPS - 1 ? past[j] : now[r];
+            acc.x = fmaf(wj[j].x, u.x, acc.x); acc.y = fmaf(wj[j].y, u.y, acc.y); acc.z = fmaf(wj[j].z, u.z, acc.z); acc.w = fmaf(wj[j].w, u.w, acc.w);
+        }
+        #pragma unroll
+        for (int j = 0; j < TAPS - 1; j++) past[j] = j < TAPS - 2 ? past[j + 1] : now[r];
+        if (act) { acc.x = ik_silu_for<TO>(acc.x); acc.y = ik_silu_for<TO>(acc.y); acc.z = ik_silu_for<TO>(acc.z); acc.w = ik_silu_for<TO>(acc.w); }
+        ik_st4(out, (size_t)t * C + c, acc);
+    }
 }
 
 // The last `taps` inputs of every sequence go into its ring.
@@ -122,6 +181,15 @@ IK_EXPORT int ik_causal_conv(const float* x, int ldx, const float* w, const floa
     if (by4 && (out_dtype == IK_F32 || out_dtype == IK_BF16)) {
         const int threads = C / 4 >= 256 ? 256 : ((C / 4 + 31) / 32) * 32;
         const dim3 grid(T, (C / 4 + threads - 1) / threads);
+        constexpr int RUN = 8;
+        const bool runs = !inl && taps >= 2 && taps <= 4 && (long long)T * grid.y >= 8LL * RUN * ik_sm_count();   // enough blocks either way
+#define IK_CONV_RUN(TO, TAPS)                                                                                                       \
+    IK_RETURN_IF_ERROR(ik_launch(causal_conv4_run_kernel<TO, TAPS, RUN>, dim3((T + RUN - 1) / RUN, grid.y), threads, 0, stream, x, ldx, w, bias, \
+                                 (const float*)ring, slots, cu_seqlens, token_seq, token_pos, (TO*)out, T, C, act))
+        if (runs && out_dtype == IK_F32) { if (taps == 2) IK_CONV_RUN(float, 2); else if (taps == 3) IK_CONV_RUN(float, 3); else IK_CONV_RUN(float, 4); }
+        else if (runs) { if (taps == 2) IK_CONV_RUN(__nv_bfloat16, 2); else if (taps == 3) IK_CONV_RUN(__nv_bfloat16, 3); else IK_CONV_RUN(__nv_bfloat16, 4); }
+        else
+#undef IK_CONV_RUN
         if (out_dtype == IK_F32)
             IK_RETURN_IF_ERROR(ik_launch(causal_conv4_kernel<float>, grid, threads, 0, stream, x, ldx, w, bias, ring, slots, cu_seqlens,
                                          token_seq, token_pos, (float*)out, T, C, taps, act, inl));

@@ -496,6 +496,9 @@ ssd_decode_kernel(const float* __restrict__ p, int ldp, int x_off, const float* 
 // out[t, i] = g_i / sqrt(mean over its part(g^2) + eps) * w[i] with g = x * silu(z), parts of d neighbouring values.  THREADS
 // threads per part (32: a warp each, eight parts a block).  The part's g stays in registers (four values times KEEP a thread)
 // where it fits.
+template <typename TO> __device__ __forceinline__ float gate(float z) {       // silu; for 16-bit results with the hardware's exponential
+    return sizeof(TO) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : ik_siluf(z);
+}
 template <typename TO, int THREADS, bool VEC>
 __global__ void __launch_bounds__(256)
 gated_group_norm_kernel(const float* __restrict__ x, const float* __restrict__ z, int ldz, const float* __restrict__ w,
@@ -530,13 +533,13 @@ gated_group_norm_kernel(const float* __restrict__ x, const float* __restrict__ z
             const int i = tid + k * THREADS;
             if (i < n4) {
                 const float4 v = ik_ld4(a, 4 * (size_t)i), q = ik_ld4(zz, 4 * (size_t)i);
-                g[k] = make_float4(v.x * ik_siluf(q.x), v.y * ik_siluf(q.y), v.z * ik_siluf(q.z), v.w * ik_siluf(q.w));
+                g[k] = make_float4(v.x * gate<TO>(q.x), v.y * gate<TO>(q.y), v.z * gate<TO>(q.z), v.w * gate<TO>(q.w));
                 ss = fmaf(g[k].x, g[k].x, fmaf(g[k].y, g[k].y, fmaf(g[k].z, g[k].z, fmaf(g[k].w, g[k].w, ss))));
             }
         }
         for (int i = tid + KEEP * THREADS; i < n4; i += THREADS) {
             const float4 v = ik_ld4(a, 4 * (size_t)i), q = ik_ld4(zz, 4 * (size_t)i);
-            const float4 e = make_float4(v.x * ik_siluf(q.x), v.y * ik_siluf(q.y), v.z * ik_siluf(q.z), v.w * ik_siluf(q.w));
+            const float4 e = make_float4(v.x * gate<TO>(q.x), v.y * gate<TO>(q.y), v.z * gate<TO>(q.z), v.w * gate<TO>(q.w));
             ss = fmaf(e.x, e.x, fmaf(e.y, e.y, fmaf(e.z, e.z, fmaf(e.w, e.w, ss))));
         }
         const float s = 1.0f / sqrtf(total(ss) / (float)d + eps);
@@ -550,13 +553,13 @@ gated_group_norm_kernel(const float* __restrict__ x, const float* __restrict__ z
         }
         for (int i = tid + KEEP * THREADS; i < n4; i += THREADS) {
             const float4 v = ik_ld4(a, 4 * (size_t)i), q = ik_ld4(zz, 4 * (size_t)i), c = ik_ld4(ww, 4 * (size_t)i);
-            ik_st4(out, (size_t)part * d + 4 * (size_t)i, make_float4(v.x * ik_siluf(q.x) * s * c.x, v.y * ik_siluf(q.y) * s * c.y,
-                                                                      v.z * ik_siluf(q.z) * s * c.z, v.w * ik_siluf(q.w) * s * c.w));
+            ik_st4(out, (size_t)part * d + 4 * (size_t)i, make_float4(v.x * gate<TO>(q.x) * s * c.x, v.y * gate<TO>(q.y) * s * c.y,
+                                                                      v.z * gate<TO>(q.z) * s * c.z, v.w * gate<TO>(q.w) * s * c.w));
         }
     } else {
-        for (int i = tid; i < d; i += THREADS) { const float v = a[i] * ik_siluf(zz[i]); ss = fmaf(v, v, ss); }
+        for (int i = tid; i < d; i += THREADS) { const float v = a[i] * gate<TO>(zz[i]); ss = fmaf(v, v, ss); }
         const float s = 1.0f / sqrtf(total(ss) / (float)d + eps);
-        for (int i = tid; i < d; i += THREADS) ik_st(out, (size_t)part * d + i, a[i] * ik_siluf(zz[i]) * s * ww[i]);
+        for (int i = tid; i < d; i += THREADS) ik_st(out, (size_t)part * d + i, a[i] * gate<TO>(zz[i]) * s * ww[i]);
     }
 }
 

@@ -310,6 +310,35 @@ def test_decode_kernel_with_its_convolution(H, G, N, Pv, taps):
         assert rel_err(state[slots[b], (n - 1) & 1].cpu().numpy(), want[b][1].numpy()) < 1e-5
 
 
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("taps,C", [(2, 2048), (3, 1028), (4, 3072), (5, 1024)])
+def test_short_convolution_of_long_prompts(dtype, taps, C):
+    """Prompts long enough for the kernel that takes several tokens a thread: sequences that begin inside a run of tokens, one
+    that goes on from its ring; the same bits as short steps give."""
+    from ithaca_b200.csrc import ops
+    g = torch.Generator().manual_seed(taps)
+    lens, slots = [3001, 2, 6100, 1], [2, 0, 3, 1]
+    x = [torch.randn(n + 5, C, generator=g) for n in lens]
+    w, cb = torch.randn(C, taps, generator=g) * 0.5, torch.randn(C, generator=g)
+    ring = torch.randn(4, taps, C, generator=g).to(DEV)
+    wd, bd = w.t().contiguous().to(DEV), cb.to(DEV)
+    out = [[] for _ in lens]
+    for lo, hi in (([0] * 4, [5, 1, 2, 1]), ([5, 1, 2, 1], [n + 1 if n > 1 else 2 for n in lens])):
+        ctx = _ctx(lo, hi, slots)
+        y = ops.causal_conv(torch.cat([x[b][lo[b]:hi[b]] for b in range(4)]).to(DEV), wd, bd, ring, ctx, dtype)
+        for b, part in enumerate(y.split([h - l for l, h in zip(lo, hi)])):
+            out[b].append(part)
+    ring2 = torch.zeros_like(ring)
+    for b, n in enumerate(lens):
+        end = n + 1 if n > 1 else 2
+        got = torch.cat(out[b])
+        want = P.silu(P.causal_conv(x[b][:end].double(), w, cb))
+        assert rel_err(got.float().cpu().numpy(), want.numpy()) < (2e-6 if dtype == torch.float32 else 5e-3), b
+        cuts = list(range(0, end, 700)) + [end]
+        again = torch.cat([ops.causal_conv(x[b][a:e].to(DEV), wd, bd, ring2, _ctx([a], [e], [0]), dtype) for a, e in zip(cuts, cuts[1:])])
+        assert torch.equal(got, again), b
+
+
 def test_decode_kernel_declines_odd_value_sizes():
     from ithaca_b200.csrc import ops
     z = lambda *s: torch.zeros(*s, device=DEV)
@@ -470,7 +499,7 @@ def test_combine_adds_one_more_result_and_the_stream():
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("d,ff,E,top,shared,T", [(64, 24, 5, 2, 40, 9), (48, 40, 1, 1, None, 3), (128, 96, 16, 4, 64, 300), (72, 16, 3, 3, 200, 1),
-                                                 (256, 64, 12, 3, 72, 1500), (30, 7, 4, 2, 21, 20)])
+                                                 (256, 64, 12, 3, 72, 1500), (30, 7, 4, 2, 21, 20), (64, 32, 9, 2, None, 600)])
 def test_routed_feed_forward_with_a_shared_expert(dtype, d, ff, E, top, shared, T):
     from ithaca_b200.config import config_from_dict
     from ithaca_b200.parts import FEED_FORWARDS, Runtime
