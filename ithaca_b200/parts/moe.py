@@ -16,8 +16,8 @@ scaled rows are formed (in float, rounded once to the operands' type) while the 
 uses; with the tensor ``shared_weight`` [1, hidden] its result is multiplied by the sigmoid of one number per token, a
 projection that the router's kernel forms as one row more.
 
-On the device: one kernel forms the router's logits and picks experts and weights per token (for long prompts on the 16-bit
-path: a tensor-core product and the picking); a counting sort groups the
+On the device: one kernel forms the router's logits and picks experts and weights per token (on the 16-bit path, where the router
+is stored in 16 bits: a tensor-core product, whose products of 16-bit numbers are exact, and the picking); a counting sort groups the
 (token, choice) pairs by expert; two grouped products run every expert over its rows (the first
 with silu(g) * u as its epilogue, so the [rows, 2 ff] intermediate is never written); a last kernel
 adds a token's choices in the order they were chosen, then the shared expert's result, straight into the stream.  Nothing is read back by the host: grids are
@@ -42,9 +42,6 @@ from ..weights.loader import TensorReq
 from .base import Runtime, as_float32, register_feed_forward, to_device
 from .feed_forward import GatedMLP
 from .linear import gemm
-
-
-PRODUCT_TOKENS = 512          # from here on the router's logits are a product of their own
 
 
 class MoEFeedForward:
@@ -122,8 +119,8 @@ class MoEFeedForward:
         self.shared_weighted = bool(self.shared) and "shared_weight" in w
         if self.shared_weighted:
             self.router = torch.cat([self.router, as_float32(tensors[w["shared_weight"]], runtime)], dim=0).contiguous()
-        # long prompts on the 16-bit path: a router that is bfloat16 as stored forms its logits on the tensor cores (16-bit operands
-        # as they are, exact products, float sums)
+        # 16-bit path: a router that is bfloat16 as stored forms its logits on the tensor cores (16-bit operands as they are, exact
+        # products, float sums)
         self.router16 = self.router.to(torch.bfloat16) if runtime.dtype == "bfloat16" and self.hidden % 8 == 0 else None
         if self.router16 is not None and not torch.equal(self.router16.to(torch.float32), self.router):
             self.router16 = None
@@ -154,7 +151,7 @@ class MoEFeedForward:
         sg = torch.empty((x.shape[0],), dtype=torch.float32, device=x.device) if self.shared_weighted else None
         extras = {"bias": self.router_bias, "gate": sg}
         routed = logits = None
-        if self.router16 is not None and x.shape[0] >= PRODUCT_TOKENS:
+        if self.router16 is not None:
             logits = gemm(x, self.router16, out_dtype=torch.float32)
         else:
             routed = ops.moe_router(x, self.router, self.top, self.n_groups, self.group_keep, self.renormalize, self.score, **extras)
