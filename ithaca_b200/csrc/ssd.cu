@@ -409,13 +409,14 @@ ssd_chunk_kernel(const bf16* __restrict__ u, int ldu, const float* __restrict__ 
 // projections themselves: x from x_off, then B and C as in `u`, then the raw steps) and the ring of earlier inputs, and then
 // the state is advanced, read out and written to the other parity's copy.  Every block convolves its group's B and C for
 // itself; the blocks of the group's first head put the new inputs into the ring (at a place that no block reads in this step).
-constexpr int DEC_ROWS = 16;                               // state rows a thread has in flight
+constexpr int DEC_ROWS = 8, DEC_THREADS = 256;              // state rows a thread has in flight
 
-__global__ void __launch_bounds__(128)
+template <int TAPS>                                        // 0: any number, given by `taps_given`
+__global__ void __launch_bounds__(DEC_THREADS)
 ssd_decode_kernel(const float* __restrict__ p, int ldp, int x_off, const float* __restrict__ cw, const float* __restrict__ cb,
                   float* __restrict__ ring, const float* __restrict__ dt_bias, const float* __restrict__ A, const float* __restrict__ Dv,
                   float* __restrict__ state, const int* __restrict__ slots, const int* __restrict__ cu_seqlens,
-                  const int* __restrict__ kv_lens, float* __restrict__ out, int H, int G, int N, int P, int taps, int pv_n) {
+                  const int* __restrict__ kv_lens, float* __restrict__ out, int H, int G, int N, int P, int taps_given, int pv_n) {
     extern __shared__ __align__(16) float sm[];            // x [4 pv_n], B [N], C [N], sums [slices][4 pv_n]
     ik_pdl_wait();
     IK_AFTER_WAIT(p);
@@ -424,7 +425,8 @@ ssd_decode_kernel(const float* __restrict__ p, int ldp, int x_off, const float* 
     IK_AFTER_WAIT(kv_lens);
     ik_pdl_launch_dependents();
     const int h = blockIdx.x, b = blockIdx.y, PT = 4 * pv_n, p0 = blockIdx.z * PT;
-    const int pv = threadIdx.x % pv_n, slice = threadIdx.x / pv_n, slices = 128 / pv_n;
+    const int pv = threadIdx.x % pv_n, slice = threadIdx.x / pv_n, slices = DEC_THREADS / pv_n;
+    const int taps = TAPS ? TAPS : taps_given;
     const int tok = cu_seqlens[b], slot = slots[b], end = kv_lens[b], pos = end - 1;
     const int grp = h / (H / G), C_all = H * P + 2 * G * N;
     const size_t per = (size_t)H * N * P;
@@ -444,22 +446,46 @@ ssd_decode_kernel(const float* __restrict__ p, int ldp, int x_off, const float* 
     const float* row = p + (size_t)tok * ldp + x_off;      // the convolution's inputs, then the raw steps
     float* rg = ring ? ring + (size_t)slot * taps * C_all : nullptr;
     const bool own_bc = h % (H / G) == 0 && blockIdx.z == 0;
-    for (int e = threadIdx.x; e < PT + 2 * N; e += 128) {
-        int c;
-        bool mine = true;
-        if (e < PT) { c = h * P + p0 + e; if (p0 + e >= P) { sm[e] = 0.f; continue; } }
-        else { const int w = e - PT; c = H * P + (w < N ? grp * N + w : G * N + grp * N + w - N); mine = own_bc; }
-        const float now = row[c];
-        float acc = fmaf(cw[(size_t)(taps - 1) * C_all + c], now, cb[c]);
-        for (int j = 0; j < taps - 1; j++) {
-            const int back = taps - 1 - j;
-            if (back <= pos) acc = fmaf(cw[(size_t)j * C_all + c], rg[(size_t)((pos - back) % taps) * C_all + c], acc);
+    // channel of the block's e-th convolved value, -1 beyond the head's columns
+    auto channel = [&](int e) -> int {
+        if (e < PT) return p0 + e < P ? h * P + p0 + e : -1;
+        const int w = e - PT;
+        return H * P + (w < N ? grp * N + w : G * N + grp * N + w - N);
+    };
+    const int at = pos % taps;                             // position p of a sequence lies in place p mod taps of its ring
+    #pragma unroll 2
+    for (int e = threadIdx.x; e < PT + 2 * N; e += DEC_THREADS) {
+        const int c = channel(e);
+        float acc = 0.f;
+        if (c >= 0) {
+            const float now = row[c];
+            acc = fmaf(cw[(size_t)(taps - 1) * C_all + c], now, cb[c]);
+            if (TAPS) {
+                float w[TAPS ? TAPS : 1], u[TAPS ? TAPS : 1];
+                #pragma unroll
+                for (int j = 0; j < TAPS - 1; j++) {       // all loads first
+                    const int back = TAPS - 1 - j, place = at >= back ? at - back : at - back + TAPS;
+                    w[j] = cw[(size_t)j * C_all + c];
+                    u[j] = back <= pos ? rg[(size_t)place * C_all + c] : 0.f;
+                }
+                #pragma unroll
+                for (int j = 0; j < TAPS - 1; j++) acc = fmaf(w[j], u[j], acc);
+            } else {
+                for (int j = 0; j < taps - 1; j++) {
+                    const int back = taps - 1 - j, place = at >= back ? at - back : at - back + taps;
+                    if (back <= pos) acc = fmaf(cw[(size_t)j * C_all + c], rg[(size_t)place * C_all + c], acc);
+                }
+            }
         }
-        if (rg && mine) rg[(size_t)(pos % taps) * C_all + c] = now;
-        sm[e] = ik_siluf(acc);
+        sm[e] = __fdividef(acc, 1.0f + __expf(-acc));
     }
     const float dt = ik_softplusf(row[C_all + h] + dt_bias[h]), a = expf(A[h] * dt);
     __syncthreads();
+    if (rg)                                                // the new inputs, behind every read of the ring in this block
+        for (int e = threadIdx.x; e < (own_bc ? PT + 2 * N : PT); e += DEC_THREADS) {
+            const int c = channel(e);
+            if (c >= 0) rg[(size_t)at * C_all + c] = row[c];
+        }
     const float4 x = *reinterpret_cast<const float4*>(sm + 4 * pv);
     const float4 xd = make_float4(dt * x.x, dt * x.y, dt * x.z, dt * x.w);
     const float* Bn = sm + PT;
@@ -484,7 +510,7 @@ ssd_decode_kernel(const float* __restrict__ p, int ldp, int x_off, const float* 
     sums[slice * PT + 4 * pv] = y.x; sums[slice * PT + 4 * pv + 1] = y.y;
     sums[slice * PT + 4 * pv + 2] = y.z; sums[slice * PT + 4 * pv + 3] = y.w;
     __syncthreads();
-    for (int e = threadIdx.x; e < PT; e += 128) {
+    for (int e = threadIdx.x; e < PT; e += DEC_THREADS) {
         if (p0 + e >= P) continue;
         float o = 0.f;
         for (int s = 0; s < slices; s++) o += sums[s * PT + e];
@@ -652,12 +678,21 @@ IK_EXPORT int ik_ssd_decode(const float* p, int ldp, int x_off, const float* cw,
     if (P % 4 || (uintptr_t)state % 16) return IK_UNSUPPORTED;
     int pv_n = 1;
     while (pv_n < 16 && 4 * pv_n < P) pv_n *= 2;
-    const int PT = 4 * pv_n, slices = 128 / pv_n;
+    const int PT = 4 * pv_n, slices = DEC_THREADS / pv_n;
     const size_t smem = (size_t)(PT + 2 * N + slices * PT) * sizeof(float);
     if (smem > 48 * 1024) return IK_UNSUPPORTED;
     const dim3 grid(H, B, (P + PT - 1) / PT);
-    IK_RETURN_IF_ERROR(ik_launch(ssd_decode_kernel, grid, 128, smem, stream, p, ldp, x_off, cw, cb, taps > 1 ? ring : nullptr, dt_bias, A, Dv,
-                                 state, slots, cu_seqlens, kv_lens, out, H, G, N, P, taps, pv_n));
+#define IK_DEC(TAPS)                                                                                                                  \
+    IK_RETURN_IF_ERROR(ik_launch(ssd_decode_kernel<TAPS>, grid, DEC_THREADS, smem, stream, p, ldp, x_off, cw, cb, taps > 1 ? ring : nullptr, dt_bias, \
+                                 A, Dv, state, slots, cu_seqlens, kv_lens, out, H, G, N, P, taps, pv_n))
+    switch (taps) {
+        case 1: IK_DEC(1); break;
+        case 2: IK_DEC(2); break;
+        case 3: IK_DEC(3); break;
+        case 4: IK_DEC(4); break;
+        default: IK_DEC(0);
+    }
+#undef IK_DEC
     IK_LAUNCH_STATUS();
 }
 
