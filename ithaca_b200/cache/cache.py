@@ -33,6 +33,7 @@ class KVRequest:
     v_head_dim: Optional[int] = None        # size of a value head when it differs from the key head's
     values_in_keys: bool = False            # the values are columns of the key rows: no value pages are kept
     keep_first: int = 0                     # under a window: this many first keys of a sequence stay visible
+    key_scales: bool = False                # a float beside every key (per kv head), by which its scores are multiplied
 
 
 @dataclass(frozen=True)
@@ -52,6 +53,7 @@ class LayerCache:
     kv_group: Optional[int] = None          # index into StepContext.tables
     k_pages: Optional[torch.Tensor] = None  # [pages, kv_heads, page_size, head_dim]
     v_pages: Optional[torch.Tensor] = None
+    key_scales: Optional[torch.Tensor] = None   # float32 [pages, kv_heads, page_size], where the mixer asked for them
     window: Optional[int] = None
     states: Optional[Dict[str, torch.Tensor]] = None   # name -> [max_slots, *shape]
 
@@ -74,14 +76,14 @@ def plan_groups(requests: Mapping[int, Sequence[object]]):
                     raise CacheError(f"cache entry {entry} asks for keys and values twice")
                 seen_kv = True
                 kv_keys.setdefault((r.n_kv_heads, r.head_dim, r.window, 0 if r.values_in_keys else r.v_head_dim or r.head_dim,
-                                    r.keep_first if r.window is not None else 0), []).append(entry)
+                                    r.keep_first if r.window is not None else 0, r.key_scales), []).append(entry)
             elif isinstance(r, StateRequest):
                 if r.dtype not in _TORCH:
                     raise CacheError(f"state '{r.name}': dtype {r.dtype} is not supported")
                 st_keys.setdefault((r.name, tuple(r.shape), r.dtype), []).append(entry)
             else:
                 raise CacheError(f"cache entry {entry}: unknown request {r!r}")
-    kv_groups = [KVGroupLayout(k[0], k[1], k[2], tuple(v), k[3], k[4]) for k, v in kv_keys.items()]     # v_head_dim 0: no value pages
+    kv_groups = [KVGroupLayout(k[0], k[1], k[2], tuple(v), k[3], k[4], k[5]) for k, v in kv_keys.items()]     # v_head_dim 0: no value pages
     st_groups = [StateGroupLayout(k[1], k[2], tuple(v), k[0]) for k, v in st_keys.items()]
     return kv_groups, st_groups
 
@@ -107,6 +109,7 @@ class SequenceCache:
         self._views: Dict[int, LayerCache] = {}
         self.k: List[torch.Tensor] = []
         self.v: List[torch.Tensor] = []
+        self.key_scales: List[Optional[torch.Tensor]] = []
         self.state: List[torch.Tensor] = []
         if device is not None:
             for g in self.kv_groups:
@@ -114,6 +117,7 @@ class SequenceCache:
                 self.k.append(torch.zeros(shape, dtype=kv_dtype, device=device))
                 self.v.append(torch.zeros(shape[:-1] + (g.head_dim if g.v_head_dim is None else g.v_head_dim,), dtype=kv_dtype,
                                           device=device))
+                self.key_scales.append(torch.zeros(shape[:-1], dtype=torch.float32, device=device) if g.key_scales else None)
             for s in self.state_groups:
                 self.state.append(torch.zeros((len(s.cache_entries), max_slots) + tuple(s.shape),
                                               dtype=_TORCH[s.dtype], device=device))
@@ -126,6 +130,7 @@ class SequenceCache:
                     view.kv_group, view.window = gi, g.window
                     if device is not None:
                         view.k_pages, view.v_pages = self.k[gi][row], (self.v[gi][row] if g.v_head_dim != 0 else None)
+                        view.key_scales = self.key_scales[gi][row] if g.key_scales else None
             for si, s in enumerate(self.state_groups):
                 if e in s.cache_entries and device is not None:
                     view.states[s.name] = self.state[si][s.cache_entries.index(e)]
@@ -138,8 +143,8 @@ class SequenceCache:
 
     def bytes_per_token(self) -> int:
         el = torch.empty((), dtype=self.kv_dtype).element_size()
-        return sum(len(g.cache_entries) * g.n_kv_heads * (g.head_dim + (g.head_dim if g.v_head_dim is None else g.v_head_dim)) * el
-                   for g in self.kv_groups)
+        return sum(len(g.cache_entries) * g.n_kv_heads
+                   * ((g.head_dim + (g.head_dim if g.v_head_dim is None else g.v_head_dim)) * el + (4 if g.key_scales else 0)) for g in self.kv_groups)
 
     # -- slots ---------------------------------------------------------------------------------
     def alloc_slot(self) -> int:

@@ -70,6 +70,7 @@ class KVGroupLayout:
     cache_entries: tuple             # cache entries (of the schedule) stored in this group, in order
     v_head_dim: Optional[int] = None # size of a value head; None: as the key head; 0: the values lie in the key rows
     keep_first: int = 0              # under a window: the first keys of a sequence that stay visible to every later query
+    key_scales: bool = False               # a float32 number beside every key
 
 
 @dataclass(frozen=True)

@@ -17,6 +17,7 @@ from .llama import LlamaConfig
 from .mimadra import MimadraConfig
 from .tiralix import TiralixConfig
 from .vebisun import VebisunConfig
+from .vovalorn import VovalornConfig
 from .zomipel import ZomipelConfig
 
 
@@ -73,3 +74,4 @@ register_architecture(TiralixConfig.ARCHITECTURE, TiralixConfig)
 register_architecture(MimadraConfig.ARCHITECTURE, MimadraConfig)
 register_architecture(GunenexConfig.ARCHITECTURE, GunenexConfig)
 register_architecture(ZomipelConfig.ARCHITECTURE, ZomipelConfig)
+register_architecture(VovalornConfig.ARCHITECTURE, VovalornConfig)

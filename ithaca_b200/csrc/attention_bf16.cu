@@ -24,6 +24,19 @@
 #include "common.cuh"
 #include "tc_common.cuh"
 
+// Two compile-time options make further modules of the same size; a module without them has none of their code.
+//  * IK_SLOPES=1: a score loses slope[head] * (i - j) behind the cap (a distance bias), and the cap's tanh is accurate
+//    to float rounding (below).
+//  * IK_ONE_ROW=1: a page's rows are keys and values (there are no value pages), and every key has a float beside it
+//    (scales[page][kv head][place]) by which its scores are multiplied: the norm of a key whose value is the key in
+//    front of the norm.  A row is brought on chip once and serves both products.
+#ifndef IK_SLOPES
+#define IK_SLOPES 0
+#endif
+#ifndef IK_ONE_ROW
+#define IK_ONE_ROW 0
+#endif
+
 #ifndef IK_HD
 #error "compile with -DIK_HD=<head size>"
 #endif
@@ -32,6 +45,7 @@ namespace {
 
 constexpr int HD = IK_HD;
 constexpr int PAGE = 64;
+constexpr bool SLOPES = IK_SLOPES != 0, ONE_ROW = IK_ONE_ROW != 0;
 constexpr int LD = HD + 8;                 // padded row: consecutive rows fall into different banks
 static_assert(HD % 16 == 0 && HD >= 16 && HD <= 512, "head size must be a multiple of 16 up to 512");
 
@@ -72,6 +86,23 @@ __device__ __forceinline__ float ik_tanh_fast(float x) {
 __device__ __forceinline__ float ik_capped(float s, float a, float b) {
     return b != 0.f ? b * ik_tanh_fast(s * a) : s * a;
 }
+// tanh to float rounding: near zero x times its Taylor polynomial in x^2 up to x^11, whose first term left out is below 2^-23 of
+// the result for |x| <= TANH_NEAR; else 1 - 2 / (1 + e^(2|x|)) with the hardware's exponential and a division, whose error is
+// a few 2^-24 of a result that is at least 0.37.
+constexpr float TANH_NEAR = 0.4f;
+__device__ __forceinline__ float ik_tanh_series(float x2) {           // tanh(x) / x
+    return fmaf(x2, fmaf(x2, fmaf(x2, fmaf(x2, fmaf(x2, -1382.0f / 155925.0f, 62.0f / 2835.0f), -17.0f / 315.0f), 2.0f / 15.0f), -1.0f / 3.0f), 1.0f);
+}
+__device__ __forceinline__ float ik_tanh_far(float x) {
+    const float e = ik_ex2(fminf(fabsf(x), 20.f) * 2.885390081777927f);
+    return copysignf(1.0f - __fdividef(2.0f, 1.0f + e), x);
+}
+// A score of the modules with options: s * key_scale, then the scale or the cap, then the distance bias; base 2.
+__device__ __forceinline__ float ik_score(float s, float key_scale, float a, float b, float slope_log2e, int distance) {
+    float x = (ONE_ROW ? s * key_scale : s) * a;
+    if (b != 0.f) x = b * (fabsf(x) <= TANH_NEAR ? x * ik_tanh_series(x * x) : ik_tanh_far(x));
+    return SLOPES ? fmaf(-slope_log2e, (float)distance, x) : x;
+}
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<uint32_t*>(&v);
@@ -88,14 +119,16 @@ __global__ void __launch_bounds__(32 * NW)
 attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                     bf16* __restrict__ out, const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
                     const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window, int keep,
-                    int sink, const float* __restrict__ sink_v, int n_pages, int* status) {
+                    int sink, const float* __restrict__ sink_v, const float* __restrict__ key_scales, const float* __restrict__ slopes,
+                    int n_pages, int* status) {
     ik_pdl_wait();
     ik_pdl_launch_dependents();
     constexpr int BM = 16 * NW, THREADS = 32 * NW, CH = HD / 8;          // CH: 16-byte chunks per row
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = (bf16*)smem_raw;                      // [BM][LD]
     bf16* Ks = Qs + BM * LD;                         // [2][PAGE][LD]
-    bf16* Vs = Ks + 2 * PAGE * LD;                   // [2][PAGE][LD]
+    bf16* Vs = ONE_ROW ? Ks : Ks + 2 * PAGE * LD;    // [2][PAGE][LD]
+    float* Cs = (float*)(Vs + 2 * PAGE * LD);        // [2][PAGE] the keys' scales (ONE_ROW)
 
     const int b = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
     const int q_begin = cu_seqlens[b], n_new = cu_seqlens[b + 1] - q_begin;
@@ -125,9 +158,12 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
         for (int idx = threadIdx.x; idx < PAGE * CH; idx += THREADS) {
             const int r = idx / CH, c = idx % CH;
             cp16(ks + r * LD + c * 8, kg + r * HD + c * 8, true);
-            cp16(vs + r * LD + c * 8, vg + r * HD + c * 8, true);
+            if (!ONE_ROW) cp16(vs + r * LD + c * 8, vg + r * HD + c * 8, true);
         }
+        if (ONE_ROW && threadIdx.x < PAGE / 4)
+            cp16(Cs + stage * PAGE + threadIdx.x * 4, key_scales + ((size_t)page * nkv + kvh) * PAGE + threadIdx.x * 4, true);
     };
+    const float slope = SLOPES && slopes ? slopes[h] * 1.4426950408889634f : 0.f;
     load_page(0, page_at(0, n_kept, p_lo));
     cp_commit();
 
@@ -182,7 +218,10 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
             for (int e = 0; e < 4; e++) {
                 const int r = e >> 1, j = jbase + n * 8 + (e & 1);
                 const bool ok = my_row[r] && j <= my_pos[r] && (window <= 0 || j > my_pos[r] - window || j < keep);
-                const float v = ok ? ik_capped(s[n][e], scale_log2e, cap_log2e) : -INFINITY;
+                float raw;
+                if (SLOPES || ONE_ROW) raw = ik_score(s[n][e], ONE_ROW ? Cs[stage * PAGE + 2 * t + n * 8 + (e & 1)] : 1.f, scale_log2e, cap_log2e, slope, my_pos[r] - j);
+                else raw = ik_capped(s[n][e], scale_log2e, cap_log2e);
+                const float v = ok ? raw : -INFINITY;
                 s[n][e] = v;
                 mx[r] = fmaxf(mx[r], v);
             }
@@ -265,20 +304,41 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
 // All mbarrier waits are bounded (tc_common.cuh); on a timeout the status word is set and the block
 // leaves its loops and frees its TMEM.
 #if IK_HD == 64 || IK_HD == 128
-constexpr int TC_BM = 128, TC_NS = 2;                          // two blocks per SM: one's softmax runs beside the other's MMAs
+constexpr int TC_BM = 128, TC_NS = ONE_ROW ? 4 : 2;            // two blocks per SM: one's softmax runs beside the other's MMAs
 constexpr int TC_BOXES = HD / 64;                              // 64-wide swizzled blocks along the head size
 constexpr int TC_Q_BYTES = TC_BM * HD * 2;
 constexpr int TC_KV_BYTES = PAGE * HD * 2;
-constexpr int TC_SMEM = TC_Q_BYTES + TC_NS * 2 * TC_KV_BYTES + 256;   // no slack for alignment: see the check in the kernel
+constexpr int TC_SMEM = TC_Q_BYTES + TC_NS * (ONE_ROW ? TC_KV_BYTES + PAGE * 4 : 2 * TC_KV_BYTES) + 256;   // no slack for alignment: see the check in the kernel
 constexpr int TC_TMEM_COLS = 256;                              // scores 2 x 64, output HD (<= 128)
 constexpr int TC_O_COL = 128;
+
+// An untiled copy of `bytes` (a multiple of 16, both addresses on 16-byte boundaries) that completes on a barrier.
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                 :: "r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+// (x0, x1) <- b * tanh(x0, x1), both within TANH_NEAR: two floats per instruction
+__device__ __forceinline__ void tanh_series_f32x2(float& x0, float& x1, float b) {
+    auto two = [](float a, float c) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(c)); return r; };
+    auto fma2 = [](uint64_t a, uint64_t c, uint64_t d) { uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(c), "l"(d)); return r; };
+    auto mul2 = [](uint64_t a, uint64_t c) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(c)); return r; };
+    const uint64_t x = two(x0, x1), x2 = mul2(x, x);
+    uint64_t t = fma2(x2, two(-1382.0f / 155925.0f, -1382.0f / 155925.0f), two(62.0f / 2835.0f, 62.0f / 2835.0f));
+    t = fma2(x2, t, two(-17.0f / 315.0f, -17.0f / 315.0f));
+    t = fma2(x2, t, two(2.0f / 15.0f, 2.0f / 15.0f));
+    t = fma2(x2, t, two(-1.0f / 3.0f, -1.0f / 3.0f));
+    t = fma2(x2, t, two(1.0f, 1.0f));
+    const uint64_t y = mul2(mul2(x, two(b, b)), t);
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(x0), "=f"(x1) : "l"(y));
+}
 
 __global__ void __launch_bounds__(192, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
                        const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
                        const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e,
-                       int window, int keep, int sink, const float* __restrict__ sink_v, int n_pages, int* status) {
+                       int window, int keep, int sink, const float* __restrict__ sink_v, const float* __restrict__ key_scales,
+                       const float* __restrict__ slopes, int n_pages, int* status) {
     extern __shared__ __align__(1024) unsigned char tc_smem[];
     ik_pdl_wait();
     ik_pdl_launch_dependents();
@@ -305,8 +365,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     }
     unsigned char* Qs = tc_smem;
     unsigned char* Ks = Qs + TC_Q_BYTES;                       // [TC_NS][TC_KV_BYTES]
-    unsigned char* Vs = Ks + TC_NS * TC_KV_BYTES;
-    uint64_t* q_full = (uint64_t*)(Vs + TC_NS * TC_KV_BYTES);
+    unsigned char* Vs = ONE_ROW ? Ks : Ks + TC_NS * TC_KV_BYTES;
+    float* Cs = (float*)(Vs + TC_NS * TC_KV_BYTES);            // [TC_NS][PAGE] the keys' scales (ONE_ROW)
+    uint64_t* q_full = (uint64_t*)(Cs + (ONE_ROW ? TC_NS * PAGE : 0));
     uint64_t* k_full = q_full + 1;                             // [TC_NS]
     uint64_t* v_full = k_full + TC_NS;
     uint64_t* k_free = v_full + TC_NS;
@@ -354,8 +415,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 if (page < 0 || page >= n_pages) { ik_set_status(status, IK_STATUS_READ_NO_PAGE); page = 0; }
                 return (page * nkv + kvh) * PAGE;
             };
+            // rows that are keys and values: one ring, a stage is free once O += P V has read it
+            for (int i = 0; ONE_ROW && i < n_iter; i++) {
+                const int s = i % TC_NS;
+                if (!mbar_wait(k_free + s, ((i / TC_NS) & 1) ^ 1, abort_flag, status, IK_WAIT_LIMIT_NS, 11, i)) break;
+                const int row = page_row(i);
+                mbar_expect_tx(k_full + s, TC_KV_BYTES + PAGE * 4);
+                for (int bx = 0; bx < TC_BOXES; bx++)
+                    tma_load_2d(Ks + s * TC_KV_BYTES + bx * (PAGE * 128), &map_k, bx * 64, row, k_full + s);
+                bulk_load(Cs + s * PAGE, key_scales + row, PAGE * 4, k_full + s);
+            }
             // keys of page i, then values of page i - 1
-            for (int i = 0; i <= n_iter; i++) {
+            for (int i = 0; !ONE_ROW && i <= n_iter; i++) {
                 if (i < n_iter) {
                     const int s = i % TC_NS;
                     if (!mbar_wait(k_free + s, ((i / TC_NS) & 1) ^ 1, abort_flag, status, IK_WAIT_LIMIT_NS, 11, i)) break;
@@ -389,14 +460,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                     umma(tmem + (i & 1) * PAGE, umma_desc(q_addr + (j / 4) * (TC_BM * 128) + (j % 4) * 32),
                          umma_desc(k_addr + (j / 4) * (PAGE * 128) + (j % 4) * 32), idesc_qk, j != 0);
                 umma_commit(s_full + (i & 1));
-                umma_commit(k_free + s);                   // the key stage is free once these products have read it
+                if (!ONE_ROW) umma_commit(k_free + s);     // the key stage is free once these products have read it
                 return true;
             };
             if (ok) ok = issue_qk(0);
             for (int i = 0; i < n_iter && ok; i++) {
                 if (i + 1 < n_iter) { ok = issue_qk(i + 1); if (!ok) break; }     // runs while page i is in the softmax
                 const int s = i % TC_NS;
-                ok = mbar_wait(p_ready + (i & 1), (i >> 1) & 1, abort_flag, status, IK_WAIT_LIMIT_NS, 15, i) && mbar_wait(v_full + s, (i / TC_NS) & 1, abort_flag, status, IK_WAIT_LIMIT_NS, 16, i);
+                ok = mbar_wait(p_ready + (i & 1), (i >> 1) & 1, abort_flag, status, IK_WAIT_LIMIT_NS, 15, i) && (ONE_ROW || mbar_wait(v_full + s, (i / TC_NS) & 1, abort_flag, status, IK_WAIT_LIMIT_NS, 16, i));
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const uint32_t v_addr = smem_u32(Vs + s * TC_KV_BYTES);
@@ -404,7 +475,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 for (int j = 0; j < PAGE / 16; j++)
                     umma_ts(tmem + TC_O_COL, tmem + (i & 1) * PAGE + j * 8, umma_desc_mn(v_addr + j * 2048, PAGE * 128),
                             idesc_pv, (i | j) != 0);
-                umma_commit(v_free + s);
+                umma_commit(ONE_ROW ? k_free + s : v_free + s);
                 umma_commit(pv_done);
             }
             if (ok) umma_commit(o_done);
@@ -416,6 +487,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         const int pos_r = pos_lo + r;
         // a sink: one more key without a value, of score 0 or (sink_v) of the head's own score, in base-2 units
         float m = sink ? (sink_v ? sink_v[h] * 1.4426950408889634f : 0.f) : -INFINITY, l = sink ? 1.f : 0.f;
+        const float slope = SLOPES && slopes ? slopes[h] * 1.4426950408889634f : 0.f;
         bool ok = true;
         for (int i = 0; i < n_iter && ok; i++) {
             const int p = page_at(i, n_kept, p_lo);
@@ -426,11 +498,49 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             #pragma unroll
             for (int c0 = 0; c0 < PAGE; c0 += 16) tmem_ld16_issue(lane_base + (i & 1) * PAGE + c0, sc + c0);
             tmem_ld_wait();
-            if (cap_log2e != 0.f) {                        // capped scores: tanh is monotone, so the maximum below still holds
+            float shift = 0.f;                             // of the page's scores for this row, beside what sc holds
+            if (SLOPES || ONE_ROW) {
+                // key scale and scale (or scale / cap)
+                if (ONE_ROW) {
+                    // the loader's copies are visible to who has seen their barrier; a stage is filled anew only after this
+                    // thread has arrived on p_ready for the page it holds now, so the parity names the right phase
+                    ok = mbar_wait(k_full + i % TC_NS, (i / TC_NS) & 1, abort_flag, status, IK_WAIT_LIMIT_NS, 22, i);
+                    if (!ok) break;
+                    const float4* cs = reinterpret_cast<const float4*>(Cs + (i % TC_NS) * PAGE);
+                    #pragma unroll
+                    for (int c = 0; c < PAGE; c += 4) {
+                        const float4 k4 = cs[c / 4];
+                        sc[c] *= k4.x * scale_log2e; sc[c + 1] *= k4.y * scale_log2e; sc[c + 2] *= k4.z * scale_log2e; sc[c + 3] *= k4.w * scale_log2e;
+                    }
+                } else {
+                    #pragma unroll
+                    for (int c = 0; c < PAGE; c++) sc[c] *= scale_log2e;
+                }
+                if (cap_log2e != 0.f) {
+                    float far[4] = {0.f, 0.f, 0.f, 0.f};
+                    #pragma unroll
+                    for (int c = 0; c < PAGE; c += 2) far[(c >> 1) & 3] = max3(far[(c >> 1) & 3], fabsf(sc[c]), fabsf(sc[c + 1]));
+                    const bool near = fmaxf(fmaxf(far[0], far[1]), fmaxf(far[2], far[3])) <= TANH_NEAR;
+                    if (__all_sync(0xffffffffu, near)) {
+                        #pragma unroll
+                        for (int c = 0; c < PAGE; c += 2) tanh_series_f32x2(sc[c], sc[c + 1], cap_log2e);
+                    } else {
+                        #pragma unroll
+                        for (int c = 0; c < PAGE; c++)
+                            sc[c] = cap_log2e * (fabsf(sc[c]) <= TANH_NEAR ? sc[c] * ik_tanh_series(sc[c] * sc[c]) : ik_tanh_far(sc[c]));
+                    }
+                }
+                if (SLOPES) {
+                    // -slope (pos_r - j) = slope c + slope (p PAGE - pos_r): the row's part is left for the subtraction below
+                    shift = slope * (float)(p * PAGE - pos_r);
+                    #pragma unroll
+                    for (int c = 0; c < PAGE; c++) sc[c] = fmaf(slope, (float)c, sc[c]);
+                }
+            } else if (cap_log2e != 0.f) {                 // capped scores: tanh is monotone, so the maximum below still holds
                 #pragma unroll
                 for (int c = 0; c < PAGE; c++) sc[c] = cap_log2e * ik_tanh_fast(sc[c] * scale_log2e);
             }
-            const float mul = cap_log2e != 0.f ? 1.f : scale_log2e;
+            const float mul = (SLOPES || ONE_ROW || cap_log2e != 0.f) ? 1.f : scale_log2e;
             const bool need_mask = (p * PAGE + PAGE - 1 > pos_lo) || (window > 0 && p * PAGE < pos_hi + 1 - window && p * PAGE + PAGE > keep);
             // Few instructions per score: the maximum is taken over the raw scores and scaled once (the scale is
             // positive), and the scaling of a score is folded into the subtraction of the reference below.  Four
@@ -450,7 +560,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 #pragma unroll
                 for (int c = 0; c < PAGE; c += 2) mx4[(c >> 1) & 3] = max3(mx4[(c >> 1) & 3], sc[c], sc[c + 1]);
             }
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * mul;
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * mul + shift;
             // m is the reference the exponentials are taken against.  It follows the running maximum only when
             // that has moved by more than 8 (a factor 256): until then the probabilities may exceed 1 by that
             // factor, which float sums and bfloat16 operands take in their stride, and O needs no rescaling.
@@ -464,7 +574,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             #pragma unroll
             for (int c = 0; c < PAGE; c += 2) {            // two scores per multiply-add and per add
                 float a0, a1;
-                fma_f32x2(a0, a1, sc[c], sc[c + 1], mul, -m_use);
+                fma_f32x2(a0, a1, sc[c], sc[c + 1], mul, shift - m_use);
                 sc[c] = ik_ex2(a0);
                 sc[c + 1] = ik_ex2(a1);
                 add_f32x2(sum4[c & 2], sum4[(c & 2) + 1], sc[c], sc[c + 1]);
@@ -553,13 +663,14 @@ __global__ void __launch_bounds__(128)
 attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                    float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ kv_lens,
                    const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window, int keep,
-                   int n_pages, int chunk_pages, int n_splits, int* status) {
+                   const float* __restrict__ key_scales, const float* __restrict__ slopes, int n_pages, int chunk_pages, int n_splits, int* status) {
     ik_pdl_wait();
     constexpr int CH = HD / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = (bf16*)smem_raw;                      // [16][LD]
     bf16* Ks = Qs + 16 * LD;                         // [NS][PAGE][LD]
-    bf16* Vs = Ks + NS * PAGE * LD;                  // [NS][PAGE][LD]
+    bf16* Vs = ONE_ROW ? Ks : Ks + NS * PAGE * LD;   // [NS][PAGE][LD]
+    float* Cs = (float*)(Vs + NS * PAGE * LD);       // [NS][PAGE] the keys' scales (ONE_ROW)
 
     const int b = blockIdx.x, split = blockIdx.z;
     const int G = nh / nkv, n_hc = (G + 15) / 16;
@@ -590,9 +701,16 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
         for (int idx = threadIdx.x; idx < PAGE * CH; idx += 128) {
             const int r = idx / CH, c = idx % CH;
             cp16(ks + r * LD + c * 8, kg + r * HD + c * 8, true);
-            cp16(vs + r * LD + c * 8, vg + r * HD + c * 8, true);
+            if (!ONE_ROW) cp16(vs + r * LD + c * 8, vg + r * HD + c * 8, true);
         }
+        if (ONE_ROW && threadIdx.x < PAGE / 4)
+            cp16(Cs + stage * PAGE + threadIdx.x * 4, key_scales + ((size_t)page * nkv + kvh) * PAGE + threadIdx.x * 4, true);
     };
+    float slope[2] = {0.f, 0.f};
+    if (SLOPES && slopes) {
+        if ((threadIdx.x & 31) / 4 < n_here) slope[0] = slopes[h0 + (threadIdx.x & 31) / 4] * 1.4426950408889634f;
+        if ((threadIdx.x & 31) / 4 + 8 < n_here) slope[1] = slopes[h0 + (threadIdx.x & 31) / 4 + 8] * 1.4426950408889634f;
+    }
     #pragma unroll
     for (int s = 0; s < NS; s++) {
         if (i_first + s <= i_last) load_page(s, page_at(i_first + s, n_kept, p_lo));
@@ -639,7 +757,10 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
             for (int e = 0; e < 4; e++) {
                 const int r = e >> 1, j = jbase + n * 8 + (e & 1);
                 const bool ok = my_row[r] && j <= pos && (j >= j0 || j < keep);
-                const float v = ok ? ik_capped(s[n][e], scale_log2e, cap_log2e) : -INFINITY;
+                float raw;
+                if (SLOPES || ONE_ROW) raw = ik_score(s[n][e], ONE_ROW ? Cs[stage * PAGE + warp * 16 + 2 * t + n * 8 + (e & 1)] : 1.f, scale_log2e, cap_log2e, slope[r], pos - j);
+                else raw = ik_capped(s[n][e], scale_log2e, cap_log2e);
+                const float v = ok ? raw : -INFINITY;
                 s[n][e] = v;
                 mx[r] = fmaxf(mx[r], v);
             }
@@ -756,20 +877,24 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
 
 IK_EXPORT int ik_attn_head_dim() { return HD; }
 
+// A module takes slopes only if it was compiled for them, and rows that are keys and values need their keys' scales.
+static bool options_fit(const float* key_scales, const float* slopes) { return (SLOPES || !slopes) && ONE_ROW == (key_scales != nullptr); }
+
 // Sites of the tcgen05 prefill kernel's waits: 11, 12 = loader for a free key / value stage; 13 = issuer for the
 // queries; 14 = issuer for keys; 15 = issuer for the probabilities; 16 = issuer for values; 17 = softmax for scores;
-// 18 = softmax for the product before a rescaling; 21 = softmax for the tile's last product.
+// 18 = softmax for the product before a rescaling; 21 = softmax for the tile's last product; 22 = softmax for the keys' scales.
 IK_EXPORT int ik_attn_take_wait_record(int* out4) { return ik_take_wait_record(out4); }
 
 IK_EXPORT int ik_attn_prefill(const void* q, const void* k_pages, const void* v_pages, void* out, const int* cu_seqlens,
                               const int* kv_lens, const int* table, int table_stride, int B, int max_new, int nh,
-                              int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, int page_size, int n_pages, int* status,
-                              cudaStream_t stream) {
+                              int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, const float* key_scales,
+                              const float* slopes, int page_size, int n_pages, int* status, cudaStream_t stream) {
+    if (!options_fit(key_scales, slopes)) return IK_UNSUPPORTED;
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     if (B <= 0 || max_new <= 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size != PAGE || B > 65535 || nh > 65535)
         return IK_BAD_ARGUMENT;
     constexpr int NW = 4, BM = 16 * NW;
-    const size_t smem = (size_t)(BM + 4 * PAGE) * LD * sizeof(bf16);
+    const size_t smem = (size_t)(BM + (ONE_ROW ? 2 : 4) * PAGE) * LD * sizeof(bf16) + (ONE_ROW ? 2 * PAGE * sizeof(float) : 0);
     auto kern = attn_prefill_kernel<NW>;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -778,20 +903,22 @@ IK_EXPORT int ik_attn_prefill(const void* q, const void* k_pages, const void* v_
     dim3 grid((max_new + BM - 1) / BM, nh, B);
     IK_RETURN_IF_ERROR(ik_launch(kern, grid, 32 * NW, smem, stream, (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, (bf16*)out,
                                           cu_seqlens, kv_lens, table, table_stride, nh, nkv,
-                                          sc_a, sc_b, window, keep, sink, sink_v, n_pages, status));
+                                          sc_a, sc_b, window, keep, sink, sink_v, key_scales, slopes, n_pages, status));
     IK_LAUNCH_STATUS();
 }
 
 // The tcgen05 kernel (head sizes 64 and 128; IK_UNSUPPORTED otherwise).  T: rows of q.
 IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void* v_pages, void* out, const int* cu_seqlens,
                                  const int* kv_lens, const int* table, int table_stride, int T, int B, int max_new, int nh,
-                                 int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, int page_size, int n_pages, int* status,
-                                 cudaStream_t stream) {
+                                 int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, const float* key_scales,
+                                 const float* slopes, int page_size, int n_pages, int* status, cudaStream_t stream) {
+    if (!options_fit(key_scales, slopes)) return IK_UNSUPPORTED;
 #if IK_HD == 64 || IK_HD == 128
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     if (T <= 0 || B <= 0 || max_new <= 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size != PAGE || B > 65535 || nh > 65535)
         return IK_BAD_ARGUMENT;
-    if (((uintptr_t)q % 16) || ((uintptr_t)k_pages % 16) || ((uintptr_t)v_pages % 16)) return IK_UNSUPPORTED;
+    if (ONE_ROW) v_pages = k_pages;
+    if (((uintptr_t)q % 16) || ((uintptr_t)k_pages % 16) || ((uintptr_t)v_pages % 16) || ((uintptr_t)key_scales % 16)) return IK_UNSUPPORTED;
     if (!(scale > 0.f)) return IK_UNSUPPORTED;             // the kernel takes the maximum of the raw scores
     CUtensorMap mq, mk, mv;
     int st = ik_make_map(&mq, q, (unsigned long long)T, nh * HD, (unsigned long long)nh * HD, TC_BM);
@@ -806,7 +933,7 @@ IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void*
     if (e != cudaSuccess) return (int)e;
     dim3 grid((max_new + TC_BM - 1) / TC_BM, nh, B);
     IK_RETURN_IF_ERROR(ik_launch(kern, grid, 192, TC_SMEM, stream, mq, mk, mv, (bf16*)out, cu_seqlens, kv_lens, table,
-                                 table_stride, nh, nkv, sc_a, sc_b, window, keep, sink, sink_v, n_pages, status));
+                                 table_stride, nh, nkv, sc_a, sc_b, window, keep, sink, sink_v, key_scales, slopes, n_pages, status));
     IK_LAUNCH_STATUS();
 #else
     return IK_UNSUPPORTED;
@@ -818,8 +945,10 @@ IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void*
 // its pages; with one: those of the first `keep` keys and those the window reaches into).
 IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_pages, void* out, float* part_o,
                              float* part_ml, const int* kv_lens, const int* table, int table_stride, int B, int nh,
-                             int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, int page_size, int n_pages, int chunk_pages,
-                             int n_splits, int ring_kb, int* status, cudaStream_t stream) {
+                             int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, const float* key_scales,
+                             const float* slopes, int page_size, int n_pages, int chunk_pages, int n_splits, int ring_kb, int* status,
+                             cudaStream_t stream) {
+    if (!options_fit(key_scales, slopes)) return IK_UNSUPPORTED;
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     if (B <= 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size != PAGE || chunk_pages <= 0 || n_splits <= 0 ||
         n_splits > 65535)
@@ -828,11 +957,14 @@ IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_p
     if ((long long)nkv * n_hc > 65535) return IK_BAD_ARGUMENT;
     dim3 grid(B, nkv * n_hc, n_splits);
     // as many ring stages as fit ring_kb (default 105 KB), at least 2, at most 4
-    const size_t q_bytes = (size_t)16 * LD * sizeof(bf16), stage_bytes = (size_t)2 * PAGE * LD * sizeof(bf16);
+    const size_t q_bytes = (size_t)16 * LD * sizeof(bf16), stage_bytes = ONE_ROW ? PAGE * (LD * sizeof(bf16) + sizeof(float))
+                                                                                              : (size_t)2 * PAGE * LD * sizeof(bf16);
     if (ring_kb <= 0) ring_kb = 105;
     int ns = (int)(((size_t)ring_kb * 1024 - q_bytes) / stage_bytes);
     ns = ns < 2 ? 2 : ns > 4 ? 4 : ns;
-    const size_t smem = q_bytes + ns * stage_bytes;
+    // the ring's space is also where the warps' partial results meet at the end
+    const size_t merge_bytes = (size_t)4 * 16 * (HD + 2) * sizeof(float);
+    const size_t smem = q_bytes + (ns * stage_bytes > merge_bytes ? ns * stage_bytes : merge_bytes);
 #define IK_DEC(NS_)                                                                                                  \
     {                                                                                                                \
         auto kern = attn_decode_kernel<NS_>;                                                                         \
@@ -842,7 +974,7 @@ IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_p
         }                                                                                                            \
         IK_RETURN_IF_ERROR(ik_launch(kern, grid, 128, smem, stream, (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, part_o, part_ml, \
                                           kv_lens, table, table_stride, nh, nkv, sc_a, sc_b, window, keep, \
-                                          n_pages, chunk_pages, n_splits, status));                                   \
+                                          key_scales, slopes, n_pages, chunk_pages, n_splits, status));                                   \
     }
     if (ns == 2) IK_DEC(2) else if (ns == 3) IK_DEC(3) else IK_DEC(4)
 #undef IK_DEC

@@ -13,6 +13,10 @@
 // (pages[page][kv head][position in page][size], page = table[seq * table_stride + pos / page_size]).
 // `bias` (or null) is a vector over p's columns that is added to q, k and v as they are read.  With v_norm every value head
 // is divided by the root mean square of its own hdv values (eps inside the root, no weight) before it is stored.
+// per_head = 2: every q and k head is divided by the root mean square of its own values and there is no weight.  q is then
+// multiplied by 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1) (temp_every 0: by nothing).  key_scales (per_head = 2): the
+// key is stored as projected, for it is the value too (there are no value pages), and 1 / its root mean square goes to the
+// key's place among the scales (scales[page][kv head][position in page]).
 template <typename TQ, typename TC>
 __global__ void __launch_bounds__(256)
 norm_rope_append_kernel(const float* __restrict__ p, int ldp, int q_off, int k_off, int v_off, const float* __restrict__ q_w,
@@ -20,7 +24,7 @@ norm_rope_append_kernel(const float* __restrict__ p, int ldp, int q_off, int k_o
                         TC* __restrict__ v_pages, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                         const int* __restrict__ table, int table_stride, const float* __restrict__ inv_freq, float magnitude,
                         int nh, int nkv, int hd, int hdv, int rot, int pairing, int page_size, int n_pages, int write_cache,
-                        int per_head, const float* __restrict__ bias, int v_norm, int* status) {
+                        int per_head, const float* __restrict__ bias, int v_norm, float temp_coef, int temp_every, float* __restrict__ key_scales, int* status) {
     extern __shared__ __align__(16) float cs[];          // [rot/2] cos, [rot/2] sin, [nh + nkv] 1 / rms (per_head), [nkv] 1 / rms of v
     __shared__ float red[32];
     ik_pdl_wait();
@@ -31,6 +35,8 @@ norm_rope_append_kernel(const float* __restrict__ p, int ldp, int q_off, int k_o
     ik_pdl_launch_dependents();
     const int t = blockIdx.x, half = rot / 2, pos = token_pos[t];
     const float* row = p + (size_t)t * ldp;
+    const float temp = temp_every > 0 ? fmaf(temp_coef, logf((float)((pos + 1) / temp_every + 1)), 1.0f) : 1.0f;
+    const bool unit = per_head == 2;
     for (int i = threadIdx.x; i < half; i += 256) {
         const float ang = __fmul_rn((float)pos, inv_freq[i]);
         cs[i] = cosf(ang) * magnitude;
@@ -58,7 +64,7 @@ norm_rope_append_kernel(const float* __restrict__ p, int ldp, int q_off, int k_o
             const float* src = row + col;
             const float* b = bias ? bias + col : nullptr;
             float ss = 0.f;
-            if (is_q ? q_w != nullptr : k_w != nullptr) {
+            if (unit || (is_q ? q_w != nullptr : k_w != nullptr)) {
                 for (int i = threadIdx.x & 31; i < hd; i += 32) { const float v = b ? src[i] + b[i] : src[i]; ss = fmaf(v, v, ss); }
                 #pragma unroll
                 for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
@@ -97,22 +103,25 @@ norm_rope_append_kernel(const float* __restrict__ p, int ldp, int q_off, int k_o
         const float* w = is_q ? (q_w ? q_w + (per_head ? 0 : head * hd) : nullptr) : (k_w ? k_w + (per_head ? 0 : (head - nh) * hd) : nullptr);
         const float r = per_head ? head_r[head] : is_q ? rq : rk;
         const float mine = b ? src[i] + b[i] : src[i];
-        float val = w ? mine * r * w[i] : mine;
+        const bool scaled = unit && (is_q || !key_scales);
+        float val = w ? mine * r * w[i] : scaled ? mine * r : mine;
         if (i < rot) {
             int partner, f;
             bool first;
             if (pairing == 0) { first = i < half; partner = first ? i + half : i - half; f = first ? i : i - half; }
             else { first = (i & 1) == 0; partner = first ? i + 1 : i - 1; f = i >> 1; }
             const float theirs = b ? src[partner] + b[partner] : src[partner];
-            const float other = w ? theirs * r * w[partner] : theirs;
+            const float other = w ? theirs * r * w[partner] : scaled ? theirs * r : theirs;
             const float c = cs[f], s = cs[half + f];
             // (u, v) -> (u c - v s, v c + u s); `first` holds u
             val = first ? __fsub_rn(__fmul_rn(val, c), __fmul_rn(other, s)) : __fadd_rn(__fmul_rn(val, c), __fmul_rn(other, s));
         }
-        if (is_q) ik_st(q_out, ((size_t)t * nh + head) * hd + i, val);
+        if (is_q) ik_st(q_out, ((size_t)t * nh + head) * hd + i, val * temp);
         else ik_st(k_pages, (page_off + (size_t)(head - nh) * page_size) * hd + i, val);
     }
-    if (page_ok) {
+    if (page_ok && key_scales) {
+        for (int head = threadIdx.x; head < nkv; head += 256) key_scales[page_off + (size_t)head * page_size] = head_r[nh + head];
+    } else if (page_ok) {
         for (int e = threadIdx.x; e < nkv * hdv; e += 256) {
             const int head = e / hdv, i = e - head * hdv;
             float val = row[v_off + e];
@@ -127,17 +136,19 @@ IK_EXPORT int ik_norm_rope_append(const float* p, int ldp, int q_off, int k_off,
                                   float eps, void* q_out, int q_dtype, void* k_pages, void* v_pages, int cache_dtype,
                                   const int* token_seq, const int* token_pos, const int* table, int table_stride,
                                   const float* inv_freq, float magnitude, int T, int nh, int nkv, int hd, int hdv, int rot,
-                                  int pairing, int page_size, int n_pages, int write_cache, int per_head, const float* bias, int v_norm, int* status,
-                                  cudaStream_t stream) {
+                                  int pairing, int page_size, int n_pages, int write_cache, int per_head, const float* bias, int v_norm, float temp_coef, int temp_every,
+                                  float* key_scales, int* status, cudaStream_t stream) {
     if (T < 0 || nh <= 0 || nkv <= 0 || hd <= 0 || hdv <= 0 || rot < 0 || rot > hd || (rot & 1) || page_size <= 0)
         return IK_BAD_ARGUMENT;
     if (rot > 0 && !inv_freq) return IK_BAD_ARGUMENT;
+    if (per_head < 0 || per_head > 2 || (per_head == 2 && (q_w || k_w)) || temp_every < 0) return IK_BAD_ARGUMENT;
+    if (key_scales ? per_head != 2 || rot || v_norm : !v_pages) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
     const size_t smem = (size_t)(rot + (per_head ? nh + nkv : 0) + (v_norm ? nkv : 0)) * sizeof(float);
 #define IK_NRA(TQ, TC)                                                                                                       \
     IK_RETURN_IF_ERROR(ik_launch(norm_rope_append_kernel<TQ, TC>, T, 256, smem, stream, p, ldp, q_off, k_off, v_off, q_w, k_w, eps, \
                                  (TQ*)q_out, (TC*)k_pages, (TC*)v_pages, token_seq, token_pos, table, table_stride, inv_freq,  \
-                                 magnitude, nh, nkv, hd, hdv, rot, pairing, page_size, n_pages, write_cache, per_head, bias, v_norm, status))
+                                 magnitude, nh, nkv, hd, hdv, rot, pairing, page_size, n_pages, write_cache, per_head, bias, v_norm, temp_coef, temp_every, key_scales, status))
     if (q_dtype == IK_F32 && cache_dtype == IK_F32) IK_NRA(float, float);
     else if (q_dtype == IK_BF16 && cache_dtype == IK_BF16) IK_NRA(__nv_bfloat16, __nv_bfloat16);
     else return IK_BAD_ARGUMENT;

@@ -10,7 +10,9 @@
 // (cap 0 = none), value heads of another size than the key heads (hdv), values that are the leading hdv columns of the
 // key rows themselves (v_pages = k_pages with ldv = hd: a latent that serves as key and value), and a sink: one more
 // key of score 0 that carries no value, so that the weights are exp(s_j) / (1 + sum exp(s_j)).  Under a window the first
-// `keep` keys of the sequence may stay visible to every later query.
+// `keep` keys of the sequence may stay visible to every later query.  With key_scales (scales[page][kv head][position in page])
+// every score is multiplied by its key's number, for keys that are stored as projected because they are the values too and whose
+// norm is a factor.  With slopes [nh] a score loses slope * (i - j), behind the cap.
 #include <math.h>
 #define IK_FAMILY 4
 #include "common.cuh"
@@ -25,7 +27,8 @@ __global__ void __launch_bounds__(TILE)
 attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pages, const TC* __restrict__ v_pages,
                       TO* __restrict__ out, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                       const int* __restrict__ table, int table_stride, int nh, int nkv, int hd, int hdv, int ldv, float scale,
-                      float softcap, int window, int keep, int sink, const float* __restrict__ sink_v, int page_size, int n_pages, int* status) {
+                      float softcap, int window, int keep, int sink, const float* __restrict__ sink_v, const float* __restrict__ key_scales,
+                      const float* __restrict__ slopes, int page_size, int n_pages, int* status) {
     ik_pdl_wait();
     ik_pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smem[];
@@ -68,7 +71,9 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pages, 
             float dot = 0.f;
             for (int i = 0; i < hd; i++) dot = fmaf(qs[i], ik_ld(kr, i), dot);
             s = dot * scale;
+            if (key_scales) s *= key_scales[off];
             if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+            if (slopes) s = fmaf(-slopes[h], (float)(pos - j), s);
         }
         row[tid] = off;
         const float tile_max = ik_block_max<TILE>(s, red);
@@ -108,7 +113,8 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pages, 
 IK_EXPORT int ik_attention_simt(const void* q, int q_dtype, const void* k_pages, const void* v_pages, int cache_dtype,
                                 void* out, int out_dtype, const int* token_seq, const int* token_pos, const int* table,
                                 int table_stride, int T, int nh, int nkv, int hd, int hdv, int ldv, float scale, float softcap, int window, int keep,
-                                int sink, const float* sink_v, int page_size, int n_pages, int* status, cudaStream_t stream) {
+                                int sink, const float* sink_v, const float* key_scales, const float* slopes, int page_size, int n_pages, int* status,
+                                cudaStream_t stream) {
     if (ldv < hdv) return IK_BAD_ARGUMENT;
     if (T < 0 || nh <= 0 || nkv <= 0 || nh % nkv || hd <= 0 || hdv <= 0 || hdv > TILE * MAX_R || page_size <= 0 || softcap < 0.f || keep < 0) return IK_BAD_ARGUMENT;
     if (q_dtype != out_dtype) return IK_BAD_ARGUMENT;
@@ -117,7 +123,7 @@ IK_EXPORT int ik_attention_simt(const void* q, int q_dtype, const void* k_pages,
     const size_t smem = (size_t)(hd + TILE + 32) * sizeof(float) + TILE * sizeof(size_t);
 #define IK_ATT(TQ, TC)                                                                                                \
     IK_RETURN_IF_ERROR(ik_launch(attention_simt_kernel<TQ, TC, TQ>, grid, TILE, smem, stream, (const TQ*)q, (const TC*)k_pages, (const TC*)v_pages, \
-        (TQ*)out, token_seq, token_pos, table, table_stride, nh, nkv, hd, hdv, ldv, scale, softcap, window, keep, sink, sink_v, page_size, n_pages, status))
+        (TQ*)out, token_seq, token_pos, table, table_stride, nh, nkv, hd, hdv, ldv, scale, softcap, window, keep, sink, sink_v, key_scales, slopes, page_size, n_pages, status))
     if (q_dtype == IK_F32 && cache_dtype == IK_F32) IK_ATT(float, float);
     else if (q_dtype == IK_BF16 && cache_dtype == IK_BF16) IK_ATT(__nv_bfloat16, __nv_bfloat16);
     else if (q_dtype == IK_F32 && cache_dtype == IK_BF16) IK_ATT(float, __nv_bfloat16);

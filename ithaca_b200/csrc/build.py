@@ -30,7 +30,7 @@ _COMMON_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "-Xcom
                  "--expt-relaxed-constexpr"]
 
 # The always-needed kernels.  Specialised modules are listed in SPECIALISED.
-CORE_SOURCES = ["elementwise.cu", "layernorm.cu", "short_conv.cu", "recurrent.cu", "delta.cu", "row_decay.cu", "ssd.cu", "ssd_tcgen05.cu", "hyper.cu", "latent.cu", "attention_extras.cu", "moe.cu", "gemm_simt.cu", "gemm_mma.cu", "gemm_tcgen05.cu",
+CORE_SOURCES = ["elementwise.cu", "layernorm.cu", "dynamic_tanh.cu", "short_conv.cu", "recurrent.cu", "delta.cu", "row_decay.cu", "ssd.cu", "ssd_tcgen05.cu", "hyper.cu", "latent.cu", "attention_extras.cu", "moe.cu", "gemm_simt.cu", "gemm_mma.cu", "gemm_tcgen05.cu",
                 "attention_simt.cu", "sampling.cu"]
 
 _lock = threading.Lock()
@@ -155,6 +155,16 @@ def core() -> ctypes.CDLL:
 ATTENTION_HEAD_SIZES = (16, 32, 48, 64, 128)     # the sizes the tests and the benchmark use; others compile on demand
 
 
+# (head size, distance bias, rows that are keys and values): the modules of that kind built ahead of time
+ATTENTION_OPTION_MODULES = ((64, True, True), (128, True, True))
+
+
+def attention_module(head_dim: int, slopes: bool = False, one_row: bool = False) -> tuple:
+    """Name, sources and defines of the attention module of a head size and its options."""
+    defines = [f"IK_HD={head_dim}"] + (["IK_SLOPES=1"] if slopes else []) + (["IK_ONE_ROW=1"] if one_row else [])
+    return f"ithaca_attn{'_slopes' if slopes else ''}{'_onerow' if one_row else ''}_hd{head_dim}", ["attention_bf16.cu"], defines
+
+
 PAIRS_SOURCE = "gemm_tcgen05_mc.cu"        # the pair mode of the tcgen05 product: a library of its own, optional
 
 
@@ -171,6 +181,8 @@ def build_all() -> None:
     every usual head size, and the pair mode of the tcgen05 product where its source is there."""
     core()
     for hd in ATTENTION_HEAD_SIZES:
-        build_library(f"ithaca_attn_hd{hd}", ["attention_bf16.cu"], defines=[f"IK_HD={hd}"])
+        build_library(*attention_module(hd))
+    for options in ATTENTION_OPTION_MODULES:
+        build_library(*attention_module(*options))
     if pairs_available():
         build_library("ithaca_gemm_pairs", [PAIRS_SOURCE], includes=["gemm_tcgen05.cu"])

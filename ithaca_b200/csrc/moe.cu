@@ -6,9 +6,11 @@
 //             score = 1 the sigmoid of every logit by itself.  Experts form `n_groups` equal groups of
 //             neighbours; a group counts by its best score, only experts of the `keep` best groups can be chosen
 //             (n_groups <= 1: all can), and the `top` best of them are.  The weights are the chosen experts' scores as
-//             they are, or divided by their sum (renorm).  Equal scores: the lower index wins.  A bias may join the
-//             logits (`bias` [E]), and the router may have one row more, whose sigmoid goes to `gate` [T] (the weight of an
-//             expert that every token uses).
+//             they are, or divided by their sum (renorm; `weight_eps` joins the sum), times `weight_scale`.  Equal scores: the
+//             lower index wins.  A bias may join the logits (`bias` [E]), and the router may have one row more, whose sigmoid
+//             goes to `gate` [T] (the weight of an expert that every token uses).  A correction (`correction` [E]) may be
+//             added to the scores for the choice alone: groups and experts are chosen by corrected scores, which can be
+//             negative, the weights are made of the plain ones.  With `two` a group counts by the sum of its two best.
 //   sort      a counting sort of the A = T * top assignments by expert: sorted[] lists assignment ids (t * top + k)
 //             expert by expert; tiles[] cuts every expert's run into row tiles of MOE_BM for the products.
 //   gemm      for every row tile, rows of X (chosen through `sorted`) times the tile's expert's matrix.  Mode 0:
@@ -33,11 +35,22 @@ namespace {
 constexpr int MOE_BM = 64, MOE_BN = 64, MOE_BK = 16, MOE_TM = 4, MOE_TN = 4;
 
 // ------------------------------------------------------------------------------------------ route
-// One warp routes one token.  sc [E]: the token's router logits on entry (any memory the warp may write), its scores
-// with the taken ones marked on exit; gb [n_groups]: scratch.
-__device__ __forceinline__ void route_token(float* sc, float* gb, int lane, int* __restrict__ chosen, float* __restrict__ weight,
-                                            int E, int top, int ng, int keep, int renorm, int score) {
-    if (score == 1) {                 // every expert's score is the sigmoid of its own logit
+// How a token's experts are chosen and weighted.
+struct Routing {
+    int top, n_groups, keep, two, renorm, score;
+    float weight_eps, weight_scale;
+    const float* correction;
+    __host__ __device__ int ng() const { return n_groups > 1 ? n_groups : 0; }
+    __host__ __device__ int words(int E) const { return E + ng() + (correction ? E : 0); }      // shared floats per token
+};
+
+// One warp routes one token.  sc [E]: the token's router logits on entry (any memory the warp may write); behind it
+// the groups' scores [ng] and, with a correction, the plain scores [E].
+__device__ __forceinline__ void route_token(float* sc, int lane, int* __restrict__ chosen, float* __restrict__ weight, int E, const Routing& R) {
+    const int ng = R.ng();
+    float* gb = sc + E;
+    float* plain = gb + ng;
+    if (R.score == 1) {                 // every expert's score is the sigmoid of its own logit
         for (int e = lane; e < E; e += 32) sc[e] = 1.0f / (1.0f + expf(-sc[e]));
     } else {
         float m = -INFINITY;
@@ -49,10 +62,12 @@ __device__ __forceinline__ void route_token(float* sc, float* gb, int lane, int*
         const float inv = 1.0f / sum;
         for (int e = lane; e < E; e += 32) sc[e] *= inv;
     }
+    if (R.correction)
+        for (int e = lane; e < E; e += 32) { const float s = sc[e]; plain[e] = s; sc[e] = s + R.correction[e]; }
     __syncwarp();
-    // warp-wide argmax over n values v(i) >= 0 (taken ones are marked -1); the lower index wins a tie
+    // warp-wide argmax over n values (taken and struck-out ones are marked -inf); the lower index wins a tie
     auto argmax = [&](const float* v, int n) -> int {
-        float bv = -2.f; int bi = 0x7fffffff;
+        float bv = -INFINITY; int bi = 0x7fffffff;
         for (int i = lane; i < n; i += 32) if (v[i] > bv) { bv = v[i]; bi = i; }
         for (int o = 16; o > 0; o >>= 1) {
             const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
@@ -64,36 +79,44 @@ __device__ __forceinline__ void route_token(float* sc, float* gb, int lane, int*
     if (ng) {
         const int per = E / ng;
         for (int g = lane; g < ng; g += 32) {
-            float b = -1.f;
-            for (int i = 0; i < per; i++) b = fmaxf(b, sc[g * per + i]);
-            gb[g] = b;
+            float b = -INFINITY, c = -INFINITY;            // the group's best and second best
+            for (int i = 0; i < per; i++) {
+                const float v = sc[g * per + i];
+                c = fmaxf(c, fminf(b, v));
+                b = fmaxf(b, v);
+            }
+            gb[g] = R.two && per > 1 ? b + c : b;
         }
         __syncwarp();
-        // groups that are kept are marked by -1; then the others' experts are struck out
-        for (int k = 0; k < keep; k++) {
+        // groups that are kept are marked by -inf; then the others' experts are struck out
+        for (int k = 0; k < R.keep; k++) {
             const int g = argmax(gb, ng);
-            if (lane == 0) gb[g] = -1.f;
+            if (lane == 0 && g < ng) gb[g] = -INFINITY;
             __syncwarp();
         }
-        for (int e = lane; e < E; e += 32) if (gb[e / per] != -1.f) sc[e] = -(sc[e] + 2.f);     // struck out: -(s + 2) <= -2
+        for (int e = lane; e < E; e += 32) if (gb[e / per] != -INFINITY) sc[e] = -INFINITY;
         __syncwarp();
     }
     float wsum = 0.f;
-    for (int k = 0; k < top; k++) {
-        const int e = argmax(sc, E);
-        const float s = sc[e];
+    for (int k = 0; k < R.top; k++) {
+        int e = argmax(sc, E);
+        if (e >= E) e = 0;                                 // only scores that are not numbers leave nothing to choose
+        const float s = R.correction ? plain[e] : sc[e];
         wsum += s;
         __syncwarp();
-        if (lane == 0) { chosen[k] = e; weight[k] = s; sc[e] = -1.f; }
+        if (lane == 0) { chosen[k] = e; weight[k] = s; sc[e] = -INFINITY; }
         __syncwarp();
     }
-    if (renorm && lane == 0) for (int k = 0; k < top; k++) weight[k] /= wsum;
+    if (lane == 0 && (R.renorm || R.weight_scale != 1.0f)) {
+        const float div = R.renorm ? wsum + R.weight_eps : 1.0f;
+        for (int k = 0; k < R.top; k++) weight[k] = weight[k] / div * R.weight_scale;
+    }
 }
 
-// From ready-made logits: one warp per token.  smem: scores [E] then group bests [n_groups] per warp.
+// From ready-made logits: one warp per token.  smem: R.words(E) floats per warp.
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ bias, int* __restrict__ chosen,
-                 float* __restrict__ weight, float* __restrict__ gate, int T, int E, int top, int n_groups, int keep, int renorm, int score) {
+                 float* __restrict__ weight, float* __restrict__ gate, int T, int E, Routing R) {
     ik_pdl_wait();
     IK_AFTER_WAIT(logits);
     ik_pdl_launch_dependents();
@@ -101,31 +124,30 @@ moe_route_kernel(const float* __restrict__ logits, int ldl, const float* __restr
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + warp;
     if (t >= T) return;
-    const int ng = n_groups > 1 ? n_groups : 0;
-    float* sc = sm + (size_t)warp * (E + ng);
+    float* sc = sm + (size_t)warp * R.words(E);
     for (int e = lane; e < E; e += 32) sc[e] = logits[(size_t)t * ldl + e] + (bias ? bias[e] : 0.f);
     if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-logits[(size_t)t * ldl + E]));
     __syncwarp();
-    route_token(sc, sc + E, lane, chosen + (size_t)t * top, weight + (size_t)t * top, E, top, ng, keep, renorm, score);
+    route_token(sc, lane, chosen + (size_t)t * R.top, weight + (size_t)t * R.top, E, R);
 }
 
 // The router's product and the routing in one kernel.  A block takes TOK tokens: their activations go to shared memory
 // as floats; warp w forms the logits of experts w, w + warps, ...: its lanes stride over K four elements at a time (a weight
 // row is read once per block, 512 bytes per warp and load), each lane keeps one partial sum per token, added over its k in
 // ascending order and then across the lanes by a fixed tree, so a logit depends on its token and expert alone.  Then a warp
-// routes each token.  Everything in float.  K a multiple of 4.  smem: x [TOK][K], logits [TOK][E + n_groups].
+// routes each token.  Everything in float.  K a multiple of 4.  smem: x [TOK][K], then R.words(E) floats a token.
 // Few tokens (decode): one token a block and 32 warps, so that a token's experts are spread over many warps.
 template <int TOK, int THREADS, typename TX>
 __global__ void __launch_bounds__(THREADS)
 moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, const float* __restrict__ bias, int* __restrict__ chosen,
-                  float* __restrict__ weight, float* __restrict__ gate, int T, int K, int E, int top, int n_groups, int keep, int renorm, int score, int ldx) {
+                  float* __restrict__ weight, float* __restrict__ gate, int T, int K, int E, Routing R, int ldx) {
     ik_pdl_wait();
     IK_AFTER_WAIT(x);
     ik_pdl_launch_dependents();
     extern __shared__ __align__(16) float sm[];
-    const int ng = n_groups > 1 ? n_groups : 0;
+    const int words = R.words(E);
     float* xs = sm;                                   // [TOK][K]
-    float* lg = sm + (size_t)TOK * K;                 // [TOK][E + ng]
+    float* lg = sm + (size_t)TOK * K;                 // [TOK][words]
     const int ER = E + (gate ? 1 : 0);                // rows of the router
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * TOK;
@@ -188,7 +210,7 @@ moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, const 
                 float v = acc[j][i];
                 for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
                 if (lane != 0) continue;
-                if (e < E) lg[i * (E + ng) + e] = bias ? v + bias[e] : v;
+                if (e < E) lg[i * words + e] = bias ? v + bias[e] : v;
                 else if (t0 + i < T) gate[t0 + i] = 1.0f / (1.0f + expf(-v));
             }
         }
@@ -197,8 +219,7 @@ moe_router_kernel(const TX* __restrict__ x, const float* __restrict__ wr, const 
     for (int i = warp; i < TOK; i += THREADS / 32) {
         const int t = t0 + i;
         if (t >= T) continue;
-        float* sc = lg + (size_t)i * (E + ng);
-        route_token(sc, sc + E, lane, chosen + (size_t)t * top, weight + (size_t)t * top, E, top, ng, keep, renorm, score);
+        route_token(lg + (size_t)i * words, lane, chosen + (size_t)t * R.top, weight + (size_t)t * R.top, E, R);
     }
 }
 
@@ -448,28 +469,31 @@ IK_EXPORT int ik_moe_tile_rows() { return MOE_BM; }
 
 // logits [T, E] (rows ldl apart; with `gate` one column more)
 IK_EXPORT int ik_moe_route(const float* logits, int ldl, const float* bias, int* chosen, float* weight, float* gate, int T, int E, int top,
-                           int n_groups, int keep, int renorm, int score, cudaStream_t stream) {
+                           int n_groups, int keep, int renorm, int score, const float* correction, int two, float weight_eps, float weight_scale,
+                           cudaStream_t stream) {
     if (T < 0 || E <= 0 || top <= 0 || top > E || ldl < E + (gate ? 1 : 0)) return IK_BAD_ARGUMENT;
     if (n_groups > 1 && (E % n_groups || keep <= 0 || keep > n_groups || top > keep * (E / n_groups))) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
-    const size_t smem = 4 * (size_t)(E + (n_groups > 1 ? n_groups : 0)) * sizeof(float);
+    const Routing R{top, n_groups, keep, two, renorm, score, weight_eps, weight_scale, correction};
+    const size_t smem = 4 * (size_t)R.words(E) * sizeof(float);
     if (smem > 48 * 1024) return IK_UNSUPPORTED;
-    IK_RETURN_IF_ERROR(ik_launch(moe_route_kernel, (T + 3) / 4, 128, smem, stream, logits, ldl, bias, chosen, weight, gate, T, E, top, n_groups, keep, renorm, score));
+    IK_RETURN_IF_ERROR(ik_launch(moe_route_kernel, (T + 3) / 4, 128, smem, stream, logits, ldl, bias, chosen, weight, gate, T, E, R));
     IK_LAUNCH_STATUS();
 }
 
 // x [T, K] (float or bfloat16, rows ldx apart), wr [E, K] float (with `gate` [E + 1, K]) -> chosen, weight [T, top], gate [T]
 IK_EXPORT int ik_moe_router(const void* x, int x_dtype, const float* wr, const float* bias, int* chosen, float* weight, float* gate, int T, int K, int E, int top,
-                            int n_groups, int keep, int renorm, int score, int ldx, cudaStream_t stream) {
+                            int n_groups, int keep, int renorm, int score, const float* correction, int two, float weight_eps, float weight_scale,
+                            int ldx, cudaStream_t stream) {
     if (T < 0 || E <= 0 || K <= 0 || top <= 0 || top > E || ldx < K) return IK_BAD_ARGUMENT;
     if (n_groups > 1 && (E % n_groups || keep <= 0 || keep > n_groups || top > keep * (E / n_groups))) return IK_BAD_ARGUMENT;
     if (K % 4 || ((uintptr_t)wr % 16)) return IK_UNSUPPORTED;
     if (T == 0) return IK_OK;
-    const int ng = n_groups > 1 ? n_groups : 0;
+    const Routing R{top, n_groups, keep, two, renorm, score, weight_eps, weight_scale, correction};
     // few tokens (decode): a block per token, so that the step's tokens spread over the SMs; else eight tokens a block,
     // or four where eight rows of activations would leave room for one block per SM only
     const int tok = T <= 64 ? 1 : K <= 2048 ? 8 : K <= 6144 ? 4 : 1;
-    const size_t smem = ((size_t)tok * K + (size_t)tok * (E + ng)) * sizeof(float);
+    const size_t smem = ((size_t)tok * K + (size_t)tok * R.words(E)) * sizeof(float);
     if (smem > 200 * 1024) return IK_UNSUPPORTED;
 #define IK_ROUTER(TOK, TX)                                                                                                 \
     {                                                                                                                      \
@@ -479,8 +503,8 @@ IK_EXPORT int ik_moe_router(const void* x, int x_dtype, const float* wr, const f
             cudaError_t e0 = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
             if (e0 != cudaSuccess) return (int)e0;                                                                         \
         }                                                                                                                  \
-        IK_RETURN_IF_ERROR(ik_launch(kern, (T + TOK - 1) / TOK, THREADS, smem, stream, (const TX*)x, wr, bias, chosen, weight, gate, T, K, E, top, \
-                                     n_groups, keep, renorm, score, ldx));                                                        \
+        IK_RETURN_IF_ERROR(ik_launch(kern, (T + TOK - 1) / TOK, THREADS, smem, stream, (const TX*)x, wr, bias, chosen, weight, gate, T, K, E, R, \
+                                     ldx));                                                                                      \
     }
     if (x_dtype == IK_F32) { if (tok == 1) IK_ROUTER(1, float) else if (tok == 4) IK_ROUTER(4, float) else IK_ROUTER(8, float) }
     else if (x_dtype == IK_BF16) { if (tok == 1) IK_ROUTER(1, __nv_bfloat16) else if (tok == 4) IK_ROUTER(4, __nv_bfloat16) else IK_ROUTER(8, __nv_bfloat16) }

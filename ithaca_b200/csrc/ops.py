@@ -85,7 +85,7 @@ _SIGNATURES = {
     "ik_rope_table": [_vp, _vp, _vp, _i, _i, _vp],
     "ik_gemm_qkv_rope_mma": [_vp, _vp, _i, _i, _i, _i, _i, _vp, _vp],
     "ik_gemm_qkv_rope_tcgen05": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp],
-    "ik_attention_simt": [_vp, _i, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _i, _i, _vp, _vp],
+    "ik_attention_simt": [_vp, _i, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _vp],
     "ik_gemm_simt_batched": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _u64, _u64, _u64, _vp],
     "ik_scale_add_norm": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _vp],
     "ik_plain_act": [_vp, _vp, _i, _u64, _i, _vp],
@@ -99,8 +99,8 @@ _SIGNATURES = {
     "ik_conv_rope_append": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i,
                             _i, _i, _i, _i, _i, _vp, _vp],
     "ik_moe_tile_rows": [],
-    "ik_moe_route": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
-    "ik_moe_router": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "ik_moe_route": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _f, _f, _vp],
+    "ik_moe_router": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _f, _f, _i, _vp],
     "ik_moe_sort": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "ik_moe_gemm": [_i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp],
     "ik_moe_combine": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
@@ -127,7 +127,7 @@ _SIGNATURES = {
     "ik_gated_group_norm": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _f, _vp],
     "ik_decay_attention": [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "ik_norm_rope_append": [_vp, _i, _i, _i, _i, _vp, _vp, _f, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _f, _i, _i, _i, _i,
-                            _i, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp],
+                            _i, _i, _i, _i, _i, _i, _i, _vp, _i, _f, _i, _vp, _vp, _vp],
     "ik_head_gate": [_vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _i, _vp],
     "ik_gated_rmsnorm": [_vp, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _f, _f, _vp],
     "ik_hyper_start": [_vp, _vp, _i, _i, _i, _vp],
@@ -138,7 +138,11 @@ _SIGNATURES = {
     "ik_rmsnorm_range": [_vp, _i, _vp, _vp, _i, _i, _i, _f, _vp],
     "ik_decay_rows": [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
     "ik_token_shift": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _u64, _i, _i, _i, _i, _i, _vp],
-    "ik_row_decay": [_i, _vp, _i, _i, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "ik_row_decay": [_i, _vp, _i, _i, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
+    "ik_lowrank_decay": [_vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _f, _vp],
+    "ik_dynamic_tanh": [_vp, _vp, _vp, _vp, _f, _vp, _i, _i, _i, _vp],
+    "ik_dynamic_tanh_embed": [_vp, _vp, _i, _vp, _vp, _f, _vp, _i, _i, _i, _f, _vp, _vp],
+    "ik_dynamic_tanh_add": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _f, _vp, _f, _vp, _vp, _f, _vp, _i, _i, _i, _vp],
 }
 
 _lib = None
@@ -627,11 +631,21 @@ def sink_values(sink, n_heads: int) -> Optional[torch.Tensor]:
     return sink
 
 
+def check_score_extras(key_scales: Optional[torch.Tensor], slopes: Optional[torch.Tensor], k_pages: torch.Tensor, n_heads: int) -> None:
+    if key_scales is not None and (key_scales.dtype != torch.float32 or key_scales.shape != k_pages.shape[:3] or not key_scales.is_contiguous()):
+        raise KernelError("attention: the key scales need one float32 number per place in the key pages")
+    if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != n_heads or not slopes.is_contiguous()):
+        raise KernelError("attention: the distance bias needs one float32 slope per head")
+
+
 def attention_simt(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, token_seq: torch.Tensor,
                    token_pos: torch.Tensor, table: torch.Tensor, n_heads: int, scale: float, window: int,
                    status: Optional[torch.Tensor], out: Optional[torch.Tensor] = None, softcap: float = 0.0, sink=False,
-                   values_in_keys: int = 0, keep: int = 0) -> torch.Tensor:
-    """``softcap``: scores become cap * tanh(score / cap) after the scale (0 = no cap).  The value pages may
+                   values_in_keys: int = 0, keep: int = 0, key_scales: Optional[torch.Tensor] = None,
+                   slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``key_scales`` [pages, kv heads, page size] float: every score is multiplied by its key's number.  ``slopes`` [n_heads] float:
+    a score loses slope * (distance of the key), behind the cap.
+    ``softcap``: scores become cap * tanh(score / cap) after the scale (0 = no cap).  The value pages may
     have a head size of their own; the output is then [T, n_heads * that size].  ``sink``: one more key of score 0
     that carries no value (the weights are exp(s_j) / (1 + sum exp(s_j))); a float32 tensor [n_heads] instead of True gives
     every head's sink a score of its own (not scaled).  ``values_in_keys`` = n > 0: a key row's
@@ -651,13 +665,14 @@ def attention_simt(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor
         hdv = ldv = v_pages.shape[3]
     if q.shape[1] != n_heads * hd or v_pages.shape[:3] != k_pages.shape[:3] or v_pages.dtype != k_pages.dtype:
         raise KernelError("attention: q or the value pages have the wrong shape")
+    check_score_extras(key_scales, slopes, k_pages, n_heads)
     if out is None:
         out = torch.empty((T, n_heads * hdv), dtype=q.dtype, device=q.device)
     _work(f"attention_simt {T}x{n_heads}", _nbytes(q, out))
     _check(lib().ik_attention_simt(_ptr(q), _code(q), _ptr(k_pages), _ptr(v_pages), _code(k_pages), _ptr(out),
                                    _code(out), _ptr(token_seq), _ptr(token_pos), _ptr(table), table.stride(0), T,
                                    n_heads, nkv, hd, hdv, ldv, scale, softcap, window, keep, sink_flag(sink), _ptr(sink_values(sink, n_heads)),
-                                   page_size, n_pages, _ptr(status), _stream()),
+                                   _ptr(key_scales), _ptr(slopes), page_size, n_pages, _ptr(status), _stream()),
            "attention_simt")
     return out
 
@@ -737,6 +752,7 @@ def conv_rope_append(qkv: torch.Tensor, conv_w: Optional[torch.Tensor], ring: Op
 
 
 MOE_SCORES = {"softmax": 0, "sigmoid": 1}
+MOE_GROUP_SCORES = {"best": 0, "best_two": 1}
 
 
 def _router_extras(T: int, E: int, bias: Optional[torch.Tensor], gate: Optional[torch.Tensor]) -> None:
@@ -748,9 +764,21 @@ def _router_extras(T: int, E: int, bias: Optional[torch.Tensor], gate: Optional[
         raise KernelError("moe router: the bias needs one number per expert, the gate one per token")
 
 
+def _choice_args(E: int, correction: Optional[torch.Tensor], group_score: str, weight_eps: float, weight_scale: float):
+    if correction is not None:
+        _need(correction, "correction", torch.float32)
+        if correction.numel() != E:
+            raise KernelError("moe router: the correction needs one number per expert")
+    return (_ptr(correction), MOE_GROUP_SCORES[group_score], weight_eps, weight_scale)
+
+
 def moe_route(logits: torch.Tensor, top: int, n_groups: int = 0, keep: int = 0, renorm: bool = False, score: str = "softmax",
-              bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
-    """Scores over the experts (``score``: the softmax over all logits, or the sigmoid of each by itself) and the ``top`` best among the ``keep`` best of ``n_groups`` groups of
+              bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None,
+              group_score: str = "best", weight_eps: float = 0.0, weight_scale: float = 1.0):
+    """``correction`` [E] float is added to the scores for the choice of groups and experts, not for the weights.  A group counts
+    by its ``best`` score or by the sum of its ``best_two``.  ``weight_eps`` joins the sum that ``renorm`` divides by; the weights
+    are multiplied by ``weight_scale``.
+    Scores over the experts (``score``: the softmax over all logits, or the sigmoid of each by itself) and the ``top`` best among the ``keep`` best of ``n_groups`` groups of
     neighbours (0 groups: among all).  ``bias`` [E] float is added to the logits.  ``gate`` [T] float: the logits have one
     column more, whose sigmoid is written there.  Returns (chosen int32 [T, top], weights float [T, top])."""
     _need(logits, "logits", torch.float32)
@@ -761,12 +789,13 @@ def moe_route(logits: torch.Tensor, top: int, n_groups: int = 0, keep: int = 0, 
     weight = torch.empty((T, top), dtype=torch.float32, device=logits.device)
     _work(f"moe_route {T}x{E}", _nbytes(logits, chosen, weight))
     _check(lib().ik_moe_route(_ptr(logits), logits.shape[1], _ptr(bias), _ptr(chosen), _ptr(weight), _ptr(gate), T, E, top, n_groups, keep, 1 if renorm else 0,
-                              MOE_SCORES[score], _stream()), "moe_route")
+                              MOE_SCORES[score], *_choice_args(E, correction, group_score, weight_eps, weight_scale), _stream()), "moe_route")
     return chosen, weight
 
 
 def moe_router(x: torch.Tensor, router: torch.Tensor, top: int, n_groups: int = 0, keep: int = 0, renorm: bool = False,
-               score: str = "softmax", bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
+               score: str = "softmax", bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+               correction: Optional[torch.Tensor] = None, group_score: str = "best", weight_eps: float = 0.0, weight_scale: float = 1.0):
     """The router's logits ``x router^T`` (float products and sums, whatever type ``x`` has) and the routing of
     ``moe_route``, in one kernel.  Returns (chosen int32 [T, top], weights float [T, top]), or None when the kernel does
     not take these sizes (the caller forms the logits with a product and routes them).  ``bias`` [E] float is added to the
@@ -782,7 +811,7 @@ def moe_router(x: torch.Tensor, router: torch.Tensor, top: int, n_groups: int = 
     weight = torch.empty((T, top), dtype=torch.float32, device=x.device)
     _work(f"moe_router {T}x{E}x{K}", T * K * x.element_size() + E * K * 4 + 8 * T * top, 2 * T * E * K)
     st = lib().ik_moe_router(_ptr(x), _code(x), _ptr(router), _ptr(bias), _ptr(chosen), _ptr(weight), _ptr(gate), T, K, E, top, n_groups, keep,
-                             1 if renorm else 0, MOE_SCORES[score], x.stride(0), _stream())
+                             1 if renorm else 0, MOE_SCORES[score], *_choice_args(E, correction, group_score, weight_eps, weight_scale), x.stride(0), _stream())
     if st == -2:
         return None
     _check(st, "moe_router")
@@ -1162,8 +1191,12 @@ def norm_rope_append(p: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w: O
                      eps: float, q_out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, token_seq: torch.Tensor,
                      token_pos: torch.Tensor, table: torch.Tensor, inv_freq: Optional[torch.Tensor], magnitude: float,
                      n_heads: int, rotary_dim: int, pairing: int, write_cache: bool, status: Optional[torch.Tensor],
-                     per_head: bool = False, bias: Optional[torch.Tensor] = None, v_norm: bool = False) -> None:
-    """``bias``: a float vector over ``p``'s columns, added to q, k and v as they are read.  ``v_norm``: every value head is
+                     per_head: bool = False, bias: Optional[torch.Tensor] = None, v_norm: bool = False, unit: bool = False,
+                     q_temp=None, key_scales: Optional[torch.Tensor] = None) -> None:
+    """``unit``: every q and k head is divided by its own root mean square, without a weight.  ``q_temp`` = (coef, every): q is
+    multiplied by 1 + coef ln(floor((pos + 1) / every) + 1).  ``key_scales`` [pages, kv heads, page size] float (with ``unit``):
+    the keys are stored as projected, for they are the values too (``v_pages`` None), and 1 / their root mean square goes there.
+    ``bias``: a float vector over ``p``'s columns, added to q, k and v as they are read.  ``v_norm``: every value head is
     divided by the root mean square of its own values (``eps`` inside the root) before it is stored.
     RMS norm of q and of k over their whole projections (``q_w``, ``k_w``: weights of that size; None = no norm;
     ``per_head``: every head over its own values, with a weight of one head's size that the heads share),
@@ -1172,11 +1205,17 @@ def norm_rope_append(p: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w: O
     _need(p, "p", torch.float32, contiguous=False)
     _need(q_out, "q_out")
     _need(k_pages, "k_pages")
-    _need(v_pages, "v_pages")
     _need(table, "table", torch.int32)
     n_pages, nkv, page_size, hd = k_pages.shape
+    if key_scales is not None:
+        if not unit or v_pages is not None:
+            raise KernelError("norm_rope_append: key scales go with the unit norm and without value pages")
+        check_score_extras(key_scales, None, k_pages, n_heads)
+        v_pages, v_off = k_pages, k_off                       # nothing is stored there; the sizes below hold
+    _need(v_pages, "v_pages")
     hdv = v_pages.shape[3]
     T = p.shape[0]
+    coef, every = q_temp if q_temp is not None else (0.0, 0)
     if p.stride(1) != 1 or q_out.shape != (T, n_heads * hd) or v_pages.shape[:3] != k_pages.shape[:3] or v_pages.dtype != k_pages.dtype \
             or max(q_off + n_heads * hd, k_off + nkv * hd, v_off + nkv * hdv) > p.shape[1] \
             or (q_w is not None and q_w.numel() != (hd if per_head else n_heads * hd)) \
@@ -1187,8 +1226,8 @@ def norm_rope_append(p: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w: O
     _check(lib().ik_norm_rope_append(_ptr(p), p.stride(0), q_off, k_off, v_off, _ptr(q_w), _ptr(k_w), eps, _ptr(q_out), _code(q_out),
                                      _ptr(k_pages), _ptr(v_pages), _code(k_pages), _ptr(token_seq), _ptr(token_pos), _ptr(table),
                                      table.stride(0), _ptr(inv_freq), magnitude, T, n_heads, nkv, hd, hdv, rotary_dim, pairing,
-                                     page_size, n_pages, 1 if write_cache else 0, 1 if per_head else 0, _ptr(bias), 1 if v_norm else 0, _ptr(status),
-                                     _stream()), "norm_rope_append")
+                                     page_size, n_pages, 1 if write_cache else 0, 2 if unit else 1 if per_head else 0, _ptr(bias), 1 if v_norm else 0,
+                                     float(coef), int(every), _ptr(key_scales), _ptr(status), _stream()), "norm_rope_append")
 
 
 def head_gate(att: torch.Tensor, p: Optional[torch.Tensor], g_off: int, out: torch.Tensor, n_heads: int, mult: float = 1.0,
@@ -1542,6 +1581,20 @@ def decay_rows(x: torch.Tensor, bias: Optional[torch.Tensor], form: str, A_log: 
     return out
 
 
+def lowrank_decay(p: torch.Tensor, off: int, w: torch.Tensor, bias: Optional[torch.Tensor], power: float) -> torch.Tensor:
+    """sigmoid(z)^power [T, C] with z = p[:, off : off + rank] w + bias: decays whose logits are a projection of a low-rank factor
+    that lies in columns of the float matrix ``p``; ``w`` float [rank, C]."""
+    _need(p, "p", torch.float32, contiguous=False)
+    _need(w, "w", torch.float32)
+    T, (rank, C) = p.shape[0], w.shape
+    if p.stride(1) != 1 or off + rank > p.shape[1] or (bias is not None and (bias.numel() != C or bias.dtype != torch.float32)):
+        raise KernelError("lowrank_decay: the sizes do not fit together")
+    out = torch.empty((T, C), dtype=torch.float32, device=p.device)
+    _work(f"lowrank_decay {T}x{rank}x{C}", 4 * (T * (rank + C) + rank * C), 2 * T * rank * C)
+    _check(lib().ik_lowrank_decay(_ptr(p), p.stride(0), off, rank, _ptr(w), _ptr(bias), _ptr(out), T, C, power, _stream()), "lowrank_decay")
+    return out
+
+
 def token_shift(x: torch.Tensor, mu: torch.Tensor, ring: torch.Tensor, ctx) -> torch.Tensor:
     """[n_mix, T, d]: x + (x' - x) * mu[m] with x' the input one position earlier in the same sequence (zeros at position
     0; across steps from ``ring`` [slots, 2, d] float, which then receives every sequence's last input)."""
@@ -1560,13 +1613,13 @@ def token_shift(x: torch.Tensor, mu: torch.Tensor, ring: torch.Tensor, ctx) -> t
     return out
 
 
-ROW_RULES = {"delta": 0, "bonus": 1}
+ROW_RULES = {"delta": 0, "bonus": 1, "plain": 2}
 
 
 def row_decay(rule: str, u: torch.Tensor, x1_off: int, k_off: int, v_off: int, dec: torch.Tensor, beta: Optional[torch.Tensor],
-              bonus: Optional[torch.Tensor], state: torch.Tensor, ctx, n_heads: int, n_qk_heads: int, dk: int, dv: int) -> torch.Tensor:
+              bonus: Optional[torch.Tensor], state: torch.Tensor, ctx, n_heads: int, n_qk_heads: int, dk: int, dv: int, scale: float = 1.0) -> torch.Tensor:
     """A matrix state per head with a decay per key channel.  ``delta``: S <- diag(a) S; u = beta (v - S^T k); S <- S + k u^T;
-    o = S^T q.  ``bonus``: o = (S + diag(bonus) k v^T)^T r; S <- diag(w) S + k v^T.  q (or r), k and v are column ranges of
+    o = S^T q.  ``bonus``: o = (S + diag(bonus) k v^T)^T r; S <- diag(w) S + k v^T.  ``plain``: S <- diag(a) S + k v^T; o = scale S^T q.  q (or r), k and v are column ranges of
     the float matrix ``u``; ``dec`` [T, heads * dk]; ``beta`` [T, heads] (rows may lie further apart); ``bonus`` [heads * dk]; ``state`` [slots, 2, heads,
     dv, dk] float.  Returns [T, heads * dv] float."""
     _need(u, "u", torch.float32, contiguous=False)
@@ -1584,7 +1637,7 @@ def row_decay(rule: str, u: torch.Tensor, x1_off: int, k_off: int, v_off: int, d
     _work(f"row_decay {rule} {T}x{H}x{dk}x{dv}", 2 * n_state + T * (2 * G * dk + H * dk + 2 * H * dv) * 4, 6 * T * H * dk * dv)
     st = lib().ik_row_decay(ROW_RULES[rule], _ptr(u), u.stride(0), x1_off, k_off, v_off, _ptr(dec), _ptr(beta), beta.stride(0) if beta is not None else 0, _ptr(bonus), _ptr(state),
                             _ptr(ctx.slots), _ptr(ctx.cu_seqlens), _ptr(ctx.kv_lens), _ptr(out), T, ctx.n_seqs, H, G, dk, dv,
-                            1 if ctx.is_decode else 0, _stream())
+                            1 if ctx.is_decode else 0, scale, _stream())
     _check(st, "row_decay")
     return out
 
@@ -1689,3 +1742,76 @@ def gated_group_norm(x: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, gro
     _check(lib().ik_gated_group_norm(_ptr(x), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), _code(out), T, groups, d // groups, eps, _stream()),
            "gated_group_norm")
     return out
+
+
+# ---------------------------------------------------------------------------------------------
+# The norm without statistics, tanh(alpha x) * w + b.  A norm is handed over as (w, b, alpha).
+def _dyt(norm, d: int):
+    w, b, alpha = norm
+    _need(w, "weight", torch.float32)
+    _need(b, "bias", torch.float32)
+    if w.numel() != d or b.numel() != d:
+        raise KernelError("dynamic_tanh: weight and bias need one number per column")
+    return _ptr(w), _ptr(b), float(alpha)
+
+
+def dynamic_tanh(x: torch.Tensor, norm, out_dtype: torch.dtype, rows_in: Optional[torch.Tensor] = None) -> torch.Tensor:
+    _need(x, "x", torch.float32)
+    d = x.shape[-1]
+    rows = x.numel() // d if rows_in is None else rows_in.numel()
+    if rows_in is not None:
+        _need(rows_in, "rows_in", torch.int32)
+    out = torch.empty((rows, d), dtype=out_dtype, device=x.device)
+    _work(f"dynamic_tanh {rows}x{d}", rows * d * (4 + out.element_size()))
+    _check(lib().ik_dynamic_tanh(_ptr(x), _ptr(rows_in), *_dyt(norm, d), _ptr(out), _code(out), rows, d, _stream()), "dynamic_tanh")
+    return out
+
+
+def dynamic_tanh_embed(ids: torch.Tensor, table: torch.Tensor, norm, scale: float = 1.0, status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """norm(table[ids] * scale) in float."""
+    _need(ids, "ids", torch.int32)
+    _need(table, "table")
+    T, (V, d) = ids.numel(), table.shape
+    out = torch.empty((T, d), dtype=torch.float32, device=ids.device)
+    _work(f"dynamic_tanh embed {T}x{d}", T * d * (table.element_size() + 4))
+    _check(lib().ik_dynamic_tanh_embed(_ptr(ids), _ptr(table), _code(table), *_dyt(norm, d), _ptr(out), T, d, V, scale, _ptr(status), _stream()),
+           "dynamic_tanh_embed")
+    return out
+
+
+class ExpertSum:
+    """What ``moe_combine`` adds up, not yet added up: its arguments, for a kernel that takes the sum as it goes."""
+    __slots__ = ("parts", "weight", "row_of", "unweighted", "extra", "extra_weight")
+
+    def __init__(self, parts, weight, row_of=None, unweighted=False, extra=None, extra_weight=None):
+        self.parts, self.weight, self.row_of, self.unweighted, self.extra, self.extra_weight = parts, weight, row_of, unweighted, extra, extra_weight
+
+
+def dynamic_tanh_add(y, norm, residual: torch.Tensor, mult: float = 1.0, next_norm=None, next_dtype: Optional[torch.dtype] = None):
+    """residual += mult * norm(y), ``y`` a float matrix or an ``ExpertSum``.  With ``next_norm`` also returns that norm of the new
+    residual in ``next_dtype``."""
+    _need(residual, "residual", torch.float32)
+    T, d = residual.shape
+    copy = torch.empty((T, d), dtype=next_dtype, device=residual.device) if next_norm is not None else None
+    nxt = _dyt(next_norm, d) if next_norm is not None else (0, 0, 0.0)
+    cargs = (_ptr(copy), _code(copy) if copy is not None else F32)
+    if isinstance(y, ExpertSum):
+        top = y.weight.shape[1]
+        _need(y.parts, "parts", torch.float32)
+        _need(y.weight, "weight", torch.float32)
+        if y.weight.shape[0] != T or y.parts.shape[1] != d or (y.row_of is None and y.parts.shape[0] != T * top) \
+                or (y.extra is not None and (y.extra.shape != (T, d) or y.extra.dtype != torch.float32 or not y.extra.is_contiguous())) \
+                or (y.extra_weight is not None and (y.extra_weight.numel() != T or y.extra_weight.dtype != torch.float32)):
+            raise KernelError("dynamic_tanh_add: the sizes do not fit together")
+        _work(f"dynamic_tanh +sum +add {T}x{d}", T * d * (4 * top + 8) + _nbytes(y.extra, copy))
+        _check(lib().ik_dynamic_tanh_add(0, _ptr(y.parts), 0 if y.unweighted else _ptr(y.weight), _ptr(y.row_of), _ptr(y.extra),
+                                         _ptr(y.extra_weight), top, *_dyt(norm, d), _ptr(residual), mult, *nxt, *cargs, T, d, _stream()),
+               "dynamic_tanh_add")
+    else:
+        _need(y, "y", torch.float32)
+        if y.shape != residual.shape:
+            raise KernelError("dynamic_tanh_add: the sizes do not fit together")
+        _work(f"dynamic_tanh +add {T}x{d}", T * d * 12 + _nbytes(copy))
+        _check(lib().ik_dynamic_tanh_add(_ptr(y), 0, 0, 0, 0, 0, 0, *_dyt(norm, d), _ptr(residual), mult, *nxt, *cargs, T, d, _stream()),
+               "dynamic_tanh_add")
+    return copy

@@ -1,20 +1,23 @@
 // Recurrent mixers whose state is a matrix per head that decays row by row: every key channel has a decay of its own
-// per token.  Two rules share one kernel:
+// per token.  Three rules share one kernel:
 //
 //   rule 0, the delta rule with a decay per key channel:
 //       S <- diag(a) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q          (the read-out sees the token's own write)
 //   rule 1, token-shift time mixing with a bonus for the current token:
 //       o = (S + diag(bonus) k v^T)^T r;   S <- diag(w) S + k v^T                       (the read-out sees the state before the token)
+//   rule 2, gated linear attention:
+//       S <- diag(a) S + k v^T;   o = scale S^T q                                       (the read-out sees the token's own write)
 //
 // S is dk x dv per head, zero before a sequence's first token, float.  The layout of the work is the delta rule's
 // (delta.cu): a column of S is a recurrence of its own, L lanes of a warp share a column and keep 16 of its rows each in
 // registers, tokens pass through shared memory in tiles with the next tile on its way, sums run in the same order
 // whatever step or tile brings a token.  Rule 0 takes both sums from the decayed state, sd = a * S: A = sd^T k,
 // B = sd^T q, u = beta (v - A), S = sd + k u^T, o = B + (k . q) u.  Rule 1: B = S^T r, o = B + (sum_i bonus_i k_i r_i) v,
-// S = w * S + k v^T.  The state lies as [2, heads, dv, dk] per slot, the two copies by the parity of the position
+// S = w * S + k v^T.  Rule 2 forms S = a * S + k v^T and then S^T q.  The state lies as [2, heads, dv, dk] per slot, the two copies by the parity of the position
 // the state belongs to, as for the other recurrences.
 //
-// Around it: the decays themselves (two forms, float with the accurate exponential and logarithm), and the token shift (every token's input
+// Around it: the decays themselves (two forms of a ready projection and one that forms its projection from a low-rank factor,
+// float with the accurate exponential and logarithm), and the token shift (every token's input
 // mixed with the input one position earlier, which is part of the sequence's state).
 #include "common.cuh"
 
@@ -50,6 +53,50 @@ __global__ void decay_rows_kernel(const float* __restrict__ x, int ldx, const fl
             r = expf(-expf(z));
         }
         out[idx] = r;
+    }
+}
+
+// A decay whose logit is a projection of a low-rank factor that lies in columns of a wider product:
+//   z[t, c] = sum_r w[r, c] p[t, off + r] + bias[c],   out[t, c] = sigmoid(z)^power = exp(power * log sigmoid(z)).
+// w is stored [rank, C] (a factor's weights of neighbouring channels lie together).  A block takes TOK tokens and 256 channels; the
+// factors of its tokens go through shared memory, RC at a time, and a weight that is read serves all of its tokens.
+constexpr int LR_RC = 64;
+template <int TOK>
+__global__ void __launch_bounds__(256)
+lowrank_decay_kernel(const float* __restrict__ p, int ldp, int off, int rank, const float* __restrict__ w, const float* __restrict__ bias,
+                     float* __restrict__ out, int T, int C, float power) {
+    __shared__ float low[TOK][LR_RC];
+    ik_pdl_wait();
+    IK_AFTER_WAIT(p);
+    ik_pdl_launch_dependents();
+    const int t0 = blockIdx.x * TOK, c = blockIdx.y * 256 + threadIdx.x;
+    float acc[TOK];
+    #pragma unroll
+    for (int i = 0; i < TOK; i++) acc[i] = 0.f;
+    for (int r0 = 0; r0 < rank; r0 += LR_RC) {
+        const int n = min(LR_RC, rank - r0);
+        __syncthreads();
+        for (int f = threadIdx.x; f < TOK * n; f += 256) {
+            const int i = f / n, r = f - i * n;
+            low[i][r] = t0 + i < T ? p[(size_t)(t0 + i) * ldp + off + r0 + r] : 0.f;
+        }
+        __syncthreads();
+        if (c < C) {
+            #pragma unroll 4
+            for (int r = 0; r < n; r++) {
+                const float wv = w[(size_t)(r0 + r) * C + c];
+                #pragma unroll
+                for (int i = 0; i < TOK; i++) acc[i] = fmaf(wv, low[i][r], acc[i]);
+            }
+        }
+    }
+    if (c >= C) return;
+    const float b = bias ? bias[c] : 0.f;
+    #pragma unroll
+    for (int i = 0; i < TOK; i++) {
+        if (t0 + i >= T) break;
+        const float z = acc[i] + b, tail = log1pf(expf(-fabsf(z)));
+        out[(size_t)(t0 + i) * C + c] = expf(power * ((z < 0.f ? z : 0.f) - tail));
     }
 }
 
@@ -100,12 +147,13 @@ token_shift_ring_kernel(const TX* __restrict__ x, float* __restrict__ ring, cons
 // ------------------------------------------------------------------ the recurrence
 // x1 (q or r) and k come from the float matrix u (row stride ldu) at x1_off / k_off + (query/key head) * dk, v at
 // v_off + h * dv, the decays from dec [T, H * dk], the steps from beta (row stride ldb, one per head; rule 0), the bonus from bonus [H * dk] (rule 1).
+// `scale` multiplies the read-out of rule 2.
 template <int L, int R, int RULE>
 __global__ void __launch_bounds__(256, 4)
 row_decay_kernel(const float* __restrict__ u, int ldu, int x1_off, int k_off, int v_off, const float* __restrict__ dec,
                  const float* __restrict__ beta, int ldb, const float* __restrict__ bonus, float* __restrict__ state,
                  const int* __restrict__ slots, const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
-                 float* __restrict__ out, int H, int G, int dk, int dv, int TT, int W, int vec) {
+                 float* __restrict__ out, int H, int G, int dk, int dv, int TT, int W, int vec, float scale) {
     extern __shared__ __align__(16) float sm[];          // [2][TT][W]: x1, k, decay (16 L each), the block's v, step, c
     ik_pdl_wait();
     IK_AFTER_WAIT(u);
@@ -174,7 +222,7 @@ row_decay_kernel(const float* __restrict__ u, int ldu, int x1_off, int k_off, in
     for (int t0 = lo; t0 < hi; t0 += TT, buf ^= 1) {
         if (t0 + TT < hi) stage(t0 + TT, buf ^ 1);
         const int n_here = min(TT, hi - t0);
-        for (int tt = warp; tt < n_here; tt += nwarps) {        // c of the tile's tokens, lanes in index order, then the tree
+        for (int tt = warp; RULE != 2 && tt < n_here; tt += nwarps) {        // c of the tile's tokens, lanes in index order, then the tree
             float* x = sm + buf * per_tile + tt * W;
             float c = 0.f;
             for (int i = lane; i < LR; i += 32) {
@@ -185,7 +233,7 @@ row_decay_kernel(const float* __restrict__ u, int ldu, int x1_off, int k_off, in
             for (int o = 16; o > 0; o >>= 1) c += __shfl_xor_sync(0xffffffffu, c, o);
             if (lane == 0) x[3 * LR + CB + 1] = c;
         }
-        __syncthreads();
+        if (RULE != 2) __syncthreads();
         #pragma unroll 2
         for (int tt = 0; tt < n_here; tt++) {
             const float* x = sm + buf * per_tile + tt * W;
@@ -223,6 +271,25 @@ row_decay_kernel(const float* __restrict__ u, int ldu, int x1_off, int k_off, in
                     S[4 * f + 3] = fmaf(kk[f].w, un, S[4 * f + 3]);
                 }
                 if (part == 0 && live) out[(size_t)(t0 + tt) * H * dv + h * dv + col] = fmaf(c, un, B);
+            } else if (RULE == 2) {
+                float b0 = 0.f, b1 = 0.f, b2 = 0.f, b3 = 0.f;
+                #pragma unroll
+                for (int f = 0; f < NF; f++) {
+                    kk[f] = k4[f * L + part];
+                    const float4 qq = x4[f * L + part], dd = d4[f * L + part];
+                    S[4 * f] = fmaf(dd.x, S[4 * f], kk[f].x * v);
+                    S[4 * f + 1] = fmaf(dd.y, S[4 * f + 1], kk[f].y * v);
+                    S[4 * f + 2] = fmaf(dd.z, S[4 * f + 2], kk[f].z * v);
+                    S[4 * f + 3] = fmaf(dd.w, S[4 * f + 3], kk[f].w * v);
+                    b0 = fmaf(S[4 * f], qq.x, b0);
+                    b1 = fmaf(S[4 * f + 1], qq.y, b1);
+                    b2 = fmaf(S[4 * f + 2], qq.z, b2);
+                    b3 = fmaf(S[4 * f + 3], qq.w, b3);
+                }
+                float B = (b0 + b1) + (b2 + b3);
+                #pragma unroll
+                for (int o = 1; o < L; o <<= 1) B += __shfl_xor_sync(0xffffffffu, B, o);
+                if (part == 0 && live) out[(size_t)(t0 + tt) * H * dv + h * dv + col] = scale * B;
             } else {
                 float b0 = 0.f, b1 = 0.f, b2 = 0.f, b3 = 0.f;
                 #pragma unroll
@@ -259,7 +326,7 @@ row_decay_kernel(const float* __restrict__ u, int ldu, int x1_off, int k_off, in
 template <int L, int R, int RULE>
 cudaError_t row_decay_launch(dim3 grid, int threads, size_t smem, cudaStream_t stream, const float* u, int ldu, int x1_off, int k_off,
                              int v_off, const float* dec, const float* beta, int ldb, const float* bonus, float* state, const int* slots,
-                             const int* cu_seqlens, const int* kv_lens, float* out, int H, int G, int dk, int dv, int TT, int W, int vec) {
+                             const int* cu_seqlens, const int* kv_lens, float* out, int H, int G, int dk, int dv, int TT, int W, int vec, float scale) {
     static bool raised = false;
     if (smem > 48 * 1024 && !raised) {
         const cudaError_t e = cudaFuncSetAttribute(row_decay_kernel<L, R, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
@@ -267,7 +334,7 @@ cudaError_t row_decay_launch(dim3 grid, int threads, size_t smem, cudaStream_t s
         raised = true;
     }
     return ik_launch(row_decay_kernel<L, R, RULE>, grid, dim3(threads), smem, stream, u, ldu, x1_off, k_off, v_off, dec, beta, ldb, bonus, state,
-                     slots, cu_seqlens, kv_lens, out, H, G, dk, dv, TT, W, vec);
+                     slots, cu_seqlens, kv_lens, out, H, G, dk, dv, TT, W, vec, scale);
 }
 
 }  // namespace
@@ -279,6 +346,19 @@ IK_EXPORT int ik_decay_rows(const float* x, int ldx, const float* bias, const fl
     const size_t total = (size_t)T * C, want = (total + 255) / 256, cap = (size_t)ik_sm_count() * 32;
     IK_RETURN_IF_ERROR(ik_launch(decay_rows_kernel, (int)(want < cap ? want : cap), 256, 0, stream, x, ldx, bias, A_log, out, total, C,
                                  per_head > 0 ? per_head : 1, kind));
+    IK_LAUNCH_STATUS();
+}
+
+IK_EXPORT int ik_lowrank_decay(const float* p, int ldp, int off, int rank, const float* w, const float* bias, float* out, int T, int C,
+                               float power, cudaStream_t stream) {
+    if (T < 0 || C <= 0 || rank <= 0 || off < 0 || ldp < off + rank || !w) return IK_BAD_ARGUMENT;
+    if (T == 0) return IK_OK;
+    // a few tokens: one a block, so that they spread over the SMs; a prompt: sixteen share a weight that is read
+    if (T <= 64) {
+        IK_RETURN_IF_ERROR(ik_launch(lowrank_decay_kernel<1>, dim3(T, (C + 255) / 256), 256, 0, stream, p, ldp, off, rank, w, bias, out, T, C, power));
+    } else {
+        IK_RETURN_IF_ERROR(ik_launch(lowrank_decay_kernel<16>, dim3((T + 15) / 16, (C + 255) / 256), 256, 0, stream, p, ldp, off, rank, w, bias, out, T, C, power));
+    }
     IK_LAUNCH_STATUS();
 }
 
@@ -304,8 +384,8 @@ IK_EXPORT int ik_token_shift(const void* x, int dtype, const float* mu, float* r
 
 IK_EXPORT int ik_row_decay(int rule, const float* u, int ldu, int x1_off, int k_off, int v_off, const float* dec, const float* beta,
                            int ldb, const float* bonus, float* state, const int* slots, const int* cu_seqlens, const int* kv_lens, float* out,
-                           int T, int B, int H, int G, int dk, int dv, int one_token_each, cudaStream_t stream) {
-    if (T < 0 || B < 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || !state || !dec || rule < 0 || rule > 1) return IK_BAD_ARGUMENT;
+                           int T, int B, int H, int G, int dk, int dv, int one_token_each, float scale, cudaStream_t stream) {
+    if (T < 0 || B < 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || !state || !dec || rule < 0 || rule > 2) return IK_BAD_ARGUMENT;
     if ((rule == 0 && !beta) || (rule == 1 && !bonus)) return IK_BAD_ARGUMENT;
     if (T == 0 || B == 0) return IK_OK;
     if (dk > 32 * 16) return IK_UNSUPPORTED;         // 32 lanes of 16 rows
@@ -325,10 +405,13 @@ IK_EXPORT int ik_row_decay(int rule, const float* u, int ldu, int x1_off, int k_
     case LL:                                                                                                                         \
         if (rule == 0)                                                                                                               \
             IK_RETURN_IF_ERROR((row_decay_launch<LL, R, 0>(grid, 32 * nwarps, smem, stream, u, ldu, x1_off, k_off, v_off, dec, beta, ldb, bonus, \
-                                                           state, slots, cu_seqlens, kv_lens, out, H, G, dk, dv, TT, W, vec)));      \
-        else                                                                                                                         \
+                                                           state, slots, cu_seqlens, kv_lens, out, H, G, dk, dv, TT, W, vec, scale)));      \
+        else if (rule == 1)                                                                                                          \
             IK_RETURN_IF_ERROR((row_decay_launch<LL, R, 1>(grid, 32 * nwarps, smem, stream, u, ldu, x1_off, k_off, v_off, dec, beta, ldb, bonus, \
-                                                           state, slots, cu_seqlens, kv_lens, out, H, G, dk, dv, TT, W, vec)));      \
+                                                           state, slots, cu_seqlens, kv_lens, out, H, G, dk, dv, TT, W, vec, scale)));      \
+        else                                                                                                                         \
+            IK_RETURN_IF_ERROR((row_decay_launch<LL, R, 2>(grid, 32 * nwarps, smem, stream, u, ldu, x1_off, k_off, v_off, dec, beta, ldb, bonus, \
+                                                           state, slots, cu_seqlens, kv_lens, out, H, G, dk, dv, TT, W, vec, scale)));      \
         break
     switch (L) {
         IK_RD(1);

@@ -72,6 +72,11 @@ class DecoderModel:
             for name in shared:
                 tensors[name] = self.embedding.table                        # one copy on the device for both
         self.head = HEADS.get(spec.head.kind)(spec.head, tensors, runtime)
+        # the norm that reads the stream behind each run: a block that takes it may form it at its own end
+        self.following = [None] * len(spec.schedule)
+        for n, e in enumerate(spec.schedule[1:]):
+            if not e.adds_input and hasattr(self.layers[spec.schedule[n].layer], "entry_norm"):
+                self.following[n] = getattr(self.layers[e.layer], "entry_norm", None)
 
     @property
     def graph_safe(self) -> bool:
@@ -105,15 +110,19 @@ class DecoderModel:
         """Runs the step's tokens through every scheduled run; returns float32 logits
         [wanted rows, vocab], or None when no row is wanted."""
         h = self.embedding.forward(ctx.token_ids, ctx)
-        ctx.shared.pop("stream_copy", None)                    # nothing of an earlier pass over this description counts
+        for made in ("stream_copy", "stream_normed"):
+            ctx.shared.pop(made, None)                         # nothing of an earlier pass over this description counts
         h0 = h.clone() if any(e.adds_input for e in self.spec.schedule) else None
         if self.spec.streams > 0:
             h = ops.hyper_start(h, self.spec.streams)          # [T, streams, d]; the final norm reads the streams' sum
-        for e in self.spec.schedule:
+        for e, following in zip(self.spec.schedule, self.following):
             if e.adds_input:
                 ops.add_(h, h0)
                 ctx.shared.pop("stream_copy", None)            # a block's 16-bit copy of the stream is stale now
-            self.layers[e.layer].forward(h, ctx, cache.layer(e.cache), e.writes_cache)
+            if following is not None:
+                self.layers[e.layer].forward(h, ctx, cache.layer(e.cache), e.writes_cache, next_norm=following)
+            else:
+                self.layers[e.layer].forward(h, ctx, cache.layer(e.cache), e.writes_cache)
         if ctx.n_logit_rows == 0:
             return None
         xn = self.final_norm.forward(h, rows=ctx.logit_rows)

@@ -34,9 +34,15 @@ Options a spec may give (all off by default):
 * ``keep_first``: under a window the first ``keep_first`` keys of a sequence stay visible to every later query, at their true
   positions; the cache never releases their pages.
 * ``v_norm``: every value head is divided by its root mean square (``norm_eps`` inside the root, no weight) and cached so.
+* ``qk_norm: "unit"``: every q and k head is divided by its own root mean square, without a weight.
+* ``q_temp`` = (coef, every): q is multiplied by 1 + coef ln(floor((pos + 1) / every) + 1).
+* ``distance_slopes`` [n_heads]: a score loses slope * (pos - j), behind the cap.
+* ``values: "keys"`` (with ``qk_norm: "unit"``, no rotation, no ``v`` tensor): the values are the keys as projected, in front of their
+  norm.  The cache then holds ONE row per key, the projected one, and beside it 1 / its root mean square as a float: that
+  number multiplies the key's scores, so the kernels read a row once and use it as key and as value.
 * a position part whose cos and sin carry a constant factor (``magnitude``).
 
-With ``qk_norm``, ``head_gate``, ``sink``, ``v_norm``, an output bias or a magnitude (and with ``bias: "qkv"`` where the product's own
+With ``qk_norm``, ``q_temp``, ``head_gate``, ``sink``, ``v_norm``, an output bias or a magnitude (and with ``bias: "qkv"`` where the product's own
 epilogue cannot rotate and append) the mixer runs "wide": one product gives [q | k | v | g] in float, one kernel norms, rotates
 and appends, the attention kernel runs, and the gate kernel writes the output projection's operand.  A wide mixer can
 also serve as a branch of a composite (``parts/parallel.py``): ``branch_in()`` / ``branch_out()`` hand out its matrices
@@ -66,9 +72,10 @@ class Attention:
         d, nh, nkv, hd = spec["hidden_size"], spec["n_heads"], spec["n_kv_heads"], spec["head_dim"]
         w = spec.weights
         hdv = spec.get("v_head_dim") or hd
-        out = {w["q"]: TensorReq((nh * hd, d)), w["k"]: TensorReq((nkv * hd, d)),
-               w["v"]: TensorReq((nkv * hdv, d)), w["o"]: TensorReq((d, nh * hdv))}
-        if spec.get("qk_norm"):
+        out = {w["q"]: TensorReq((nh * hd, d)), w["k"]: TensorReq((nkv * hd, d)), w["o"]: TensorReq((d, nh * hdv))}
+        if spec.get("values") != "keys":
+            out[w["v"]] = TensorReq((nkv * hdv, d))
+        if spec.get("qk_norm") in ("head", "projection"):
             per_head = spec.get("qk_norm") == "head"
             out[w["q_norm"]] = TensorReq((hd if per_head else nh * hd,), init="ones")
             out[w["k_norm"]] = TensorReq((hd if per_head else nkv * hd,), init="ones")
@@ -116,9 +123,24 @@ class Attention:
         w = spec.weights
         wq, wk = tensors[w["q"]], tensors[w["k"]]
         qk_norm = spec.get("qk_norm")
-        if qk_norm not in (None, "projection", "head"):
-            raise ValueError(f"attention: qk_norm {qk_norm!r} is not supported (projection, head)")
-        self.norm_per_head = qk_norm == "head"
+        if qk_norm not in (None, "projection", "head", "unit"):
+            raise ValueError(f"attention: qk_norm {qk_norm!r} is not supported (projection, head, unit)")
+        self.norm_per_head, self.norm_unit = qk_norm == "head", qk_norm == "unit"
+        temp = spec.get("q_temp")
+        self.q_temp = (float(temp[0]), int(temp[1])) if temp is not None else None
+        if self.q_temp is not None and self.q_temp[1] <= 0:
+            raise ValueError(f"attention: q_temp needs a positive number of positions, found {self.q_temp[1]}")
+        if spec.get("values") not in (None, "keys"):
+            raise ValueError(f"attention: values {spec.get('values')!r} is not supported (keys)")
+        self.values_are_keys = spec.get("values") == "keys"
+        if self.values_are_keys and (not self.norm_unit or position is not None or spec.get("v_norm") or self.v_head_dim != self.head_dim):
+            raise ValueError("attention: values that are the keys go with the unit norm and without positions, a value norm or a size of their own")
+        slopes = spec.get("distance_slopes")
+        self.slopes = None
+        if slopes is not None:
+            if len(slopes) != self.n_heads:
+                raise ValueError(f"attention: {len(slopes)} distance slopes for {self.n_heads} heads")
+            self.slopes = torch.tensor([float(x) for x in slopes], dtype=torch.float32, device=runtime.device)
         self.head_gate = bool(spec.get("head_gate"))
         self.gate_wide = spec.get("head_gate") == "wide"
         self.sink = bool(spec.get("sink"))
@@ -130,11 +152,11 @@ class Attention:
         if spec.get("bias") not in (None, False, True, "qkv"):
             raise ValueError(f"attention: bias {spec.get('bias')!r} is not supported (true, qkv)")
         self.biased = bool(spec.get("bias"))
-        self.wide = bool(qk_norm or self.head_gate or self.sink or self.v_norm or (self.biased and spec.get("bias") != "qkv")
+        self.wide = bool(qk_norm or self.q_temp or self.head_gate or self.sink or self.v_norm or (self.biased and spec.get("bias") != "qkv")
                          or (position is not None and getattr(position, "magnitude", 1.0) != 1.0) or not standalone)
         self.norm_eps = float(spec.get("norm_eps") or 0.0)
-        self.q_norm_w = as_float32(tensors[w["q_norm"]], runtime) if qk_norm else None
-        self.k_norm_w = as_float32(tensors[w["k_norm"]], runtime) if qk_norm else None
+        self.q_norm_w = as_float32(tensors[w["q_norm"]], runtime) if qk_norm in ("head", "projection") else None
+        self.k_norm_w = as_float32(tensors[w["k_norm"]], runtime) if qk_norm in ("head", "projection") else None
         # bfloat16 path with the whole head rotated: the rows of the q and k weights are reordered so that the
         # two members of a rotary pair are neighbours, (i, i + hd/2) -> (2i, 2i + 1).  Scores do not change (q and k
         # are reordered alike, and the cache holds k in that order); the product's epilogue can then rotate a pair
@@ -156,16 +178,18 @@ class Attention:
             if self.biased:
                 bq, bk = bq.view(self.n_heads, -1)[:, order].reshape(-1), bk.view(self.n_kv_heads, -1)[:, order].reshape(-1)
             self.pairing = 1                                       # pairs are (2i, 2i + 1) from here on
-        self._in = [wq, wk, tensors[w["v"]]] + ([tensors[w["g"]]] if self.head_gate else [])
+        self._in = [wq, wk] + ([] if self.values_are_keys else [tensors[w["v"]]]) + ([tensors[w["g"]]] if self.head_gate else [])
         self._out = tensors[w["o"]]
         self.k_off = self.n_heads * self.head_dim
         self.v_off = self.k_off + self.n_kv_heads * self.head_dim
-        self.g_off = self.v_off + self.n_kv_heads * self.v_head_dim
+        self.g_off = self.v_off + (0 if self.values_are_keys else self.n_kv_heads * self.v_head_dim)
         self.n_mid = self.n_heads * self.v_head_dim
         self.n_in = self.g_off + ((self.n_mid if self.gate_wide else self.n_heads) if self.head_gate else 0)
         # the projections' biases as one vector over the columns of the wide product (the gate has none)
         self.in_bias = None
         self._out_bias = None
+        if self.biased and self.values_are_keys:
+            raise ValueError("attention: biases and values that are the keys do not go together")
         if self.biased:
             zeros = torch.zeros(self.n_in - self.g_off, dtype=torch.float32)
             self.in_bias = torch.cat([b.to(torch.float32).cpu() for b in (bq, bk, tensors[w["v_bias"]])] + [zeros]).to(runtime.device).contiguous()
@@ -204,9 +228,10 @@ class Attention:
         ops.norm_rope_append(p, 0, self.k_off, self.v_off, self.q_norm_w, self.k_norm_w, self.norm_eps, q, cache.k_pages,
                              cache.v_pages, ctx.token_seq, ctx.token_pos, table, pos.inv_freq if pos is not None else None,
                              getattr(pos, "magnitude", 1.0), self.n_heads, pos.rotary_dim if pos is not None else 0,
-                             self.pairing, writes_cache, rt.status, per_head=self.norm_per_head, bias=self.in_bias, v_norm=self.v_norm)
+                             self.pairing, writes_cache, rt.status, per_head=self.norm_per_head, bias=self.in_bias, v_norm=self.v_norm,
+                             unit=self.norm_unit, q_temp=self.q_temp, key_scales=cache.key_scales)
         return attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, sink=self.sink_arg,
-                      keep=self.keep_first)
+                      keep=self.keep_first, slopes=self.slopes)
 
     def core(self, p: torch.Tensor, mid: torch.Tensor, ctx, cache: LayerCache, writes_cache: bool = True, mult: float = 1.0) -> None:
         """``p`` [T, n_in] float: [q | k | v | g] (a column range of a wider matrix may be given); ``mid`` [T, n_mid] in the
@@ -216,7 +241,8 @@ class Attention:
 
     def cache_requests(self) -> List[object]:
         v = self.v_head_dim if self.v_head_dim != self.head_dim else None
-        out: List[object] = [KVRequest(self.n_kv_heads, self.head_dim, self.window, v, keep_first=self.keep_first)]
+        out: List[object] = [KVRequest(self.n_kv_heads, self.head_dim, self.window, v, values_in_keys=self.values_are_keys,
+                                       keep_first=self.keep_first, key_scales=self.values_are_keys)]
         if self.conv_taps > 1:
             out.append(StateRequest("conv_ring", (self.conv_taps, self.channels), "float32"))
         return out
@@ -263,22 +289,24 @@ class Attention:
             ops.rope_append(qkv, q, cache.k_pages, cache.v_pages, ctx.token_seq, ctx.token_pos, table,
                             pos.inv_freq if pos is not None else None, self.n_heads, self.n_kv_heads, self.head_dim,
                             pos.rotary_dim if pos is not None else 0, self.pairing, writes_cache, rt.status)
-        att = attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, keep=self.keep_first)
+        att = attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, keep=self.keep_first, slopes=self.slopes)
         self.o(att, out=residual, accumulate=accumulate)
 
 
 def attend(q: torch.Tensor, cache: LayerCache, ctx, table: torch.Tensor, n_heads: int, scale: float, window: int,
-           rt: Runtime, softcap: float = 0.0, sink=False, keep: int = 0) -> torch.Tensor:
+           rt: Runtime, softcap: float = 0.0, sink=False, keep: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Chooses the attention kernel: tensor-core kernels for bfloat16 when they take the
-    head sizes, else the CUDA-core kernel (always for float32)."""
-    if q.dtype == torch.bfloat16 and cache.v_pages.shape[3] == cache.k_pages.shape[3]:
+    head sizes, else the CUDA-core kernel (always for float32).  A cache entry without value pages (but with key scales) holds
+    rows that are keys and values."""
+    if q.dtype == torch.bfloat16 and (cache.v_pages is None or cache.v_pages.shape[3] == cache.k_pages.shape[3]):
         from ..csrc import attention_bf16
         out = attention_bf16.attend(q, cache.k_pages, cache.v_pages, ctx, table, n_heads, scale, window, rt.status,
-                                    softcap=softcap, sink=sink, keep=keep)
+                                    softcap=softcap, sink=sink, keep=keep, key_scales=cache.key_scales, slopes=slopes)
         if out is not None:
             return out
     return ops.attention_simt(q, cache.k_pages, cache.v_pages, ctx.token_seq, ctx.token_pos, table, n_heads, scale,
-                              window, rt.status, softcap=softcap, sink=sink, keep=keep)
+                              window, rt.status, softcap=softcap, sink=sink, keep=keep, key_scales=cache.key_scales, slopes=slopes,
+                              values_in_keys=cache.k_pages.shape[3] if cache.v_pages is None else 0)
 
 
 register_mixer("attention", Attention)

@@ -14,7 +14,9 @@ and both sublayers add into the float stream.  The feed-forward may be absent.
 ``sandwich``: a norm in front of and behind each sublayer, and a constant on what joins the
 stream: x += m * norm_out(mixer(norm(x))); x += m * norm_out'(feed_forward(norm'(x))).  The
 sublayer writes into a float32 buffer of its own (the stream is not what it adds to); the norm
-behind it scales and adds in one kernel.  The feed-forward may be absent.
+behind it scales and adds in one kernel.  The feed-forward may be absent.  A norm that can do so (``takes_sums``) forms the norm
+that reads the stream next in the same kernel, across the layer's end too (the model tells a run which norm follows it), and takes
+routed experts' results before they are added up.
 
 ``outnorm``: a norm behind each sublayer only: x += norm_out(mixer(x)); x += norm_out'(feed_forward(x)).  The
 sublayers read the stream itself.  On the 16-bit path their operand is a 16-bit copy of the stream, which the
@@ -154,6 +156,7 @@ class ParallelBlock:
 
 
 class SandwichBlock:
+    NORMED = "stream_normed"    # in StepContext.shared: (norm, its result for the stream as of the last add)
     NORMS = ("mixer", "mixer_out", "feed_forward", "feed_forward_out")
 
     @classmethod
@@ -199,13 +202,36 @@ class SandwichBlock:
     def cache_requests(self) -> List[object]:
         return list(self.mixer.cache_requests())
 
-    def forward(self, residual: torch.Tensor, ctx, cache: LayerCache, writes_cache: bool = True) -> None:
+    @property
+    def entry_norm(self):
+        """The norm that reads the stream when a run of this layer starts."""
+        return self.mixer_norm
+
+    def _add(self, norm, y, residual: torch.Tensor, reader=None):
+        """residual += mult * norm(y); where the kernel can, also what ``reader`` (a norm or None) makes of the new stream."""
+        if not getattr(norm, "takes_sums", False):
+            norm.add_into(y, residual, self.mult)
+            return None
+        return norm.add_into(y, residual, self.mult, next_norm=reader if type(reader) is type(norm) else None)
+
+    def forward(self, residual: torch.Tensor, ctx, cache: LayerCache, writes_cache: bool = True, next_norm=None) -> None:
+        """``next_norm``: the norm that reads the stream next, if this run's end may already form it."""
+        made = ctx.shared.pop(self.NORMED, None)
+        xn = made[1] if made is not None and made[0] is self.mixer_norm else self.mixer_norm.forward(residual)
         y = torch.empty_like(residual)
-        self.mixer.forward(self.mixer_norm.forward(residual), ctx, cache, y, writes_cache, accumulate=False)
-        self.mixer_out_norm.add_into(y, residual, self.mult)
-        if self.feed_forward is not None:
-            self.feed_forward.forward(self.ff_norm.forward(residual), ctx, y, accumulate=False)
-            self.ff_out_norm.add_into(y, residual, self.mult)
+        self.mixer.forward(xn, ctx, cache, y, writes_cache, accumulate=False)
+        has_ff = self.feed_forward is not None
+        xn = self._add(self.mixer_out_norm, y, residual, self.ff_norm if has_ff else next_norm)
+        if has_ff:
+            if xn is None:
+                xn = self.ff_norm.forward(residual)
+            if getattr(self.ff_out_norm, "takes_sums", False) and hasattr(self.feed_forward, "unsummed"):
+                y = self.feed_forward.unsummed(xn, ctx)
+            else:
+                self.feed_forward.forward(xn, ctx, y, accumulate=False)
+            xn = self._add(self.ff_out_norm, y, residual, next_norm)
+        if xn is not None:
+            ctx.shared[self.NORMED] = (next_norm, xn)
 
 
 class OutNormBlock:

@@ -2,6 +2,7 @@
 
 x[t, :] = E[id_t, :] * scale (src/model.cpp:1381-1383).  The reference clamps an id
 outside the vocabulary; here the step function rejects it before anything runs.
+With a norm of its own (``normed_embedding``, parameter ``norm``: the norm's record) the stream starts as norm(E[id] * scale).
 logits = W_out xn, where W_out is the embedding matrix when the model has no
 output matrix of its own (src/model.cpp:132, 1590-1592).  A head may scale its logits by a constant
 (``scale``) and cap them, cap * tanh(logit / cap) (``softcap``), both in float.
@@ -15,7 +16,7 @@ import torch
 from ..config.spec import PartSpec
 from ..csrc import ops
 from ..weights.loader import TensorReq
-from .base import Runtime, register_embedding, register_head, to_device
+from .base import NORMS, Runtime, register_embedding, register_head, to_device
 from .linear import Linear
 
 
@@ -33,6 +34,23 @@ class Embedding:
 
     def forward(self, ids: torch.Tensor, ctx=None) -> torch.Tensor:
         return ops.embed(ids, self.table, self.scale, self.runtime.status)
+
+
+class NormedEmbedding(Embedding):
+    @classmethod
+    def manifest(cls, spec: PartSpec) -> Dict[str, TensorReq]:
+        out = super().manifest(spec)
+        out.update(NORMS.get(spec["norm"].kind).manifest(spec["norm"]))
+        return out
+
+    def __init__(self, spec: PartSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
+        super().__init__(spec, tensors, runtime)
+        self.norm = NORMS.get(spec["norm"].kind)(spec["norm"], tensors, runtime)
+
+    def forward(self, ids: torch.Tensor, ctx=None) -> torch.Tensor:
+        if hasattr(self.norm, "embed"):
+            return self.norm.embed(ids, self.table, self.scale)
+        return self.norm.forward(super().forward(ids, ctx), out_dtype=torch.float32)
 
 
 class OutputHead:
@@ -54,4 +72,5 @@ class OutputHead:
 
 
 register_embedding("embedding", Embedding)
+register_embedding("normed_embedding", NormedEmbedding)
 register_head("lm_head", OutputHead)

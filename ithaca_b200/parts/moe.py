@@ -3,9 +3,10 @@
 Router: z = Wr x in float32 (x may be the activations' 16-bit rounding), scores = softmax(z)
 over all experts (``score: "sigmoid"``: the sigmoid of every logit by itself).  With the tensor ``router_bias`` [experts] a
 bias joins the logits.  Experts may form equal groups of neighbours: a group counts by its best
-score, and only experts of the ``group_keep`` best groups can be chosen.  The ``top`` best of
-them are; their weights are their scores (``renormalize``: divided by their sum; with softmax scores that is the softmax over
-the chosen experts' logits).  An expert is
+score, and only experts of the ``group_keep`` best groups can be chosen.  (``group_score: "best_two"``: by the sum of its two best.)  The ``top`` best of
+them are; with the tensor ``correction`` [experts] groups and experts are chosen by score + correction, while the weights stay those of
+the plain scores; their weights are their scores (``renormalize``: divided by their sum; with softmax scores that is the softmax over
+the chosen experts' logits; ``weight_eps`` joins that sum), times ``weight_scale``.  An expert is
 y = Wd (silu(Wg x) * (Wu x)); the layer's output is the weighted sum of the chosen experts'.
 
 ``expert: "plain"``: an expert is ungated, y = Wd act(Wu x) with ``activation`` ``relu2`` or ``gelu_tanh`` (no ``gate`` tensors).
@@ -67,6 +68,8 @@ class MoEFeedForward:
         w, n = spec.weights, spec.get("shared") or 0
         if "router_bias" in w:
             out[w["router_bias"]] = TensorReq((spec["n_experts"],))
+        if "correction" in w:
+            out[w["correction"]] = TensorReq((spec["n_experts"],), std=0.1)
         if n:
             out[w["shared_gate"]], out[w["shared_up"]], out[w["shared_down"]] = TensorReq((n, d)), TensorReq((n, d)), TensorReq((d, n))
             if "shared_weight" in w:
@@ -100,6 +103,11 @@ class MoEFeedForward:
         self.n_groups = int(spec.get("n_groups") or 0)
         self.group_keep = int(spec.get("group_keep") or 0)
         self.renormalize = bool(spec.get("renormalize", False))
+        self.weight_eps = float(spec.get("weight_eps") or 0.0)
+        self.weight_scale = float(spec.get("weight_scale", 1.0))
+        self.group_score = spec.get("group_score", "best")
+        if self.group_score not in ops.MOE_GROUP_SCORES:
+            raise ValueError(f"moe: group_score {self.group_score!r} is not supported ({', '.join(ops.MOE_GROUP_SCORES)})")
         if not 1 <= self.top <= self.n_experts:
             raise ValueError(f"moe: top must lie in 1..{self.n_experts}, found {self.top}")
         if self.n_groups > 1:
@@ -114,6 +122,7 @@ class MoEFeedForward:
         self.router = to_device(tensors[router], runtime).to(torch.float32).contiguous()
         w = spec.weights
         self.router_bias = as_float32(tensors[w["router_bias"]], runtime) if "router_bias" in w else None
+        self.correction = as_float32(tensors[w["correction"]], runtime) if "correction" in w else None
         # a gated expert for every token, and, as the router's last row, the projection behind its weight
         self.shared = int(spec.get("shared") or 0)
         self.shared_weighted = bool(self.shared) and "shared_weight" in w
@@ -147,9 +156,16 @@ class MoEFeedForward:
         return 256 if per >= 1024 else 128 if per > 64 else max(16, -(-per // 16) * 16)
 
     def forward(self, x: torch.Tensor, ctx, residual: torch.Tensor, accumulate: bool = True) -> None:
+        y = self.unsummed(x, ctx)
+        ops.moe_combine(y.parts, y.weight, out=residual, row_of=y.row_of, unweighted=y.unweighted, extra=y.extra, extra_weight=y.extra_weight,
+                        accumulate=accumulate)
+
+    def unsummed(self, x: torch.Tensor, ctx) -> "ops.ExpertSum":
+        """The layer's result as the experts' rows and what adds them up, for a caller whose next kernel does that."""
         rt = self.runtime
         sg = torch.empty((x.shape[0],), dtype=torch.float32, device=x.device) if self.shared_weighted else None
-        extras = {"bias": self.router_bias, "gate": sg}
+        extras = {"bias": self.router_bias, "gate": sg, "correction": self.correction, "group_score": self.group_score,
+                  "weight_eps": self.weight_eps, "weight_scale": self.weight_scale}
         routed = logits = None
         if self.router16 is not None:
             logits = gemm(x, self.router16, out_dtype=torch.float32)
@@ -185,7 +201,7 @@ class MoEFeedForward:
         if self.shared_expert is not None:
             every = torch.empty((x.shape[0], self.hidden), dtype=torch.float32, device=x.device)
             self.shared_expert.forward(x, ctx, every, accumulate=False)
-        ops.moe_combine(parts, weight, out=residual, row_of=row_of, unweighted=on_input, extra=every, extra_weight=sg, accumulate=accumulate)
+        return ops.ExpertSum(parts, weight, row_of, on_input, every, sg)
 
 
 register_feed_forward("moe", MoEFeedForward)

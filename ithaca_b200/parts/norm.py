@@ -6,6 +6,8 @@ deviations, in float32.  A norm may also stand behind a sublayer: ``add_into`` t
 ``mult * y`` to the residual stream in the same kernel.  The RMS norm may carry a second vector
 (``scale``, a per-channel "layer scale") that multiplies what it adds to the stream.  With ``scalar_weight`` the RMS
 norm's weight is ONE number for all coordinates (stored as a tensor without dimensions); the kernels get it spread out.
+Dynamic tanh: y = tanh(alpha x) * w + b with one alpha, no statistics.  Behind a sublayer it takes the experts' results
+unsummed (``takes_sums``) and forms the norm that reads the stream next (``next_norm``, of its own kind) in the same kernel.
 With ``unit_offset`` the stored weight is the distance from one: y = x / rms(x) * (1 + w), the sum formed in float at load."""
 from __future__ import annotations
 
@@ -72,5 +74,33 @@ class LayerNorm:
         ops.layernorm(x, self.weight, self.bias, self.eps, torch.float32, into=residual, mult=mult)
 
 
+class DynamicTanh:
+    takes_sums = True
+
+    @classmethod
+    def manifest(cls, spec: PartSpec) -> Dict[str, TensorReq]:
+        w = spec.weights
+        return {w["weight"]: TensorReq((spec["size"],), init="ones"), w["bias"]: TensorReq((spec["size"],)),
+                w["alpha"]: TensorReq((), init="ones")}
+
+    def __init__(self, spec: PartSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
+        w = spec.weights
+        self.args = (as_float32(tensors[w["weight"]], runtime), as_float32(tensors[w["bias"]], runtime), float(tensors[w["alpha"]]))
+        self.runtime = runtime
+
+    def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None,
+                out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        return ops.dynamic_tanh(x, self.args, out_dtype or self.runtime.act_dtype, rows_in=rows)
+
+    def embed(self, ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
+        """The norm of the rows ``ids`` of an embedding table, in float."""
+        return ops.dynamic_tanh_embed(ids, table, self.args, scale, self.runtime.status)
+
+    def add_into(self, x, residual: torch.Tensor, mult: float = 1.0, next_norm=None) -> Optional[torch.Tensor]:
+        """residual += mult * norm(x); returns ``next_norm`` (a DynamicTanh) of the new residual in the activation type."""
+        return ops.dynamic_tanh_add(x, self.args, residual, mult, next_norm.args if next_norm is not None else None, self.runtime.act_dtype)
+
+
+register_norm("dynamic_tanh", DynamicTanh)
 register_norm("rmsnorm", RMSNorm)
 register_norm("layernorm", LayerNorm)
