@@ -21,6 +21,11 @@
                                                                 attention that keeps the first keys; routed experts beside one that
                                                                 every token uses; a looped span of layers) beside a Tiralix of equal
                                                                 width, heads, active feed-forward and layer runs, in the same form
+    python bench.py --only vovalorn [--batch B]                 the Vovalorn decoder (dynamic tanh norms around both sublayers; gated linear
+                                                                attention; attention whose values are its keys, with a distance bias; routed
+                                                                experts beside one that every token uses; layers that run others' tensors)
+                                                                beside a Zomipel of equal width, heads, state, experts and layer runs, in the
+                                                                same form
     python bench.py --config 1b-unequal|13b-long                the other two workloads alone, through Engine.generate
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at the given batch with every
@@ -674,6 +679,43 @@ def zomipel_pair(size, vocab=32000):
     return zom, tiralix, len(runs)
 
 
+VOVALORN_SIZES = [
+    # name, width, heads, kv heads, head size, gla heads, key size, value size, experts, chosen, groups, kept, expert width, shared
+    # width, layers (a number: that layer's tensors once more)
+    ("2048 wide, 16 heads of 128, 16 gla heads of 64 x 128, 16 experts of 1024", 2048, 16, 4, 128, 16, 64, 128, 16, 4, 4, 2, 1024, 4096,
+     ("gla", "attention", "gla", 1, 2, "gla")),
+    ("4096 wide, 32 heads of 128, 32 gla heads of 64 x 128, 8 experts of 3584", 4096, 32, 8, 128, 32, 64, 128, 8, 2, 4, 2, 3584, 7168,
+     ("gla", "attention", "gla", 1, 2, "gla")),
+]
+
+
+def vovalorn_pair(size, vocab=32000):
+    """The Vovalorn configuration of a size and the Zomipel next to it: the same width, attention heads and head size, values and
+    state entries of the recurrent layers (two heads of 64 values by 64 states for one of 128 by 64), experts and layer runs, of
+    which as many use tensors again.  Zomipel's windows are as long as the prompt, so both see every key."""
+    _, d, nh, nkv, hd, H, dk, dv, E, top, groups, keep, ff, shared, kinds = size
+    gla = {"heads": H, "dim": dk, "vdim": dv, "tau": 16.0}
+    att = {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 50.0, "q_temp": {"coef": 0.1, "every": 1024}}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared},
+           "router": {"experts": E, "top": top, "scale": 2.0, "groups": {"count": groups, "keep": keep}}}
+    layers, zkinds = [], []
+    for k in kinds:
+        if isinstance(k, int):
+            layers.append({**layers[k], "weights_of": k})
+        else:
+            layers.append({"type": k, "mixer": gla if k == "gla" else att, "mlp": moe})
+            zkinds.append("mamba2" if k == "gla" else "attention")
+    vov = {"architecture": "Vovalorn", "vocab": vocab, "width": d, "norm": {"eps": 1e-6}, "residual_mult": 0.7, "layers": layers}
+    zom, _, _ = zomipel_pair(("", d, nh, nkv, hd, H * dv // 64, 64, dk, 8, E, top, ff, shared, 1 << 20, 0, tuple(zkinds), (1, 3, 2)), vocab)
+    for l in zom["layers"]:
+        l["mlp"] = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": E, "top": top}, "shared": {"ff": shared}}
+    return vov, zom, len(kinds)
+
+
+def vovalorn_run(pk, batch, steps, warmup, context=2048, prompt=4096):
+    return vebisun_run(pk, batch, steps, warmup, context, prompt, sizes=VOVALORN_SIZES, pair=vovalorn_pair, name="vovalorn", partner="zomipel")
+
+
 def zomipel_run(pk, batch, steps, warmup, context=2048, prompt=4096):
     return vebisun_run(pk, batch, steps, warmup, context, prompt, sizes=ZOMIPEL_SIZES, pair=zomipel_pair, name="zomipel", partner="tiralix")
 
@@ -782,7 +824,7 @@ def main():
                     help="with --only decode / prefill: another context length (decode) or prompt length (prefill) than the default run's")
     ap.add_argument("--config", default=None, choices=["1b-unequal", "13b-long"],
                     help="run one of the other workloads alone and print its figures")
-    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "attention", "products", "marginal", "issue-rate", "vebisun", "tiralix", "mimadra", "gunenex", "zomipel"],
+    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "attention", "products", "marginal", "issue-rate", "vebisun", "tiralix", "mimadra", "gunenex", "zomipel", "vovalorn"],
                     help="run one part only and print its figures (for profiling a small case)")
     args = ap.parse_args()
 
@@ -820,6 +862,9 @@ def main():
         return 0
     if args.only == "zomipel":
         print(json.dumps({"only": "zomipel", "peaks": pk, "sizes": zomipel_run(pk, args.batch, min(args.steps, 64), args.warmup)}))
+        return
+    if args.only == "vovalorn":
+        print(json.dumps({"only": "vovalorn", "peaks": pk, "sizes": vovalorn_run(pk, args.batch, min(args.steps, 64), args.warmup)}))
         return
     if args.only == "issue-rate":
         # what the thread that issues tensor-core products costs: cycles per instruction, one or two issuing threads

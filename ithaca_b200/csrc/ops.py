@@ -139,7 +139,9 @@ _SIGNATURES = {
     "ik_decay_rows": [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
     "ik_token_shift": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _u64, _i, _i, _i, _i, _i, _vp],
     "ik_row_decay": [_i, _vp, _i, _i, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
-    "ik_lowrank_decay": [_vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _f, _vp],
+    "ik_lowrank_decay": [_vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _f, _i, _vp],
+    "ik_gla_places": [_i, _i],
+    "ik_gla_chunks": [_vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _f, _f, _vp, _i, _i, _i, _i, _i, _vp],
     "ik_dynamic_tanh": [_vp, _vp, _vp, _vp, _f, _vp, _i, _i, _i, _vp],
     "ik_dynamic_tanh_embed": [_vp, _vp, _i, _vp, _vp, _f, _vp, _i, _i, _i, _f, _vp, _vp],
     "ik_dynamic_tanh_add": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _f, _vp, _f, _vp, _vp, _f, _vp, _i, _i, _i, _vp],
@@ -1581,8 +1583,9 @@ def decay_rows(x: torch.Tensor, bias: Optional[torch.Tensor], form: str, A_log: 
     return out
 
 
-def lowrank_decay(p: torch.Tensor, off: int, w: torch.Tensor, bias: Optional[torch.Tensor], power: float) -> torch.Tensor:
-    """sigmoid(z)^power [T, C] with z = p[:, off : off + rank] w + bias: decays whose logits are a projection of a low-rank factor
+def lowrank_decay(p: torch.Tensor, off: int, w: torch.Tensor, bias: Optional[torch.Tensor], power: float,
+                  log2: bool = False) -> torch.Tensor:
+    """sigmoid(z)^power [T, C] (``log2``: its logarithm to base 2) with z = p[:, off : off + rank] w + bias: decays whose logits are a projection of a low-rank factor
     that lies in columns of the float matrix ``p``; ``w`` float [rank, C]."""
     _need(p, "p", torch.float32, contiguous=False)
     _need(w, "w", torch.float32)
@@ -1591,7 +1594,36 @@ def lowrank_decay(p: torch.Tensor, off: int, w: torch.Tensor, bias: Optional[tor
         raise KernelError("lowrank_decay: the sizes do not fit together")
     out = torch.empty((T, C), dtype=torch.float32, device=p.device)
     _work(f"lowrank_decay {T}x{rank}x{C}", 4 * (T * (rank + C) + rank * C), 2 * T * rank * C)
-    _check(lib().ik_lowrank_decay(_ptr(p), p.stride(0), off, rank, _ptr(w), _ptr(bias), _ptr(out), T, C, power, _stream()), "lowrank_decay")
+    _check(lib().ik_lowrank_decay(_ptr(p), p.stride(0), off, rank, _ptr(w), _ptr(bias), _ptr(out), T, C, power, 1 if log2 else 0, _stream()), "lowrank_decay")
+    return out
+
+
+def gla_chunks(p: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, log2_decay: torch.Tensor, state: torch.Tensor, ctx,
+               n_heads: int, dk: int, dv: int, norm_w: torch.Tensor, eps: float, scale: float) -> Optional[torch.Tensor]:
+    """The recurrence of ``row_decay("plain", ...)`` by chunks of 64 tokens on the tensor cores, with what follows it: every head's
+    result RMS-normed over its values with one weight, times silu of columns ``g_off``.. of ``p``.  Returns bfloat16 [T, heads * dv], or
+    None when the kernels do not take these sizes."""
+    _need(p, "p", torch.float32, contiguous=False)
+    _need(log2_decay, "log2_decay", torch.float32)
+    _need(state, "state", torch.float32)
+    _need(norm_w, "norm_w", torch.float32)
+    T, H, B = p.shape[0], n_heads, ctx.n_seqs
+    if p.stride(1) != 1 or log2_decay.shape != (T, H * dk) or tuple(state.shape[1:]) != (2, H, dv, dk) or norm_w.numel() != dv \
+            or max(q_off + H * dk, k_off + H * dk, v_off + H * dv, g_off + H * dv) > p.shape[1]:
+        raise KernelError("gla_chunks: the sizes do not fit together")
+    if dk % 16 or dk > 128 or dv % 32 or dv > 256:
+        return None
+    places = lib().ik_gla_places(T, B)
+    ws = torch.empty((places, H, dv, dk), dtype=torch.float32, device=p.device)
+    keep = torch.empty((places, H, dk), dtype=torch.float32, device=p.device)
+    out = torch.empty((T, H * dv), dtype=torch.bfloat16, device=p.device)
+    _work(f"gla_chunks {T}x{H}x{dk}x{dv}", 8 * B * H * dk * dv + T * H * ((3 * dk + 2 * dv) * 4 + 2 * dv), T * H * (4 * dk * dv + 64 * (dk + dv)))
+    st = lib().ik_gla_chunks(_ptr(p), p.stride(0), q_off, k_off, v_off, g_off, _ptr(log2_decay), _ptr(ws), _ptr(keep), _ptr(state),
+                             _ptr(ctx.slots), _ptr(ctx.cu_seqlens), _ptr(ctx.kv_lens), _ptr(norm_w), eps, scale, _ptr(out), T, B, H, dk, dv,
+                             _stream())
+    if st == -2:
+        return None
+    _check(st, "gla_chunks", kernels=3)
     return out
 
 

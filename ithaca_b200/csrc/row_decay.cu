@@ -57,14 +57,14 @@ __global__ void decay_rows_kernel(const float* __restrict__ x, int ldx, const fl
 }
 
 // A decay whose logit is a projection of a low-rank factor that lies in columns of a wider product:
-//   z[t, c] = sum_r w[r, c] p[t, off + r] + bias[c],   out[t, c] = sigmoid(z)^power = exp(power * log sigmoid(z)).
+//   z[t, c] = sum_r w[r, c] p[t, off + r] + bias[c],   out[t, c] = sigmoid(z)^power = exp(power * log sigmoid(z)), or its log2.
 // w is stored [rank, C] (a factor's weights of neighbouring channels lie together).  A block takes TOK tokens and 256 channels; the
 // factors of its tokens go through shared memory, RC at a time, and a weight that is read serves all of its tokens.
 constexpr int LR_RC = 64;
 template <int TOK>
 __global__ void __launch_bounds__(256)
 lowrank_decay_kernel(const float* __restrict__ p, int ldp, int off, int rank, const float* __restrict__ w, const float* __restrict__ bias,
-                     float* __restrict__ out, int T, int C, float power) {
+                     float* __restrict__ out, int T, int C, float power, int log2_form) {
     __shared__ float low[TOK][LR_RC];
     ik_pdl_wait();
     IK_AFTER_WAIT(p);
@@ -96,7 +96,8 @@ lowrank_decay_kernel(const float* __restrict__ p, int ldp, int off, int rank, co
     for (int i = 0; i < TOK; i++) {
         if (t0 + i >= T) break;
         const float z = acc[i] + b, tail = log1pf(expf(-fabsf(z)));
-        out[(size_t)(t0 + i) * C + c] = expf(power * ((z < 0.f ? z : 0.f) - tail));
+        const float l = power * ((z < 0.f ? z : 0.f) - tail);
+        out[(size_t)(t0 + i) * C + c] = log2_form ? l * 1.4426950408889634f : expf(l);
     }
 }
 
@@ -350,14 +351,14 @@ IK_EXPORT int ik_decay_rows(const float* x, int ldx, const float* bias, const fl
 }
 
 IK_EXPORT int ik_lowrank_decay(const float* p, int ldp, int off, int rank, const float* w, const float* bias, float* out, int T, int C,
-                               float power, cudaStream_t stream) {
+                               float power, int log2_form, cudaStream_t stream) {
     if (T < 0 || C <= 0 || rank <= 0 || off < 0 || ldp < off + rank || !w) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
     // a few tokens: one a block, so that they spread over the SMs; a prompt: sixteen share a weight that is read
     if (T <= 64) {
-        IK_RETURN_IF_ERROR(ik_launch(lowrank_decay_kernel<1>, dim3(T, (C + 255) / 256), 256, 0, stream, p, ldp, off, rank, w, bias, out, T, C, power));
+        IK_RETURN_IF_ERROR(ik_launch(lowrank_decay_kernel<1>, dim3(T, (C + 255) / 256), 256, 0, stream, p, ldp, off, rank, w, bias, out, T, C, power, log2_form));
     } else {
-        IK_RETURN_IF_ERROR(ik_launch(lowrank_decay_kernel<16>, dim3((T + 15) / 16, (C + 255) / 256), 256, 0, stream, p, ldp, off, rank, w, bias, out, T, C, power));
+        IK_RETURN_IF_ERROR(ik_launch(lowrank_decay_kernel<16>, dim3((T + 15) / 16, (C + 255) / 256), 256, 0, stream, p, ldp, off, rank, w, bias, out, T, C, power, log2_form));
     }
     IK_LAUNCH_STATUS();
 }

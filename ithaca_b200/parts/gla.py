@@ -13,6 +13,9 @@ Per sequence and cache entry the mixer keeps S as float32 [2, heads, v_head_dim,
 position the state belongs to, as the other recurrences do, so that a decode step never overwrites what it read).  One product gives
 [q | k | v | g | Wa1 x] in float; the decay's second factor, the sigmoid and the root are one kernel on its last columns.  Decays, the
 state, its sums and the norm are float32 on both paths; only the products' operands are 16-bit on the bfloat16 path.
+
+A prompt on the bfloat16 path runs recurrence, norm and gate by chunks of 64 tokens on the tensor cores (``csrc/gla_chunk.cu``); single
+tokens, a few at a time, the float32 path and sizes that kernel does not take run the recurrence token by token.
 """
 from __future__ import annotations
 
@@ -28,6 +31,7 @@ from .base import Runtime, as_float32, register_mixer, to_device
 from .linear import Linear
 
 STATE = "gla_state"
+CHUNKED_FROM = 8            # tokens the longest sequence of a step brings
 
 
 class GatedLinearAttention:
@@ -75,9 +79,15 @@ class GatedLinearAttention:
         n = self.in_proj.out_features
         p = torch.empty((T, -(-n // 4) * 4), dtype=torch.float32, device=x.device)[:, :n]
         self.in_proj(x, out=p)                                                # [T, q | k | v | g | a1]
-        dec = ops.lowrank_decay(p, self.a_off, self.a2, self.a2_bias, self.power)
-        o = ops.row_decay("plain", p, 0, self.k_off, self.v_off, dec, None, None, cache.state(STATE), ctx, H, H, dk, dv, self.scale)
-        mid = ops.head_norm_gate(o, self.norm_w, self.norm_eps, p, self.g_off, H, rt.act_dtype, gate="silu")
+        mid = None
+        if rt.dtype == "bfloat16" and ctx.max_new >= CHUNKED_FROM:
+            decay = ops.lowrank_decay(p, self.a_off, self.a2, self.a2_bias, self.power, log2=True)
+            mid = ops.gla_chunks(p, 0, self.k_off, self.v_off, self.g_off, decay, cache.state(STATE), ctx, H, dk, dv, self.norm_w, self.norm_eps,
+                                 self.scale)
+        if mid is None:
+            decay = ops.lowrank_decay(p, self.a_off, self.a2, self.a2_bias, self.power)
+            o = ops.row_decay("plain", p, 0, self.k_off, self.v_off, decay, None, None, cache.state(STATE), ctx, H, H, dk, dv, self.scale)
+            mid = ops.head_norm_gate(o, self.norm_w, self.norm_eps, p, self.g_off, H, rt.act_dtype, gate="silu")
         self.o(mid, out=residual, accumulate=accumulate)
 
 
