@@ -26,7 +26,8 @@
 
 // Two compile-time options make further modules of the same size; a module without them has none of their code.
 //  * IK_SLOPES=1: a score loses slope[head] * (i - j) behind the cap (a distance bias), and the cap's tanh is accurate
-//    to float rounding (below).
+//    to float rounding (below).  Where a bound on the scores is known, keys so far back that the bias leaves all of them together
+//    less than half a unit in the last place of the softmax's sum are not visited.
 //  * IK_ONE_ROW=1: a page's rows are keys and values (there are no value pages), and every key has a float beside it
 //    (scales[page][kv head][place]) by which its scores are multiplied: the norm of a key whose value is the key in
 //    front of the norm.  A row is brought on chip once and serves both products.
@@ -108,6 +109,28 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// How far back a head can see under its distance bias.  No score in front of the bias is larger than B (what queries and keys of a
+// known length can reach, or the cap), so the keys at distances >= D weigh at most e^(2 B - slope D) / (1 - e^-slope) times what
+// the query's own key does; D makes that 2^-25.  norm: B without the query's temperature 1 + coef ln(floor((pos + 1) / every) + 1),
+// which is monotone in the position: a tile's largest stands at one of its ends.  norm 0: nothing is known, or no slope.
+struct Reach { float norm, cap, coef; int every; };
+__device__ __forceinline__ int reach_of(const Reach& R, float slope, int pos_a, int pos_b) {
+    if (!(R.norm > 0.f) || !(slope > 0.f)) return 0x3fffffff;
+    float B = R.norm;
+    if (R.every > 0)
+        B *= fmaxf(fabsf(fmaf(R.coef, logf((float)((pos_a + 1) / R.every + 1)), 1.0f)), fabsf(fmaf(R.coef, logf((float)((pos_b + 1) / R.every + 1)), 1.0f)));
+    if (R.cap > 0.f) B = fminf(B, R.cap);
+    const float D = (2.0f * B + 17.4f - logf(-expm1f(-slope))) / slope;
+    return D < 1e9f ? (int)D + 1 : 0x3fffffff;
+}
+// ... the furthest of the n heads a decode block serves
+__device__ __forceinline__ int group_reach(const Reach& R, const float* __restrict__ slopes, int h0, int n, int pos) {
+    float least = slopes[h0];
+    for (int i = 1; i < n; i++) least = fminf(least, slopes[h0 + i]);
+    return reach_of(R, least, pos, pos);
+}
+__device__ __forceinline__ int first_seen(int j_lo, int pos, int reach) { return max(j_lo, pos - reach); }
+
 // The pages a tile of queries walks: those of the first `keep` keys, which stay visible behind a window, then those from the
 // first query's window on.  Page number i of the walk; n_kept = how many of the first kind come before page p_lo.
 __device__ __forceinline__ int kept_pages(int keep, int p_lo) { return min((keep + PAGE - 1) / PAGE, p_lo); }
@@ -120,7 +143,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
                     bf16* __restrict__ out, const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
                     const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window, int keep,
                     int sink, const float* __restrict__ sink_v, const float* __restrict__ key_scales, const float* __restrict__ slopes,
-                    int n_pages, int* status) {
+                    Reach far, int n_pages, int* status) {
     ik_pdl_wait();
     ik_pdl_launch_dependents();
     constexpr int BM = 16 * NW, THREADS = 32 * NW, CH = HD / 8;          // CH: 16-byte chunks per row
@@ -137,7 +160,8 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages
     const int kv_len = kv_lens[b], start = kv_len - n_new;
     const int rows = min(BM, n_new - row0);
     const int pos_lo = start + row0, pos_hi = start + row0 + rows - 1;
-    const int j_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
+    int j_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
+    if (SLOPES && slopes) j_lo = first_seen(j_lo, pos_lo, reach_of(far, slopes[h], pos_lo, pos_hi));
     const int p_lo = j_lo / PAGE, n_kept = kept_pages(keep, p_lo), n_iter = n_kept + pos_hi / PAGE - p_lo + 1;
     const int kvh = h / (nh / nkv);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
@@ -338,7 +362,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                        const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
                        const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e,
                        int window, int keep, int sink, const float* __restrict__ sink_v, const float* __restrict__ key_scales,
-                       const float* __restrict__ slopes, int n_pages, int* status) {
+                       const float* __restrict__ slopes, Reach far, int n_pages, int* status) {
     extern __shared__ __align__(1024) unsigned char tc_smem[];
     ik_pdl_wait();
     ik_pdl_launch_dependents();
@@ -353,7 +377,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     const int kv_len = kv_lens[b], start = kv_len - n_new;
     const int rows = min(TC_BM, n_new - row0);
     const int pos_lo = start + row0, pos_hi = pos_lo + rows - 1;
-    const int j_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
+    int j_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
+    if (SLOPES && slopes) j_lo = first_seen(j_lo, pos_lo, reach_of(far, slopes[h], pos_lo, pos_hi));
     const int p_lo = j_lo / PAGE, n_kept = kept_pages(keep, p_lo), n_iter = n_kept + pos_hi / PAGE - p_lo + 1;
     const int kvh = h / (nh / nkv);
 
@@ -663,7 +688,7 @@ __global__ void __launch_bounds__(128)
 attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                    float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ kv_lens,
                    const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window, int keep,
-                   const float* __restrict__ key_scales, const float* __restrict__ slopes, int n_pages, int chunk_pages, int n_splits, int* status) {
+                   const float* __restrict__ key_scales, const float* __restrict__ slopes, Reach far, int n_pages, int chunk_pages, int n_splits, int* status) {
     ik_pdl_wait();
     constexpr int CH = HD / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -678,7 +703,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
     const int len = kv_lens[b], pos = len - 1;
     const int j0 = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
     // chunks of the pages the query sees, in their order (without a window: of all pages)
-    const int p_lo = j0 / PAGE, n_kept = kept_pages(keep, p_lo), n_seen = n_kept + pos / PAGE - p_lo + 1;
+    const int p_lo = (SLOPES && slopes ? first_seen(j0, pos, group_reach(far, slopes, kvh * G + hc * 16, min(16, G - hc * 16), pos)) : j0) / PAGE, n_kept = kept_pages(keep, p_lo), n_seen = n_kept + pos / PAGE - p_lo + 1;
     const int i_first = split * chunk_pages, i_last = min((split + 1) * chunk_pages, n_seen) - 1;
     if (i_first > i_last) return;                                  // there is no such chunk
 
@@ -849,13 +874,15 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
 // Merges the partials of each (sequence, head) in chunk order and writes the normalised output.
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                     bf16* __restrict__ out, const int* __restrict__ kv_lens, int nh, int window, int keep,
-                                    int sink, const float* __restrict__ sink_v, int chunk_pages, int n_splits) {
+                                    int sink, const float* __restrict__ sink_v, const float* __restrict__ slopes, Reach far, int nkv, int chunk_pages,
+                                    int n_splits) {
     ik_pdl_wait();
     ik_pdl_launch_dependents();
     const int b = blockIdx.x, h = blockIdx.y;
     const int len = kv_lens[b], pos = len - 1;
     const int j0 = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
-    const int p_lo = j0 / PAGE, s_last = (kept_pages(keep, p_lo) + pos / PAGE - p_lo) / chunk_pages;
+    const int G = nh / nkv, hc = (h % G) / 16;
+    const int p_lo = (SLOPES && slopes ? first_seen(j0, pos, group_reach(far, slopes, h / G * G + hc * 16, min(16, G - hc * 16), pos)) : j0) / PAGE, s_last = (kept_pages(keep, p_lo) + pos / PAGE - p_lo) / chunk_pages;
     const size_t base = ((size_t)b * nh + h) * n_splits;
     // a sink joins the merge as one more part: score 0 (or the head's own, in base-2 units), sum 1, no values
     const float m_sink = sink ? (sink_v ? sink_v[h] * 1.4426950408889634f : 0.f) : -INFINITY;
@@ -888,8 +915,9 @@ IK_EXPORT int ik_attn_take_wait_record(int* out4) { return ik_take_wait_record(o
 IK_EXPORT int ik_attn_prefill(const void* q, const void* k_pages, const void* v_pages, void* out, const int* cu_seqlens,
                               const int* kv_lens, const int* table, int table_stride, int B, int max_new, int nh,
                               int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, const float* key_scales,
-                              const float* slopes, int page_size, int n_pages, int* status, cudaStream_t stream) {
+                              const float* slopes, float reach_norm, float reach_coef, int reach_every, int page_size, int n_pages, int* status, cudaStream_t stream) {
     if (!options_fit(key_scales, slopes)) return IK_UNSUPPORTED;
+    const Reach far{reach_norm, softcap, reach_coef, reach_every};
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     if (B <= 0 || max_new <= 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size != PAGE || B > 65535 || nh > 65535)
         return IK_BAD_ARGUMENT;
@@ -903,7 +931,7 @@ IK_EXPORT int ik_attn_prefill(const void* q, const void* k_pages, const void* v_
     dim3 grid((max_new + BM - 1) / BM, nh, B);
     IK_RETURN_IF_ERROR(ik_launch(kern, grid, 32 * NW, smem, stream, (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, (bf16*)out,
                                           cu_seqlens, kv_lens, table, table_stride, nh, nkv,
-                                          sc_a, sc_b, window, keep, sink, sink_v, key_scales, slopes, n_pages, status));
+                                          sc_a, sc_b, window, keep, sink, sink_v, key_scales, slopes, far, n_pages, status));
     IK_LAUNCH_STATUS();
 }
 
@@ -911,8 +939,9 @@ IK_EXPORT int ik_attn_prefill(const void* q, const void* k_pages, const void* v_
 IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void* v_pages, void* out, const int* cu_seqlens,
                                  const int* kv_lens, const int* table, int table_stride, int T, int B, int max_new, int nh,
                                  int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, const float* key_scales,
-                                 const float* slopes, int page_size, int n_pages, int* status, cudaStream_t stream) {
+                                 const float* slopes, float reach_norm, float reach_coef, int reach_every, int page_size, int n_pages, int* status, cudaStream_t stream) {
     if (!options_fit(key_scales, slopes)) return IK_UNSUPPORTED;
+    const Reach far{reach_norm, softcap, reach_coef, reach_every};
 #if IK_HD == 64 || IK_HD == 128
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     if (T <= 0 || B <= 0 || max_new <= 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size != PAGE || B > 65535 || nh > 65535)
@@ -933,7 +962,7 @@ IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void*
     if (e != cudaSuccess) return (int)e;
     dim3 grid((max_new + TC_BM - 1) / TC_BM, nh, B);
     IK_RETURN_IF_ERROR(ik_launch(kern, grid, 192, TC_SMEM, stream, mq, mk, mv, (bf16*)out, cu_seqlens, kv_lens, table,
-                                 table_stride, nh, nkv, sc_a, sc_b, window, keep, sink, sink_v, key_scales, slopes, n_pages, status));
+                                 table_stride, nh, nkv, sc_a, sc_b, window, keep, sink, sink_v, key_scales, slopes, far, n_pages, status));
     IK_LAUNCH_STATUS();
 #else
     return IK_UNSUPPORTED;
@@ -946,9 +975,10 @@ IK_EXPORT int ik_attn_prefill_tc(const void* q, const void* k_pages, const void*
 IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_pages, void* out, float* part_o,
                              float* part_ml, const int* kv_lens, const int* table, int table_stride, int B, int nh,
                              int nkv, float scale, float softcap, int window, int keep, int sink, const float* sink_v, const float* key_scales,
-                             const float* slopes, int page_size, int n_pages, int chunk_pages, int n_splits, int ring_kb, int* status,
+                             const float* slopes, float reach_norm, float reach_coef, int reach_every, int page_size, int n_pages, int chunk_pages, int n_splits, int ring_kb, int* status,
                              cudaStream_t stream) {
     if (!options_fit(key_scales, slopes)) return IK_UNSUPPORTED;
+    const Reach far{reach_norm, softcap, reach_coef, reach_every};
     const float sc_a = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, sc_b = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     if (B <= 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size != PAGE || chunk_pages <= 0 || n_splits <= 0 ||
         n_splits > 65535)
@@ -974,7 +1004,7 @@ IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_p
         }                                                                                                            \
         IK_RETURN_IF_ERROR(ik_launch(kern, grid, 128, smem, stream, (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, part_o, part_ml, \
                                           kv_lens, table, table_stride, nh, nkv, sc_a, sc_b, window, keep, \
-                                          key_scales, slopes, n_pages, chunk_pages, n_splits, status));                                   \
+                                          key_scales, slopes, far, n_pages, chunk_pages, n_splits, status));                                   \
     }
     if (ns == 2) IK_DEC(2) else if (ns == 3) IK_DEC(3) else IK_DEC(4)
 #undef IK_DEC
@@ -982,6 +1012,6 @@ IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_p
     if (e != cudaSuccess) return (int)e;
     dim3 grid2(B, nh);
     IK_RETURN_IF_ERROR(ik_launch_family(IK_FAMILY_ATTENTION_MERGE, attn_combine_kernel, grid2, HD < 128 ? HD : 128, 0, stream, part_o, part_ml, (bf16*)out, kv_lens, nh, window, keep,
-                                                                    sink, sink_v, chunk_pages, n_splits));
+                                                                    sink, sink_v, slopes, far, nkv, chunk_pages, n_splits));
     IK_LAUNCH_STATUS();
 }

@@ -61,11 +61,11 @@ def module(head_dim: int, slopes: bool = False, one_row: bool = False) -> ctypes
     m = _modules.get(key)
     if m is None:
         m = build.load_library(*build.attention_module(head_dim, slopes, one_row))
-        m.ik_attn_prefill.argtypes = [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _vp]
+        m.ik_attn_prefill.argtypes = [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _f, _f, _i, _i, _i, _vp, _vp]
         m.ik_attn_prefill.restype = _i
-        m.ik_attn_prefill_tc.argtypes = [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _vp]
+        m.ik_attn_prefill_tc.argtypes = [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _f, _f, _i, _i, _i, _vp, _vp]
         m.ik_attn_prefill_tc.restype = _i
-        m.ik_attn_decode.argtypes = [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i,
+        m.ik_attn_decode.argtypes = [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _f, _f, _i, _i, _i, _i, _i, _i,
                                      _vp, _vp]
         m.ik_attn_decode.restype = _i
         m.ik_attn_take_wait_record.argtypes = [_vp]
@@ -80,12 +80,14 @@ def prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, cu_se
             kv_lens: torch.Tensor, table: torch.Tensor, n_seqs: int, max_new: int, n_heads: int, scale: float,
             window: int, status: Optional[torch.Tensor], out: Optional[torch.Tensor] = None,
             kind: str = "auto", work: Optional[Tuple[int, int]] = None, softcap: float = 0.0, sink=False, keep: int = 0,
-            key_scales: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+            key_scales: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None, reach=None) -> torch.Tensor:
     """``kind``: "tc" = the tcgen05 kernel (head sizes 64 and 128), "mma" = the warp-level kernel,
     "auto" = tcgen05 where it applies.  ``softcap``: scores become cap * tanh(score / cap) (0 = no cap).  ``sink``: the
     softmax's denominator counts one more key of score 0 that carries no value (True), or of a score per head (a float32
     tensor [n_heads], not scaled).  ``key_scales``: the pages' rows are keys and values (``v_pages`` None), and every score is
-    multiplied by its key's number.  ``slopes`` [n_heads]: a score loses slope * distance, behind the cap.  ``keep``: under a window the first ``keep`` keys stay visible."""
+    multiplied by its key's number.  ``slopes`` [n_heads]: a score loses slope * distance, behind the cap.  ``reach`` = (norm, coef, every): no
+    score in front of cap and bias is larger than norm * |1 + coef ln(floor((pos + 1) / every) + 1)| (every 0: than norm), so that keys
+    the bias makes negligible need not be visited (None: nothing is known).  ``keep``: under a window the first ``keep`` keys stay visible."""
     n_pages, nkv, page_size, hd = k_pages.shape
     ops.check_score_extras(key_scales, slopes, k_pages, n_heads)
     m = module(hd, slopes is not None, key_scales is not None)
@@ -95,7 +97,7 @@ def prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, cu_se
         ops._work(f"attention prefill tcgen05 {q.shape[0]}x{n_heads}", *(work or (0, 0)))
         st = m.ik_attn_prefill_tc(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(cu_seqlens), _ptr(kv_lens),
                                   _ptr(table), table.stride(0), q.shape[0], n_seqs, max_new, n_heads, nkv, scale, softcap, window, keep,
-                                  ops.sink_flag(sink), _ptr(ops.sink_values(sink, n_heads)), _ptr(key_scales), _ptr(slopes), page_size, n_pages, _ptr(status), _stream())
+                                  ops.sink_flag(sink), _ptr(ops.sink_values(sink, n_heads)), _ptr(key_scales), _ptr(slopes), *(reach or (0.0, 0.0, 0)), page_size, n_pages, _ptr(status), _stream())
         if st != -2:
             _check(st, "attention prefill (tcgen05)")
             return out
@@ -104,7 +106,7 @@ def prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, cu_se
     ops._work(f"attention prefill mma {q.shape[0]}x{n_heads}", *(work or (0, 0)))
     _check(m.ik_attn_prefill(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(cu_seqlens), _ptr(kv_lens),
                              _ptr(table), table.stride(0), n_seqs, max_new, n_heads, nkv, scale, softcap, window, keep, ops.sink_flag(sink),
-                             _ptr(ops.sink_values(sink, n_heads)), _ptr(key_scales), _ptr(slopes), page_size, n_pages, _ptr(status), _stream()), "attention prefill")
+                             _ptr(ops.sink_values(sink, n_heads)), _ptr(key_scales), _ptr(slopes), *(reach or (0.0, 0.0, 0)), page_size, n_pages, _ptr(status), _stream()), "attention prefill")
     return out
 
 
@@ -112,7 +114,7 @@ def decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, kv_len
            n_seqs: int, kv_len_bound: int, n_heads: int, scale: float, window: int, status: Optional[torch.Tensor],
            out: Optional[torch.Tensor] = None, chunk_pages: int = DECODE_CHUNK_PAGES, ring_kb: int = 0,
            work: Optional[Tuple[int, int]] = None, softcap: float = 0.0, sink=False, keep: int = 0,
-            key_scales: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+            key_scales: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None, reach=None) -> torch.Tensor:
     """``kv_len_bound``: no sequence of the step is longer than this (it sizes the grid and the
     scratch for the partial results; blocks beyond a sequence's length return at once).  ``keep``: under a window the
     first ``keep`` keys stay visible."""
@@ -127,14 +129,14 @@ def decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, kv_len
     ops._work(f"attention decode {n_seqs}x{n_heads}", *(work or (0, 0)))
     _check(m.ik_attn_decode(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(part_o), _ptr(part_ml),
                             _ptr(kv_lens), _ptr(table), table.stride(0), n_seqs, n_heads, nkv, scale, softcap, window, keep,
-                            ops.sink_flag(sink), _ptr(ops.sink_values(sink, n_heads)), _ptr(key_scales), _ptr(slopes), page_size, n_pages, chunk_pages, n_splits, ring_kb,
+                            ops.sink_flag(sink), _ptr(ops.sink_values(sink, n_heads)), _ptr(key_scales), _ptr(slopes), *(reach or (0.0, 0.0, 0)), page_size, n_pages, chunk_pages, n_splits, ring_kb,
                             _ptr(status), _stream()), "attention decode", kernels=2)
     return out
 
 
 def attend(q, k_pages, v_pages, ctx, table, n_heads: int, scale: float, window: int,
            status, softcap: float = 0.0, sink=False, keep: int = 0,
-            key_scales: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+            key_scales: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None, reach=None) -> Optional[torch.Tensor]:
     """Returns None when no specialised kernel takes these sizes or options (the caller then uses the
     CUDA-core kernel)."""
     n_pages, nkv, page_size, hd = k_pages.shape
@@ -154,6 +156,6 @@ def attend(q, k_pages, v_pages, ctx, table, n_heads: int, scale: float, window: 
         # from the bound, not from this step's longest sequence: a captured graph is replayed for other lengths
         chunk = decode_chunk_pages(ctx.n_seqs, n_heads, nkv, seen_pages(ctx.kv_len_bound, window, keep, page_size) * page_size, page_size)
         return decode(q, k_pages, v_pages, ctx.kv_lens, table, ctx.n_seqs, ctx.kv_len_bound, n_heads, scale, window,
-                      status, chunk_pages=chunk, work=work, softcap=softcap, sink=sink, keep=keep, key_scales=key_scales, slopes=slopes)
+                      status, chunk_pages=chunk, work=work, softcap=softcap, sink=sink, keep=keep, key_scales=key_scales, slopes=slopes, reach=reach)
     return prefill(q, k_pages, v_pages, ctx.cu_seqlens, ctx.kv_lens, table, ctx.n_seqs, ctx.max_new, n_heads, scale,
-                   window, status, work=work, softcap=softcap, sink=sink, keep=keep, key_scales=key_scales, slopes=slopes)
+                   window, status, work=work, softcap=softcap, sink=sink, keep=keep, key_scales=key_scales, slopes=slopes, reach=reach)

@@ -132,6 +132,57 @@ norm_rope_append_kernel(const float* __restrict__ p, int ldp, int q_off, int k_o
     }
 }
 
+// The same without rotation, bias and weights and with key scales, a warp per token and head: a lane keeps its values (four at a
+// time, hd a multiple of 4 up to 512) between the sum of squares and the division.
+template <typename TQ, typename TC>
+__global__ void __launch_bounds__(256)
+unit_append_kernel(const float* __restrict__ p, int ldp, int q_off, int k_off, float eps, TQ* __restrict__ q_out, TC* __restrict__ k_pages,
+                   const int* __restrict__ token_seq, const int* __restrict__ token_pos, const int* __restrict__ table, int table_stride, int T,
+                   int nh, int nkv, int hd, int page_size, int n_pages, int write_cache, float temp_coef, int temp_every,
+                   float* __restrict__ key_scales, int* status) {
+    ik_pdl_wait();
+    IK_AFTER_WAIT(p);
+    IK_AFTER_WAIT(token_seq);
+    IK_AFTER_WAIT(token_pos);
+    IK_AFTER_WAIT(table);
+    ik_pdl_launch_dependents();
+    const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t = unit / (nh + nkv), head = unit - t * (nh + nkv);
+    if (t >= T) return;
+    const bool is_q = head < nh;
+    const float* src = p + (size_t)t * ldp + (is_q ? q_off + head * hd : k_off + (head - nh) * hd);
+    float4 v[4];
+    float ss = 0.f;
+    #pragma unroll
+    for (int r = 0; r < 4; r++) {
+        const int i = 4 * (lane + 32 * r);
+        v[r] = i < hd ? *reinterpret_cast<const float4*>(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss = fmaf(v[r].x, v[r].x, fmaf(v[r].y, v[r].y, fmaf(v[r].z, v[r].z, fmaf(v[r].w, v[r].w, ss))));
+    }
+    #pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const int pos = token_pos[t];
+    float inv = 1.0f / sqrtf(ss / (float)hd + eps);
+    if (is_q) {
+        if (temp_every > 0) inv *= fmaf(temp_coef, logf((float)((pos + 1) / temp_every + 1)), 1.0f);
+        TQ* dst = q_out + ((size_t)t * nh + head) * hd;
+        #pragma unroll
+        for (int r = 0; r < 4; r++) {
+            const int i = 4 * (lane + 32 * r);
+            if (i < hd) ik_st4(dst, i, make_float4(v[r].x * inv, v[r].y * inv, v[r].z * inv, v[r].w * inv));
+        }
+    } else if (write_cache) {
+        const int page = table[(size_t)token_seq[t] * table_stride + pos / page_size];
+        if (page < 0 || page >= n_pages) { if (lane == 0) ik_set_status(status, IK_STATUS_WRITE_NO_PAGE); return; }
+        const size_t place = ((size_t)page * nkv + (head - nh)) * page_size + pos % page_size;
+        #pragma unroll
+        for (int r = 0; r < 4; r++) {
+            const int i = 4 * (lane + 32 * r);
+            if (i < hd) ik_st4(k_pages, place * hd + i, v[r]);
+        }
+        if (lane == 0) key_scales[place] = inv;
+    }
+}
+
 IK_EXPORT int ik_norm_rope_append(const float* p, int ldp, int q_off, int k_off, int v_off, const float* q_w, const float* k_w,
                                   float eps, void* q_out, int q_dtype, void* k_pages, void* v_pages, int cache_dtype,
                                   const int* token_seq, const int* token_pos, const int* table, int table_stride,
@@ -144,6 +195,16 @@ IK_EXPORT int ik_norm_rope_append(const float* p, int ldp, int q_off, int k_off,
     if (per_head < 0 || per_head > 2 || (per_head == 2 && (q_w || k_w)) || temp_every < 0) return IK_BAD_ARGUMENT;
     if (key_scales ? per_head != 2 || rot || v_norm : !v_pages) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
+    if (key_scales && !bias && hd % 4 == 0 && hd <= 512 && ldp % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && ((uintptr_t)p & 15) == 0 &&
+        ((uintptr_t)q_out & 15) == 0 && ((uintptr_t)k_pages & 15) == 0 && q_dtype == cache_dtype && (q_dtype == IK_F32 || q_dtype == IK_BF16)) {
+        const int blocks = (int)(((long long)T * (nh + nkv) + 7) / 8);
+#define IK_UNIT(TT)                                                                                                                    \
+    IK_RETURN_IF_ERROR(ik_launch(unit_append_kernel<TT, TT>, blocks, 256, 0, stream, p, ldp, q_off, k_off, eps, (TT*)q_out, (TT*)k_pages, token_seq, \
+                                 token_pos, table, table_stride, T, nh, nkv, hd, page_size, n_pages, write_cache, temp_coef, temp_every, key_scales, status))
+        if (q_dtype == IK_F32) IK_UNIT(float); else IK_UNIT(__nv_bfloat16);
+#undef IK_UNIT
+        IK_LAUNCH_STATUS();
+    }
     const size_t smem = (size_t)(rot + (per_head ? nh + nkv : 0) + (v_norm ? nkv : 0)) * sizeof(float);
 #define IK_NRA(TQ, TC)                                                                                                       \
     IK_RETURN_IF_ERROR(ik_launch(norm_rope_append_kernel<TQ, TC>, T, 256, smem, stream, p, ldp, q_off, k_off, v_off, q_w, k_w, eps, \

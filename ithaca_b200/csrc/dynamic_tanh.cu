@@ -22,35 +22,41 @@ __device__ __forceinline__ float4 dyt4(float4 x, const Dyt& n, int i) {
 // V elements per thread and turn (4: sizes and pointers allow 16-byte accesses)
 template <typename TO, int V>
 __global__ void __launch_bounds__(256)
-dynamic_tanh_kernel(const float* __restrict__ x, const int* __restrict__ rows_in, Dyt n, TO* __restrict__ out, size_t total, int d) {
+dynamic_tanh_kernel(const float* __restrict__ x, const int* __restrict__ rows_in, Dyt n, TO* __restrict__ out, unsigned total, unsigned d) {
     ik_pdl_wait();
     IK_AFTER_WAIT(x);
     IK_AFTER_WAIT(rows_in);
     ik_pdl_launch_dependents();
-    const size_t stride = (size_t)gridDim.x * blockDim.x * V;
-    for (size_t idx = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V; idx < total; idx += stride) {
-        const size_t r = idx / d;
-        const int i = (int)(idx - r * d);
-        const size_t src = (size_t)(rows_in ? rows_in[r] : (int)r) * d + i;
+    const unsigned stride = gridDim.x * blockDim.x * V;
+    for (unsigned idx = (blockIdx.x * blockDim.x + threadIdx.x) * V; idx < total; idx += stride) {
+        const unsigned r = idx / d, i = idx - r * d;
+        const size_t src = rows_in ? (size_t)rows_in[r] * d + i : idx;
         if (V == 4) ik_st4(out, idx, dyt4(ik_ld4(x, src), n, i));
         else ik_st(out, idx, dyt1(x[src], n.alpha, n.w[i], n.b[i]));
     }
 }
 
-template <typename TW>
+template <typename TW, int V>
 __global__ void __launch_bounds__(256)
-dynamic_tanh_embed_kernel(const int* __restrict__ ids, const TW* __restrict__ table, Dyt n, float* __restrict__ out, size_t total, int d,
-                          int V, float scale, int* status) {
+dynamic_tanh_embed_kernel(const int* __restrict__ ids, const TW* __restrict__ table, Dyt n, float* __restrict__ out, unsigned total, unsigned d,
+                          int vocab, float scale, int* status) {
     ik_pdl_wait();
     IK_AFTER_WAIT(ids);
     ik_pdl_launch_dependents();
-    const size_t stride = (size_t)gridDim.x * blockDim.x;
-    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += stride) {
-        const size_t t = idx / d;
-        const int i = (int)(idx - t * d), id = ids[t];
-        const bool ok = id >= 0 && id < V;
+    const unsigned stride = gridDim.x * blockDim.x * V;
+    for (unsigned idx = (blockIdx.x * blockDim.x + threadIdx.x) * V; idx < total; idx += stride) {
+        const unsigned t = idx / d, i = idx - t * d;
+        const int id = ids[t];
+        const bool ok = id >= 0 && id < vocab;
         if (!ok && i == 0) ik_set_status(status, IK_STATUS_BAD_TOKEN);
-        out[idx] = ok ? dyt1(ik_ld(table, (size_t)id * d + i) * scale, n.alpha, n.w[i], n.b[i]) : 0.f;
+        const size_t src = (size_t)(ok ? id : 0) * d + i;
+        if (V == 4) {
+            float4 v = ik_ld4(table, src);
+            v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+            ik_st4(out, idx, ok ? dyt4(v, n, i) : make_float4(0.f, 0.f, 0.f, 0.f));
+        } else {
+            out[idx] = ok ? dyt1(ik_ld(table, src) * scale, n.alpha, n.w[i], n.b[i]) : 0.f;
+        }
     }
 }
 
@@ -62,7 +68,7 @@ struct Parts {                                           // the experts' results
 template <typename TO, int V, bool SUM>
 __global__ void __launch_bounds__(256)
 dynamic_tanh_add_kernel(const float* __restrict__ y, Parts s, Dyt n, float* __restrict__ residual, float mult, Dyt next, TO* __restrict__ copy,
-                        size_t total, int d) {
+                        unsigned total, unsigned d) {
     ik_pdl_wait();
     IK_AFTER_WAIT(y);
     IK_AFTER_WAIT(s.parts);
@@ -72,17 +78,16 @@ dynamic_tanh_add_kernel(const float* __restrict__ y, Parts s, Dyt n, float* __re
     IK_AFTER_WAIT(s.extra_weight);
     IK_AFTER_WAIT(residual);
     ik_pdl_launch_dependents();
-    const size_t stride = (size_t)gridDim.x * blockDim.x * V;
-    for (size_t idx = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V; idx < total; idx += stride) {
-        const size_t t = idx / d;
-        const int i = (int)(idx - t * d);
+    const unsigned stride = gridDim.x * blockDim.x * V;
+    for (unsigned idx = (blockIdx.x * blockDim.x + threadIdx.x) * V; idx < total; idx += stride) {
+        const unsigned t = idx / d, i = idx - t * d;
         float v[V];
         if (SUM) {
             #pragma unroll
             for (int j = 0; j < V; j++) v[j] = 0.f;
             #pragma unroll 4
             for (int k = 0; k < s.top; k++) {
-                const size_t a = t * s.top + k;
+                const size_t a = (size_t)t * s.top + k;
                 const float wk = s.weight ? s.weight[a] : 1.0f;
                 const float* src = s.parts + (s.row_of ? (size_t)s.row_of[a] : a) * d + i;
                 if (V == 4) {
@@ -117,8 +122,8 @@ dynamic_tanh_add_kernel(const float* __restrict__ y, Parts s, Dyt n, float* __re
     }
 }
 
-inline int blocks_for(size_t turns) {
-    const size_t want = (turns + 255) / 256, cap = (size_t)ik_sm_count() * 16;
+inline int blocks_for(unsigned turns) {
+    const unsigned want = (turns + 255) / 256, cap = (unsigned)ik_sm_count() * 16;
     return (int)(want < cap ? want : cap);
 }
 inline bool on16(const void* p) { return ((uintptr_t)p & 15) == 0; }
@@ -129,7 +134,8 @@ IK_EXPORT int ik_dynamic_tanh(const float* x, const int* rows_in, const float* w
                               int rows, int d, cudaStream_t stream) {
     if (rows < 0 || d <= 0 || !w || !b) return IK_BAD_ARGUMENT;
     if (rows == 0) return IK_OK;
-    const size_t total = (size_t)rows * d;
+    if ((size_t)rows * d >= 1u << 31) return IK_UNSUPPORTED;
+    const unsigned total = (unsigned)rows * d;
     const Dyt n{w, b, alpha};
     const bool v4 = d % 4 == 0 && on16(x) && on16(w) && on16(b) && on16(out);
 #define IK_DYT(TO)                                                                                                                \
@@ -146,14 +152,17 @@ IK_EXPORT int ik_dynamic_tanh_embed(const int* ids, const void* table, int table
                                     int T, int d, int V, float scale, int* status, cudaStream_t stream) {
     if (T < 0 || d <= 0 || V <= 0 || !w || !b) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
-    const size_t total = (size_t)T * d;
+    if ((size_t)T * d >= 1u << 31) return IK_UNSUPPORTED;
+    const unsigned total = (unsigned)T * d;
     const Dyt n{w, b, alpha};
-    if (table_dtype == IK_F32)
-        IK_RETURN_IF_ERROR(ik_launch(dynamic_tanh_embed_kernel<float>, blocks_for(total), 256, 0, stream, ids, (const float*)table, n, out, total, d, V, scale, status));
-    else if (table_dtype == IK_BF16)
-        IK_RETURN_IF_ERROR(ik_launch(dynamic_tanh_embed_kernel<__nv_bfloat16>, blocks_for(total), 256, 0, stream, ids, (const __nv_bfloat16*)table, n, out,
-                                     total, d, V, scale, status));
+    const bool v4 = d % 4 == 0 && on16(table) && on16(w) && on16(b) && on16(out);
+#define IK_DYT_EMBED(TW)                                                                                                                        \
+    if (v4) IK_RETURN_IF_ERROR(ik_launch((dynamic_tanh_embed_kernel<TW, 4>), blocks_for(total / 4), 256, 0, stream, ids, (const TW*)table, n, out, total, d, V, scale, status)); \
+    else IK_RETURN_IF_ERROR(ik_launch((dynamic_tanh_embed_kernel<TW, 1>), blocks_for(total), 256, 0, stream, ids, (const TW*)table, n, out, total, d, V, scale, status))
+    if (table_dtype == IK_F32) { IK_DYT_EMBED(float); }
+    else if (table_dtype == IK_BF16) { IK_DYT_EMBED(__nv_bfloat16); }
     else return IK_BAD_ARGUMENT;
+#undef IK_DYT_EMBED
     IK_LAUNCH_STATUS();
 }
 
@@ -164,7 +173,8 @@ IK_EXPORT int ik_dynamic_tanh_add(const float* y, const float* parts, const floa
                                   const float* nw, const float* nb, float nalpha, void* copy, int copy_dtype, int T, int d, cudaStream_t stream) {
     if (T < 0 || d <= 0 || !w || !b || !residual || (!y && (!parts || top <= 0)) || (copy && (!nw || !nb))) return IK_BAD_ARGUMENT;
     if (T == 0) return IK_OK;
-    const size_t total = (size_t)T * d;
+    if ((size_t)T * d >= 1u << 31) return IK_UNSUPPORTED;
+    const unsigned total = (unsigned)T * d;
     const Dyt n{w, b, alpha}, next{nw, nb, nalpha};
     const Parts s{parts, weight, row_of, extra, extra_weight, top};
     const bool v4 = d % 4 == 0 && on16(y) && on16(parts) && on16(extra) && on16(w) && on16(b) && on16(residual) && on16(nw) && on16(nb) && on16(copy);

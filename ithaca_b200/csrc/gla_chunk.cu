@@ -5,10 +5,11 @@
 //   own     A_ij = sum_d q_i k_j 2^(sum of log2 a over j+1 .. i) for j <= i;            o_i += sum_j A_ij v_j
 //   carry   o_i += sum_d q_i 2^(sum over the chunk's tokens up to i) S_before
 //   gain    D = sum_j k_j 2^(sum over the chunk's tokens behind j) v_j^T;                S_after = 2^(sum over the chunk) S_before + D
-// No exponent is ever positive but one kind: A's rows of block I are taken as (q_i 2^L_i) . (k_j 2^(rest from j to I's beginning)), the
-// rest being a sum of totals and T_J - L_j for J < I, and -L_j for block I's own columns.  The latter grows as the block forgets;
-// up to 2^100 a product of the two factors still is a rounded one of the true term, and a block that forgets more forms its own 16 x
-// 16 entries directly.
+// A's entry of token i of block I and token j of block J is a product of a factor of i and a factor of j, q_i 2^(from a place between
+// them to i) . k_j 2^(from j to that place): the middle of the chunk if it lies between I and J, else the beginning of I.  These
+// exponents are never positive.  In block I's own columns the place (the beginning of I) lies in front of j, and k_j's exponent is
+// -L_j, which grows as the block forgets; up to 2^100 the product of the two factors still is a rounded one of the true term, and a
+// block that forgets more forms its own 16 x 16 entries directly.
 //
 // The chunks of all sequences and heads run at once, in three kernels: the gains (D and the chunk's decay), the states in front
 // of every chunk (an elementwise recurrence over the chunks, which also takes the sequence's state from its slot and puts
@@ -40,8 +41,8 @@ __device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint3
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
-// x as the sum of two bfloat16 numbers; two x at a time, packed
-__device__ __forceinline__ void split(float x, bf16& hi, bf16& lo) { hi = __float2bfloat16_rn(x); lo = __float2bfloat16_rn(x - __bfloat162float(hi)); }
+__device__ __forceinline__ void prefetch_l2(const float* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+// x and y as sums of two bfloat16 numbers each, packed
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
     hi = *reinterpret_cast<const uint32_t*>(&h);
@@ -62,10 +63,11 @@ __device__ __forceinline__ bool find_chunk(const int* __restrict__ cu, int B, in
 }
 
 // v of the chunk's tokens (zeros behind the last), as two terms: [C][dv + 8] each
-__device__ __forceinline__ void stage_values(const float* __restrict__ p, int ldp, int off, int t0, int n, int dv, bf16* vh, bf16* vl) {
+__device__ __forceinline__ void stage_values(const float* __restrict__ p, int ldp, int off, int t0, int n, int dv, bf16* vh, bf16* vl,
+                                             int first, int threads) {
     const int q4 = dv / 4, ld = dv + 8;
-    #pragma unroll 4
-    for (int idx = threadIdx.x; idx < C * q4; idx += 256) {
+    #pragma unroll 8
+    for (int idx = first; idx < C * q4; idx += threads) {
         const int r = idx / q4, x = (idx - r * q4) * 4;
         const float4 v = r < n ? *reinterpret_cast<const float4*>(p + (size_t)(t0 + r) * ldp + off + x) : make_float4(0.f, 0.f, 0.f, 0.f);
         uint2 h, l;
@@ -76,13 +78,34 @@ __device__ __forceinline__ void stage_values(const float* __restrict__ p, int ld
     }
 }
 
+// 16 tokens of two key channels: columns of a matrix with row stride ld, from token t0 on, zeros from token n on.
+__device__ __forceinline__ void load16(float2 (&x)[SUB], const float* __restrict__ src, size_t ld, int n) {
+    #pragma unroll
+    for (int i = 0; i < SUB; i++) x[i] = i < n ? *reinterpret_cast<const float2*>(src + i * ld) : make_float2(0.f, 0.f);
+}
+__device__ __forceinline__ void running_sums(float2 (&x)[SUB]) {
+    #pragma unroll
+    for (int i = 1; i < SUB; i++) { x[i].x += x[i - 1].x; x[i].y += x[i - 1].y; }
+}
+// rows[i] = x_i 2^(base + sign L_i), as two terms, channels d and d + 1 packed; the exponent at most `top`
+__device__ __forceinline__ void put16(const float2 (&x)[SUB], const float2 (&L)[SUB], float2 base, float sign, float top, bf16* hi, bf16* lo, int ld) {
+    #pragma unroll
+    for (int i = 0; i < SUB; i++) {
+        uint32_t h, l;
+        split2(x[i].x * ex2(fminf(fmaf(sign, L[i].x, base.x), top)), x[i].y * ex2(fminf(fmaf(sign, L[i].y, base.y), top)), h, l);
+        *reinterpret_cast<uint32_t*>(hi + i * ld) = h;
+        *reinterpret_cast<uint32_t*>(lo + i * ld) = l;
+    }
+}
+__device__ __forceinline__ float2 add2(float2 a, float2 b) { return make_float2(a.x + b.x, a.y + b.y); }
+
 // ------------------------------------------------------------------ gains
-// ws[place][h][dv][dk] = D (values x key channels), keep[place][h][dk] = the chunk's decay.  IT: (channel, block) pairs a thread
-// has, NK: key channels in eights (at most).
-template <int IT, int NK>
+// ws[place][h][dv][dk] = D (values x key channels), keep[place][h][dk] = the chunk's decay.  The first 128 threads bring the values,
+// the others a block's tokens of two key channels each (IT times).  NK: key channels in eights (at most).
+template <int DK, int DV, int IT, int NK>
 __global__ void __launch_bounds__(256)
 gla_gain_kernel(const float* __restrict__ p, int ldp, int k_off, int v_off, const float* __restrict__ g, const int* __restrict__ cu, int B,
-                float* __restrict__ ws, float* __restrict__ keep, int H, int dk, int dv) {
+                float* __restrict__ ws, float* __restrict__ keep, int H, int dk_, int dv_) {
     extern __shared__ __align__(16) unsigned char smem[];
     ik_pdl_wait();
     IK_AFTER_WAIT(p);
@@ -91,40 +114,41 @@ gla_gain_kernel(const float* __restrict__ p, int ldp, int k_off, int v_off, cons
     ik_pdl_launch_dependents();
     int b, c;
     if (!find_chunk(cu, B, blockIdx.x, b, c)) return;
-    const int h = blockIdx.y, t0 = cu[b] + c * C, n = min(C, cu[b + 1] - t0), ldk = dk + 8, ldv = dv + 8;
+    const int dk = DK ? DK : dk_, dv = DV ? DV : dv_;
+    const int h = blockIdx.y, t0 = cu[b] + c * C, n = min(C, cu[b + 1] - t0), ldk = dk + 8, ldv = dv + 8, pairs = dk / 2;
     float* tot = (float*)smem;                              // [NSUB][dk]
     bf16* kh = (bf16*)(tot + NSUB * dk);                    // [C][ldk]
     bf16* kl = kh + C * ldk;
     bf16* vh = kl + C * ldk;                                // [C][ldv]
     bf16* vl = vh + C * ldv;
-    float L[IT][SUB], k[IT][SUB];
-    #pragma unroll
-    for (int it = 0; it < IT; it++) {
-        const int item = threadIdx.x + it * 256, J = item / dk, d = item - J * dk;
-        if (J >= NSUB) break;
-        #pragma unroll
-        for (int i = 0; i < SUB; i++) {
-            const int r = J * SUB + i;
-            L[it][i] = r < n ? g[((size_t)(t0 + r) * H + h) * dk + d] : 0.f;
-            k[it][i] = r < n ? p[(size_t)(t0 + r) * ldp + k_off + h * dk + d] : 0.f;
-        }
-        #pragma unroll
-        for (int i = 1; i < SUB; i++) L[it][i] += L[it][i - 1];
-        tot[J * dk + d] = L[it][SUB - 1];
-    }
-    stage_values(p, ldp, v_off + h * dv, t0, n, dv, vh, vl);
-    __syncthreads();
     const size_t place = (size_t)blockIdx.x * H + h;
-    #pragma unroll
-    for (int it = 0; it < IT; it++) {
-        const int item = threadIdx.x + it * 256, J = item / dk, d = item - J * dk;
-        if (J >= NSUB) break;
-        float behind = 0.f;                                 // of the blocks behind J
+    const int mine = (int)threadIdx.x - 128;
+    float2 L[IT][SUB], k[IT][SUB];
+    if (mine >= 0) {
         #pragma unroll
-        for (int m = NSUB - 1; m >= 0; m--) if (m > J) behind += tot[m * dk + d];
+        for (int it = 0; it < IT; it++) {
+            const int item = mine + it * 128, J = item / pairs, d = 2 * (item - J * pairs);
+            if (J >= NSUB) break;
+            load16(L[it], g + ((size_t)(t0 + J * SUB) * H + h) * dk + d, (size_t)H * dk, n - J * SUB);
+            load16(k[it], p + (size_t)(t0 + J * SUB) * ldp + k_off + h * dk + d, ldp, n - J * SUB);
+            running_sums(L[it]);
+            *reinterpret_cast<float2*>(tot + J * dk + d) = L[it][SUB - 1];
+        }
+    } else {
+        stage_values(p, ldp, v_off + h * dv, t0, n, dv, vh, vl, threadIdx.x, 128);
+    }
+    __syncthreads();
+    if (mine >= 0) {
         #pragma unroll
-        for (int i = 0; i < SUB; i++) split(k[it][i] * ex2(behind + (L[it][SUB - 1] - L[it][i])), kh[(J * SUB + i) * ldk + d], kl[(J * SUB + i) * ldk + d]);
-        if (J == 0) keep[place * dk + d] = ex2(behind + L[it][SUB - 1]);
+        for (int it = 0; it < IT; it++) {
+            const int item = mine + it * 128, J = item / pairs, d = 2 * (item - J * pairs);
+            if (J >= NSUB) break;
+            float2 rest = L[it][SUB - 1];                   // of block J and the blocks behind it
+            #pragma unroll
+            for (int m = 1; m < NSUB; m++) if (m > J) rest = add2(rest, *reinterpret_cast<const float2*>(tot + m * dk + d));
+            put16(k[it], L[it], rest, -1.f, 0.f, kh + J * SUB * ldk + d, kl + J * SUB * ldk + d, ldk);
+            if (J == 0) *reinterpret_cast<float2*>(keep + place * dk + d) = make_float2(ex2(rest.x), ex2(rest.y));
+        }
     }
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, t = lane & 3;
@@ -167,7 +191,8 @@ gla_gain_kernel(const float* __restrict__ p, int ldp, int k_off, int v_off, cons
 }
 
 // ------------------------------------------------------------------ states
-// ws[place] goes from a chunk's gain to the state in front of it.  A thread has four key channels of one value's column.
+// ws[place] goes from a chunk's gain to the state in front of it, every four floats' place taken by their four leading bfloat16 terms
+// and then the four second ones.  A thread has four key channels of one value's column.
 __global__ void __launch_bounds__(128)
 gla_state_kernel(float* __restrict__ ws, const float* __restrict__ keep, float* __restrict__ state, const int* __restrict__ slots,
                  const int* __restrict__ cu, const int* __restrict__ kv_lens, int H, int dk, int dv) {
@@ -199,7 +224,10 @@ gla_state_kernel(float* __restrict__ ws, const float* __restrict__ keep, float* 
         #pragma unroll
         for (int j = 0; j < AHEAD; j++) {
             if (c0 + j < n) {
-                *reinterpret_cast<float4*>(w + (size_t)(c0 + j) * per) = S;
+                uint4 two;
+                split2(S.x, S.y, two.x, two.z);
+                split2(S.z, S.w, two.y, two.w);
+                *reinterpret_cast<uint4*>(w + (size_t)(c0 + j) * per) = two;
                 S.x = fmaf(K[j].x, S.x, D[j].x);
                 S.y = fmaf(K[j].y, S.y, D[j].y);
                 S.z = fmaf(K[j].z, S.z, D[j].z);
@@ -211,13 +239,19 @@ gla_state_kernel(float* __restrict__ ws, const float* __restrict__ keep, float* 
 }
 
 // ------------------------------------------------------------------ outputs
-// out[t, h, :] = rmsnorm(o) * norm_w * silu(gate) in bfloat16, gate in columns g_off of p.  A warp has a block of 16 tokens and
-// half of the values (NT eights of them at most).
-template <int IT, int NT>
-__global__ void __launch_bounds__(256)
+// Rows of the factors.  Of q: a token's 2^(from its block's beginning), block 3's from the middle, blocks 1 .. 3's from the chunk's
+// beginning.  Of k: 2^-(from its block's beginning), blocks 0 and 2's up to their end, blocks 0 and 1's up to the middle.
+constexpr int Q_OWN = 0, Q_MIDDLE = 64, Q_START = 80, Q_ROWS = 128;
+constexpr int K_OWN = 0, K_END = 64, K_MIDDLE = 96, K_ROWS = 128;
+
+// out[t, h, :] = rmsnorm(o) * norm_w * silu(gate) in bfloat16, gate in columns g_off of p.  The first 128 threads bring q, the
+// others k, a block's tokens of two channels each (IT times), all of them the values.  A warp has a block of 16 tokens and half
+// of the values (NT eights of them at most).  staged: the state passes through shared memory (over the factors of k).
+template <int DK, int DV, int IT, int NT>
+__global__ void __launch_bounds__(256, NT <= 8 && IT == 1 ? 2 : 1)
 gla_out_kernel(const float* __restrict__ p, int ldp, int q_off, int k_off, int v_off, int g_off, const float* __restrict__ g,
                const int* __restrict__ cu, int B, const float* __restrict__ ws, const float* __restrict__ norm_w, float eps, float scale,
-               bf16* __restrict__ out, int H, int dk, int dv) {
+               bf16* __restrict__ out, int H, int dk_, int dv_, int staged) {
     extern __shared__ __align__(16) unsigned char smem[];
     ik_pdl_wait();
     IK_AFTER_WAIT(p);
@@ -227,64 +261,60 @@ gla_out_kernel(const float* __restrict__ p, int ldp, int q_off, int k_off, int v
     ik_pdl_launch_dependents();
     int b, c;
     if (!find_chunk(cu, B, blockIdx.x, b, c)) return;
-    const int h = blockIdx.y, t0 = cu[b] + c * C, n = min(C, cu[b + 1] - t0), ldk = dk + 8, ldv = dv + 8;
+    const int dk = DK ? DK : dk_, dv = DV ? DV : dv_;
+    const int h = blockIdx.y, t0 = cu[b] + c * C, n = min(C, cu[b + 1] - t0), ldk = dk + 8, ldv = dv + 8, pairs = dk / 2;
     float* tot = (float*)smem;                              // [NSUB][dk]
-    float* before = tot + NSUB * dk;                        // [NSUB][dk] 2^(sum over the chunk's tokens in front of the block)
-    float* Ls = before + NSUB * dk;                         // [C][dk]
-    float* ss = Ls + C * dk;                                // [2][C] the halves' sums of squares
+    float* ss = tot + NSUB * dk;                            // [2][C] the halves' sums of squares
     int* direct = (int*)(ss + 2 * C);                       // [NSUB] the block forms its own entries directly
-    bf16* qh = (bf16*)(direct + NSUB);                      // [C][ldk] q 2^L
-    bf16* ql = qh + C * ldk;
-    bf16* kh = ql + C * ldk;                                // [160][ldk] for blocks 0 .. 3: rows of 16, 32, 48, 64 keys
-    bf16* kl = kh + 160 * ldk;
-    bf16* vh = kl + 160 * ldk;                              // [C][ldv]
+    bf16* qh = (bf16*)(direct + NSUB);                      // [Q_ROWS][ldk]
+    bf16* ql = qh + Q_ROWS * ldk;
+    bf16* vh = ql + Q_ROWS * ldk;                           // [C][ldv]
     bf16* vl = vh + C * ldv;
+    bf16* kh = vl + C * ldv;                                // [K_ROWS][ldk], later (staged) the state [dv][ldk]
+    bf16* kl = kh + K_ROWS * ldk;
     if (threadIdx.x < NSUB) direct[threadIdx.x] = 0;
-    float L[IT][SUB], q[IT][SUB], k[IT][SUB];
+    // what is read late sets out for the second-level cache now: the gates and the state in front of the chunk
+    for (int f = threadIdx.x & 3; f * 32 < dv; f += 4)
+        if ((int)threadIdx.x / 4 < n) prefetch_l2(p + (size_t)(t0 + threadIdx.x / 4) * ldp + g_off + h * dv + f * 32);
+    for (int f = threadIdx.x; f * 32 < dv * dk; f += 256) prefetch_l2(ws + ((size_t)blockIdx.x * H + h) * dv * dk + f * 32);
+    const bool is_q = threadIdx.x < 128;
+    const int mine = threadIdx.x & 127;
+    float2 L[IT][SUB], x[IT][SUB];
     #pragma unroll
     for (int it = 0; it < IT; it++) {
-        const int item = threadIdx.x + it * 256, J = item / dk, d = item - J * dk;
+        const int item = mine + it * 128, J = item / pairs, d = 2 * (item - J * pairs);
         if (J >= NSUB) break;
-        #pragma unroll
-        for (int i = 0; i < SUB; i++) {
-            const int r = J * SUB + i;
-            L[it][i] = r < n ? g[((size_t)(t0 + r) * H + h) * dk + d] : 0.f;
-            q[it][i] = r < n ? p[(size_t)(t0 + r) * ldp + q_off + h * dk + d] : 0.f;
-            k[it][i] = r < n ? p[(size_t)(t0 + r) * ldp + k_off + h * dk + d] : 0.f;
-        }
-        #pragma unroll
-        for (int i = 1; i < SUB; i++) L[it][i] += L[it][i - 1];
-        #pragma unroll
-        for (int i = 0; i < SUB; i++) Ls[(J * SUB + i) * dk + d] = L[it][i];
-        tot[J * dk + d] = L[it][SUB - 1];
+        load16(L[it], g + ((size_t)(t0 + J * SUB) * H + h) * dk + d, (size_t)H * dk, n - J * SUB);
+        load16(x[it], p + (size_t)(t0 + J * SUB) * ldp + (is_q ? q_off : k_off) + h * dk + d, ldp, n - J * SUB);
+        running_sums(L[it]);
+        if (is_q) *reinterpret_cast<float2*>(tot + J * dk + d) = L[it][SUB - 1];
     }
-    stage_values(p, ldp, v_off + h * dv, t0, n, dv, vh, vl);
+    stage_values(p, ldp, v_off + h * dv, t0, n, dv, vh, vl, threadIdx.x, 256);
     __syncthreads();
     #pragma unroll
     for (int it = 0; it < IT; it++) {
-        const int item = threadIdx.x + it * 256, J = item / dk, d = item - J * dk;
+        const int item = mine + it * 128, J = item / pairs, d = 2 * (item - J * pairs);
         if (J >= NSUB) break;
-        float front = 0.f;
-        #pragma unroll
-        for (int m = 0; m < NSUB; m++) if (m < J) front += tot[m * dk + d];
-        before[J * dk + d] = ex2(front);
-        if (-L[it][SUB - 1] > LIMIT) direct[J] = 1;
-        #pragma unroll
-        for (int i = 0; i < SUB; i++) {
-            split(q[it][i] * ex2(L[it][i]), qh[(J * SUB + i) * ldk + d], ql[(J * SUB + i) * ldk + d]);
-            const int r = 8 * J * (J + 1) + J * SUB + i;    // in block J's own rows, which begin at 8 J (J + 1)
-            split(k[it][i] * ex2(fminf(-L[it][i], LIMIT)), kh[r * ldk + d], kl[r * ldk + d]);
-        }
-        float rest = L[it][SUB - 1];
-        #pragma unroll
-        for (int I = 1; I < NSUB; I++) {
-            if (I <= J) continue;
-            #pragma unroll
-            for (int i = 0; i < SUB; i++) {
-                const int r = 8 * I * (I + 1) + J * SUB + i;
-                split(k[it][i] * ex2(rest - L[it][i]), kh[r * ldk + d], kl[r * ldk + d]);
+        const float2 none = make_float2(0.f, 0.f);
+        auto total = [&](int m) { return *reinterpret_cast<const float2*>(tot + m * dk + d); };
+        auto put = [&](bf16* hi, bf16* lo, int row, float2 base, float sign, float top) {
+            put16(x[it], L[it], base, sign, top, hi + row * ldk + d, lo + row * ldk + d, ldk);
+        };
+        if (is_q) {
+            put(qh, ql, Q_OWN + J * SUB, none, 1.f, 0.f);
+            if (J == 3) put(qh, ql, Q_MIDDLE, total(2), 1.f, 0.f);
+            if (J > 0) {
+                float2 front = total(0);
+                if (J > 1) front = add2(front, total(1));
+                if (J > 2) front = add2(front, total(2));
+                put(qh, ql, Q_START + (J - 1) * SUB, front, 1.f, 0.f);
             }
-            rest += tot[I * dk + d];
+        } else {
+            const float2 own = L[it][SUB - 1];
+            if (-fminf(own.x, own.y) > LIMIT) direct[J] = 1;
+            put(kh, kl, K_OWN + J * SUB, none, -1.f, LIMIT);
+            if ((J & 1) == 0) put(kh, kl, K_END + (J >> 1) * SUB, own, -1.f, 0.f);
+            if (J < 2) put(kh, kl, K_MIDDLE + J * SUB, J == 0 ? add2(own, total(1)) : own, -1.f, 0.f);
         }
     }
     __syncthreads();
@@ -295,27 +325,41 @@ gla_out_kernel(const float* __restrict__ p, int ldp, int q_off, int k_off, int v
     for (int j = 0; j < 2 * NSUB; j++)
         #pragma unroll
         for (int e = 0; e < 4; e++) s[j][e] = 0.f;
-    const bf16 *kbh = kh + 8 * I * (I + 1) * ldk, *kbl = kl + 8 * I * (I + 1) * ldk;
-    const int a_at = (I * SUB + (lane & 7) + ((lane >> 3) & 1) * 8) * ldk + (lane >> 4) * 8;
-    for (int ks = 0; ks < dk / 16; ks++) {
-        uint32_t ah[4], al[4];
-        ldsm4(ah, qh + a_at + ks * 16);
-        ldsm4(al, ql + a_at + ks * 16);
-        #pragma unroll
-        for (int np = 0; np < NSUB; np++) {
-            if (np <= I) {
-                uint32_t bh[4], bl[4];
-                const int bt = (np * 16 + (lane & 7) + (lane >> 4) * 8) * ldk + ks * 16 + ((lane >> 3) & 1) * 8;
-                ldsm4(bh, kbh + bt);
-                ldsm4(bl, kbl + bt);
-                mma(s[2 * np], ah, bh[0], bh[1]);
-                mma(s[2 * np + 1], ah, bh[2], bh[3]);
-                mma(s[2 * np], ah, bl[0], bl[1]);
-                mma(s[2 * np + 1], ah, bl[2], bl[3]);
-                mma(s[2 * np], al, bh[0], bh[1]);
-                mma(s[2 * np + 1], al, bh[2], bh[3]);
-            }
+    const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;
+    #pragma unroll
+    for (int np = 0; np < NSUB; np++) {
+        if (np > I) continue;
+        const bool across = I >= 2 && np < 2;
+        const int qr = across && I == 3 ? Q_MIDDLE : Q_OWN + I * SUB;
+        const int kr = np == I ? K_OWN + np * SUB : across ? K_MIDDLE + np * SUB : K_END + (np >> 1) * SUB;
+        const bf16 *qa = qh + (qr + a_row) * ldk + a_col, *ka = kh + (kr + (lane & 7) + (lane >> 4) * 8) * ldk + ((lane >> 3) & 1) * 8;
+        #pragma unroll 4
+        for (int ks = 0; ks < dk / 16; ks++) {
+            uint32_t ah[4], al[4], bh[4], bl[4];
+            ldsm4(ah, qa + ks * 16);
+            ldsm4(al, qa + ks * 16 + Q_ROWS * ldk);
+            ldsm4(bh, ka + ks * 16);
+            ldsm4(bl, ka + ks * 16 + K_ROWS * ldk);
+            mma(s[2 * np], ah, bh[0], bh[1]);
+            mma(s[2 * np + 1], ah, bh[2], bh[3]);
+            mma(s[2 * np], ah, bl[0], bl[1]);
+            mma(s[2 * np + 1], ah, bl[2], bl[3]);
+            mma(s[2 * np], al, bh[0], bh[1]);
+            mma(s[2 * np + 1], al, bh[2], bh[3]);
         }
+    }
+    // the state in front of the chunk: its two terms on their way while the own tokens' products run
+    const uint2* Sg = reinterpret_cast<const uint2*>(ws + ((size_t)blockIdx.x * H + h) * dv * dk);      // [dv][dk / 4][leading, second]
+    bf16 *Sh = kh, *Sl = kh + dv * ldk;
+    if (staged) {
+        __syncthreads();                                    // the factors of k have been read
+        const int per_row = dk / 2;
+        for (int idx = threadIdx.x; idx < dv * per_row; idx += 256) {
+            const int r = idx / per_row, f = idx - r * per_row;
+            const unsigned dst = (unsigned)__cvta_generic_to_shared((f & 1 ? Sl : Sh) + r * ldk + (f >> 1) * 4);
+            asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(dst), "l"(Sg + idx) : "memory");
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
     }
     const bool by_hand = direct[I] != 0;
     #pragma unroll
@@ -324,18 +368,31 @@ gla_out_kernel(const float* __restrict__ p, int ldp, int q_off, int k_off, int v
         #pragma unroll
         for (int j = 0; j < 2; j++)
             #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int i = gq + (e >> 1) * 8, jj = j * 8 + 2 * t + (e & 1);
-                if (jj > i) { s[2 * np + j][e] = 0.f; continue; }
-                if (!by_hand) continue;
-                float v = 0.f;
-                const int ri = I * SUB + i, rj = I * SUB + jj;
-                if (ri < n) {
-                    const float *qp = p + (size_t)(t0 + ri) * ldp + q_off + h * dk, *kp = p + (size_t)(t0 + rj) * ldp + k_off + h * dk;
-                    for (int d = 0; d < dk; d++) v = fmaf(qp[d] * kp[d], ex2(Ls[ri * dk + d] - Ls[rj * dk + d]), v);
+            for (int e = 0; e < 4; e++)
+                if (j * 8 + 2 * t + (e & 1) > gq + (e >> 1) * 8) s[2 * np + j][e] = 0.f;
+    }
+    if (by_hand) {                                          // rare: one entry at a time
+        float own[8];
+        #pragma unroll 1
+        for (int e = 0; e < 8; e++) {
+            const int i = I * SUB + gq + ((e >> 1) & 1) * 8, jj = I * SUB + (e >> 2) * 8 + 2 * t + (e & 1);
+            float v = 0.f;
+            if (jj <= i && i < n) {
+                const float *qp = p + (size_t)(t0 + i) * ldp + q_off + h * dk, *kp = p + (size_t)(t0 + jj) * ldp + k_off + h * dk;
+                for (int d = 0; d < dk; d++) {
+                    float sum = 0.f;
+                    for (int m = jj + 1; m <= i; m++) sum += g[((size_t)(t0 + m) * H + h) * dk + d];
+                    v = fmaf(qp[d] * kp[d], ex2(sum), v);
                 }
-                s[2 * np + j][e] = v;
             }
+            #pragma unroll
+            for (int f = 0; f < 8; f++) if (f == e) own[f] = v;
+        }
+        #pragma unroll
+        for (int np = 0; np < NSUB; np++)
+            if (np == I)
+                #pragma unroll
+                for (int f = 0; f < 8; f++) s[2 * np + (f >> 2)][f & 3] = own[f];
     }
     // own tokens
     const int nt = dv / 16, n0 = half * nt * 8;             // this warp's eights of values, the first value
@@ -368,36 +425,57 @@ gla_out_kernel(const float* __restrict__ p, int ldp, int q_off, int k_off, int v
             }
         }
     }
-    // what the state in front of the chunk carries, its rows decayed up to the block
-    const float* St = ws + (((size_t)blockIdx.x * H + h) * dv + n0 + gq) * dk + 2 * t;
+    // what the state in front of the chunk carries
+    const bf16* qs = qh + ((I == 0 ? Q_OWN : Q_START + (I - 1) * SUB) + a_row) * ldk + a_col;
+    if (staged) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+    }
+    #pragma unroll 4
     for (int ks = 0; ks < dk / 16; ks++) {
         uint32_t ah[4], al[4];
-        ldsm4(ah, qh + a_at + ks * 16);
-        ldsm4(al, ql + a_at + ks * 16);
-        const float2 f0 = *reinterpret_cast<const float2*>(before + I * dk + ks * 16 + 2 * t);
-        const float2 f1 = *reinterpret_cast<const float2*>(before + I * dk + ks * 16 + 2 * t + 8);
+        ldsm4(ah, qs + ks * 16);
+        ldsm4(al, qs + ks * 16 + Q_ROWS * ldk);
         #pragma unroll
-        for (int j = 0; j < NT; j++) {
+        for (int j = 0; j < NT; j += 2) {
             if (j < nt) {
-                const float2 s0 = *reinterpret_cast<const float2*>(St + (size_t)j * 8 * dk + ks * 16);
-                const float2 s1 = *reinterpret_cast<const float2*>(St + (size_t)j * 8 * dk + ks * 16 + 8);
-                uint32_t b0h, b0l, b1h, b1l;
-                split2(s0.x * f0.x, s0.y * f0.y, b0h, b0l);
-                split2(s1.x * f1.x, s1.y * f1.y, b1h, b1l);
-                mma(o[j], ah, b0h, b1h);
-                mma(o[j], ah, b0l, b1l);
-                mma(o[j], al, b0h, b1h);
+                uint32_t bh[4], bl[4];
+                if (staged) {
+                    const int bt = (n0 + j * 8 + (lane & 7) + (lane >> 4) * 8) * ldk + ks * 16 + ((lane >> 3) & 1) * 8;
+                    ldsm4(bh, Sh + bt);
+                    ldsm4(bl, Sl + bt);
+                } else {
+                    #pragma unroll
+                    for (int f = 0; f < 4; f++) {           // row gq of eight f >> 1, channels 2 t (+ 1) of half f & 1
+                        const uint32_t* src = reinterpret_cast<const uint32_t*>(Sg) + (size_t)(n0 + (j + (f >> 1)) * 8 + gq) * dk
+                                              + (ks * 4 + (f & 1) * 2 + (t >> 1)) * 4 + (t & 1);
+                        bh[f] = src[0];
+                        bl[f] = src[2];
+                    }
+                }
+                mma(o[j], ah, bh[0], bh[1]);
+                mma(o[j + 1], ah, bh[2], bh[3]);
+                mma(o[j], ah, bl[0], bl[1]);
+                mma(o[j + 1], ah, bl[2], bl[3]);
+                mma(o[j], al, bh[0], bh[1]);
+                mma(o[j + 1], al, bh[2], bh[3]);
             }
         }
     }
-    // norm over the head's values, gate
+    // norm over the head's values, gate: the results by whole rows, through the values' place
+    if (!staged) __syncthreads();                           // (staged: every warp was done with the values at the last barrier)
+    float* rows = (float*)vh;                               // [C][ldv]
     float r0 = 0.f, r1 = 0.f;
     #pragma unroll
     for (int j = 0; j < NT; j++) {
+        if (j >= nt) continue;
         #pragma unroll
         for (int e = 0; e < 4; e++) o[j][e] *= scale;
         r0 = fmaf(o[j][0], o[j][0], fmaf(o[j][1], o[j][1], r0));
         r1 = fmaf(o[j][2], o[j][2], fmaf(o[j][3], o[j][3], r1));
+        float* dst = rows + (I * SUB + gq) * ldv + n0 + j * 8 + 2 * t;
+        *reinterpret_cast<float2*>(dst) = make_float2(o[j][0], o[j][1]);
+        *reinterpret_cast<float2*>(dst + 8 * ldv) = make_float2(o[j][2], o[j][3]);
     }
     #pragma unroll
     for (int x = 1; x < 4; x <<= 1) {
@@ -406,27 +484,22 @@ gla_out_kernel(const float* __restrict__ p, int ldp, int q_off, int k_off, int v
     }
     if (t == 0) { ss[half * C + I * SUB + gq] = r0; ss[half * C + I * SUB + gq + 8] = r1; }
     __syncthreads();
-    #pragma unroll
-    for (int x = 0; x < 2; x++) {
-        const int r = I * SUB + gq + 8 * x;
-        if (r >= n) continue;
-        const float inv = 1.0f / sqrtf((ss[r] + ss[C + r]) / (float)dv + eps);
-        const float* gp = p + (size_t)(t0 + r) * ldp + g_off + h * dv + n0 + 2 * t;
-        bf16* op = out + ((size_t)(t0 + r) * H + h) * dv + n0 + 2 * t;
-        #pragma unroll
-        for (int j = 0; j < NT; j++) {
-            if (j < nt) {
-                const float2 gt = *reinterpret_cast<const float2*>(gp + j * 8), w = *reinterpret_cast<const float2*>(norm_w + n0 + 2 * t + j * 8);
-                *reinterpret_cast<__nv_bfloat162*>(op + j * 8) = __floats2bfloat162_rn(ik_swiglu_fast(gt.x, o[j][2 * x] * inv * w.x),
-                                                                                       ik_swiglu_fast(gt.y, o[j][2 * x + 1] * inv * w.y));
-            }
-        }
+    const int q4 = dv / 4;
+    #pragma unroll 8
+    for (int idx = threadIdx.x; idx < n * q4; idx += 256) {
+        const int r = idx / q4, c4 = (idx - r * q4) * 4;
+        const float4 gt = *reinterpret_cast<const float4*>(p + (size_t)(t0 + r) * ldp + g_off + h * dv + c4);
+        const float4 w = *reinterpret_cast<const float4*>(norm_w + c4), y = *reinterpret_cast<const float4*>(rows + r * ldv + c4);
+        const float inv = rsqrtf((ss[r] + ss[C + r]) / (float)dv + eps);
+        auto gated = [&](float a, float v, float wv) { return __fdividef(a, 1.0f + __expf(-a)) * (v * inv * wv); };
+        ik_st4(out, ((size_t)(t0 + r) * H + h) * dv + c4, make_float4(gated(gt.x, y.x, w.x), gated(gt.y, y.y, w.y), gated(gt.z, y.z, w.z), gated(gt.w, y.w, w.w)));
     }
 }
 
 size_t gain_smem(int dk, int dv) { return (size_t)NSUB * dk * 4 + (size_t)2 * C * (dk + 8 + dv + 8) * 2; }
-size_t out_smem(int dk, int dv) {
-    return (size_t)(2 * NSUB + C) * dk * 4 + 2 * C * 4 + NSUB * 4 + (size_t)(2 * (C + 160) * (dk + 8) + 2 * C * (dv + 8)) * 2;
+size_t out_smem(int dk, int dv, bool staged) {
+    const size_t rows = staged && dv > K_ROWS ? dv : K_ROWS;
+    return (size_t)NSUB * dk * 4 + 2 * C * 4 + NSUB * 4 + (size_t)(2 * (Q_ROWS + rows) * (dk + 8) + 2 * C * (dv + 8)) * 2;
 }
 
 }  // namespace
@@ -440,30 +513,39 @@ IK_EXPORT int ik_gla_chunks(const float* p, int ldp, int q_off, int k_off, int v
                             float* state, const int* slots, const int* cu, const int* kv_lens, const float* norm_w, float eps, float scale,
                             void* out, int T, int B, int H, int dk, int dv, cudaStream_t stream) {
     if (T < 0 || B < 0 || H <= 0 || dk <= 0 || dv <= 0) return IK_BAD_ARGUMENT;
-    if (dk % 16 || dk > 128 || dv % 32 || dv > 256 || ldp % 4 || q_off % 4 || k_off % 4 || v_off % 4 || g_off % 4 || ((uintptr_t)p & 15) || ((uintptr_t)ws & 15) ||
-        ((uintptr_t)keep & 15) || ((uintptr_t)state & 15) || ((uintptr_t)norm_w & 7) || (long long)H * dk * dv > 0x7fffffff || B > 65535 || H > 65535)
+    if (dk % 16 || dk > 128 || dv % 32 || dv > 256 || ldp % 4 || q_off % 4 || k_off % 4 || v_off % 4 || g_off % 4 || ((uintptr_t)p & 15) || ((uintptr_t)g & 15) ||
+        ((uintptr_t)ws & 15) || ((uintptr_t)keep & 15) || ((uintptr_t)state & 15) || ((uintptr_t)norm_w & 15) || (long long)H * dk * dv > 0x7fffffff ||
+        B > 65535 || H > 65535)
         return IK_UNSUPPORTED;
     if (T == 0 || B == 0) return IK_OK;
-    const size_t sg = gain_smem(dk, dv), so = out_smem(dk, dv);
+    const bool staged = out_smem(dk, dv, true) <= 227 * 1024;
+    const size_t sg = gain_smem(dk, dv), so = out_smem(dk, dv, staged);
     if (so > 227 * 1024) return IK_UNSUPPORTED;
     const dim3 grid(ik_gla_places(T, B), H);
-    cudaError_t e;
-#define IK_GLA(KERN, SMEM, ...)                                                                        \
-    {                                                                                                  \
-        auto kern = KERN;                                                                              \
-        if (SMEM > 48 * 1024) {                                                                        \
-            e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM);    \
-            if (e != cudaSuccess) return (int)e;                                                       \
-        }                                                                                              \
-        IK_RETURN_IF_ERROR(ik_launch(kern, grid, 256, SMEM, stream, __VA_ARGS__));                     \
+#define IK_GLA(SMEM, KERN, ...)                                                                                    \
+    {                                                                                                              \
+        auto kern = KERN;                                                                                          \
+        if (SMEM > 48 * 1024) {                                                                                    \
+            cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM);    \
+            if (e != cudaSuccess) return (int)e;                                                                   \
+        }                                                                                                          \
+        IK_RETURN_IF_ERROR(ik_launch(kern, grid, 256, SMEM, stream, __VA_ARGS__));                                 \
     }
-    if (dk <= 64) IK_GLA((gla_gain_kernel<1, 8>), sg, p, ldp, k_off, v_off, g, cu, B, ws, keep, H, dk, dv)
-    else IK_GLA((gla_gain_kernel<2, 16>), sg, p, ldp, k_off, v_off, g, cu, B, ws, keep, H, dk, dv)
+#define IK_GLA_GAIN(DK, DV, IT, NK) IK_GLA(sg, (gla_gain_kernel<DK, DV, IT, NK>), p, ldp, k_off, v_off, g, cu, B, ws, keep, H, dk, dv)
+#define IK_GLA_OUT(DK, DV, IT, NT)                                                                                                  \
+    IK_GLA(so, (gla_out_kernel<DK, DV, IT, NT>), p, ldp, q_off, k_off, v_off, g_off, g, cu, B, (const float*)ws, norm_w, eps, scale, \
+           (bf16*)out, H, dk, dv, staged ? 1 : 0)
+    if (dk == 64 && dv == 128) IK_GLA_GAIN(64, 128, 1, 8)
+    else if (dk <= 64) IK_GLA_GAIN(0, 0, 1, 8)
+    else IK_GLA_GAIN(0, 0, 2, 16)
     IK_RETURN_IF_ERROR(ik_launch(gla_state_kernel, dim3((H * dk * dv / 4 + 127) / 128, B), 128, 0, stream, ws, (const float*)keep, state, slots, cu, kv_lens, H, dk, dv));
-#define IK_GLA_OUT(IT, NT) IK_GLA((gla_out_kernel<IT, NT>), so, p, ldp, q_off, k_off, v_off, g_off, g, cu, B, (const float*)ws, norm_w, eps, scale, (bf16*)out, H, dk, dv)
-    if (dk <= 64) { if (dv <= 64) IK_GLA_OUT(1, 4) else if (dv <= 128) IK_GLA_OUT(1, 8) else IK_GLA_OUT(1, 16) }
-    else { if (dv <= 64) IK_GLA_OUT(2, 4) else if (dv <= 128) IK_GLA_OUT(2, 8) else IK_GLA_OUT(2, 16) }
+    if (dk == 64 && dv == 128) IK_GLA_OUT(64, 128, 1, 8)
+    else if (dk <= 64 && dv <= 128) IK_GLA_OUT(0, 0, 1, 8)
+    else if (dk <= 64) IK_GLA_OUT(0, 0, 1, 16)
+    else if (dv <= 128) IK_GLA_OUT(0, 0, 2, 8)
+    else IK_GLA_OUT(0, 0, 2, 16)
 #undef IK_GLA_OUT
+#undef IK_GLA_GAIN
 #undef IK_GLA
     IK_LAUNCH_STATUS();
 }

@@ -152,6 +152,11 @@ class Attention:
         if spec.get("bias") not in (None, False, True, "qkv"):
             raise ValueError(f"attention: bias {spec.get('bias')!r} is not supported (true, qkv)")
         self.biased = bool(spec.get("bias"))
+        # under a distance bias: what bounds a score in front of it.  Unit-normed queries and keys have a length of at most
+        # sqrt(head_dim); two hundredths for their rounding to 16 bits
+        self.reach = None
+        if self.slopes is not None and (self.norm_unit or self.softcap > 0):
+            self.reach = ((abs(self.scale) * self.head_dim * 1.02,) + (self.q_temp or (0.0, 0))) if self.norm_unit else (self.softcap, 0.0, 0)
         self.wide = bool(qk_norm or self.q_temp or self.head_gate or self.sink or self.v_norm or (self.biased and spec.get("bias") != "qkv")
                          or (position is not None and getattr(position, "magnitude", 1.0) != 1.0) or not standalone)
         self.norm_eps = float(spec.get("norm_eps") or 0.0)
@@ -231,7 +236,7 @@ class Attention:
                              self.pairing, writes_cache, rt.status, per_head=self.norm_per_head, bias=self.in_bias, v_norm=self.v_norm,
                              unit=self.norm_unit, q_temp=self.q_temp, key_scales=cache.key_scales)
         return attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, sink=self.sink_arg,
-                      keep=self.keep_first, slopes=self.slopes)
+                      keep=self.keep_first, slopes=self.slopes, reach=self.reach)
 
     def core(self, p: torch.Tensor, mid: torch.Tensor, ctx, cache: LayerCache, writes_cache: bool = True, mult: float = 1.0) -> None:
         """``p`` [T, n_in] float: [q | k | v | g] (a column range of a wider matrix may be given); ``mid`` [T, n_mid] in the
@@ -289,19 +294,19 @@ class Attention:
             ops.rope_append(qkv, q, cache.k_pages, cache.v_pages, ctx.token_seq, ctx.token_pos, table,
                             pos.inv_freq if pos is not None else None, self.n_heads, self.n_kv_heads, self.head_dim,
                             pos.rotary_dim if pos is not None else 0, self.pairing, writes_cache, rt.status)
-        att = attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, keep=self.keep_first, slopes=self.slopes)
+        att = attend(q, cache, ctx, table, self.n_heads, self.scale, self.window or 0, rt, self.softcap, keep=self.keep_first, slopes=self.slopes, reach=self.reach)
         self.o(att, out=residual, accumulate=accumulate)
 
 
 def attend(q: torch.Tensor, cache: LayerCache, ctx, table: torch.Tensor, n_heads: int, scale: float, window: int,
-           rt: Runtime, softcap: float = 0.0, sink=False, keep: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+           rt: Runtime, softcap: float = 0.0, sink=False, keep: int = 0, slopes: Optional[torch.Tensor] = None, reach=None) -> torch.Tensor:
     """Chooses the attention kernel: tensor-core kernels for bfloat16 when they take the
     head sizes, else the CUDA-core kernel (always for float32).  A cache entry without value pages (but with key scales) holds
     rows that are keys and values."""
     if q.dtype == torch.bfloat16 and (cache.v_pages is None or cache.v_pages.shape[3] == cache.k_pages.shape[3]):
         from ..csrc import attention_bf16
         out = attention_bf16.attend(q, cache.k_pages, cache.v_pages, ctx, table, n_heads, scale, window, rt.status,
-                                    softcap=softcap, sink=sink, keep=keep, key_scales=cache.key_scales, slopes=slopes)
+                                    softcap=softcap, sink=sink, keep=keep, key_scales=cache.key_scales, slopes=slopes, reach=reach)
         if out is not None:
             return out
     return ops.attention_simt(q, cache.k_pages, cache.v_pages, ctx.token_seq, ctx.token_pos, table, n_heads, scale,
