@@ -688,14 +688,13 @@ __global__ void __launch_bounds__(128)
 attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                    float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ kv_lens,
                    const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window, int keep,
-                   const float* __restrict__ key_scales, const float* __restrict__ slopes, Reach far, int n_pages, int chunk_pages, int n_splits, int* status) {
+                   int n_pages, int chunk_pages, int n_splits, int* status) {
     ik_pdl_wait();
     constexpr int CH = HD / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = (bf16*)smem_raw;                      // [16][LD]
     bf16* Ks = Qs + 16 * LD;                         // [NS][PAGE][LD]
-    bf16* Vs = ONE_ROW ? Ks : Ks + NS * PAGE * LD;   // [NS][PAGE][LD]
-    float* Cs = (float*)(Vs + NS * PAGE * LD);       // [NS][PAGE] the keys' scales (ONE_ROW)
+    bf16* Vs = Ks + NS * PAGE * LD;                  // [NS][PAGE][LD]
 
     const int b = blockIdx.x, split = blockIdx.z;
     const int G = nh / nkv, n_hc = (G + 15) / 16;
@@ -703,7 +702,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
     const int len = kv_lens[b], pos = len - 1;
     const int j0 = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
     // chunks of the pages the query sees, in their order (without a window: of all pages)
-    const int p_lo = (SLOPES && slopes ? first_seen(j0, pos, group_reach(far, slopes, kvh * G + hc * 16, min(16, G - hc * 16), pos)) : j0) / PAGE, n_kept = kept_pages(keep, p_lo), n_seen = n_kept + pos / PAGE - p_lo + 1;
+    const int p_lo = j0 / PAGE, n_kept = kept_pages(keep, p_lo), n_seen = n_kept + pos / PAGE - p_lo + 1;
     const int i_first = split * chunk_pages, i_last = min((split + 1) * chunk_pages, n_seen) - 1;
     if (i_first > i_last) return;                                  // there is no such chunk
 
@@ -726,16 +725,9 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
         for (int idx = threadIdx.x; idx < PAGE * CH; idx += 128) {
             const int r = idx / CH, c = idx % CH;
             cp16(ks + r * LD + c * 8, kg + r * HD + c * 8, true);
-            if (!ONE_ROW) cp16(vs + r * LD + c * 8, vg + r * HD + c * 8, true);
+            cp16(vs + r * LD + c * 8, vg + r * HD + c * 8, true);
         }
-        if (ONE_ROW && threadIdx.x < PAGE / 4)
-            cp16(Cs + stage * PAGE + threadIdx.x * 4, key_scales + ((size_t)page * nkv + kvh) * PAGE + threadIdx.x * 4, true);
     };
-    float slope[2] = {0.f, 0.f};
-    if (SLOPES && slopes) {
-        if ((threadIdx.x & 31) / 4 < n_here) slope[0] = slopes[h0 + (threadIdx.x & 31) / 4] * 1.4426950408889634f;
-        if ((threadIdx.x & 31) / 4 + 8 < n_here) slope[1] = slopes[h0 + (threadIdx.x & 31) / 4 + 8] * 1.4426950408889634f;
-    }
     #pragma unroll
     for (int s = 0; s < NS; s++) {
         if (i_first + s <= i_last) load_page(s, page_at(i_first + s, n_kept, p_lo));
@@ -782,10 +774,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
             for (int e = 0; e < 4; e++) {
                 const int r = e >> 1, j = jbase + n * 8 + (e & 1);
                 const bool ok = my_row[r] && j <= pos && (j >= j0 || j < keep);
-                float raw;
-                if (SLOPES || ONE_ROW) raw = ik_score(s[n][e], ONE_ROW ? Cs[stage * PAGE + warp * 16 + 2 * t + n * 8 + (e & 1)] : 1.f, scale_log2e, cap_log2e, slope[r], pos - j);
-                else raw = ik_capped(s[n][e], scale_log2e, cap_log2e);
-                const float v = ok ? raw : -INFINITY;
+                const float v = ok ? ik_capped(s[n][e], scale_log2e, cap_log2e) : -INFINITY;
                 s[n][e] = v;
                 mx[r] = fmaxf(mx[r], v);
             }
@@ -870,6 +859,195 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
         if (x == 0) { part_ml[slot * 2] = mm; part_ml[slot * 2 + 1] = ll; }
     }
 }
+
+#if IK_SLOPES || IK_ONE_ROW
+// The same for the modules with options, with the keys as the tile's rows and the heads as its columns (NT eights of them), which
+// wastes no row on a group of few heads: S^T = K Q^T (keys x heads), O^T += V^T P^T (dims x heads), P^T turned by a transposition in
+// registers.  Every warp brings its own 16 keys of a page, so the loop has no block barrier.
+template <int NS, int NT>
+__global__ void __launch_bounds__(128)
+attn_decode_keys_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
+                        float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ kv_lens,
+                        const int* __restrict__ table, int table_stride, int nh, int nkv, float scale_log2e, float cap_log2e, int window, int keep,
+                        const float* __restrict__ key_scales, const float* __restrict__ slopes, Reach far, int n_pages, int chunk_pages, int n_splits,
+                        int* status) {
+    ik_pdl_wait();
+    constexpr int CH = HD / 8, MINE = 16;                           // keys of a page a warp takes
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    bf16* Qs = (bf16*)smem_raw;                      // [16][LD]
+    bf16* Ks = Qs + 16 * LD;                         // [NS][PAGE][LD], a page's keys by warps
+    bf16* Vs = ONE_ROW ? Ks : Ks + NS * PAGE * LD;
+    float* Cs = (float*)(Vs + NS * PAGE * LD);       // [NS][PAGE] (ONE_ROW)
+
+    const int b = blockIdx.x, split = blockIdx.z;
+    const int G = nh / nkv, n_hc = (G + 15) / 16;
+    const int kvh = blockIdx.y / n_hc, hc = blockIdx.y % n_hc;
+    const int len = kv_lens[b], pos = len - 1;
+    const int h0 = kvh * G + hc * 16, n_here = min(16, G - hc * 16);
+    const int j0 = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+    const int p_lo = (SLOPES && slopes ? first_seen(j0, pos, group_reach(far, slopes, h0, n_here, pos)) : j0) / PAGE;
+    const int n_kept = kept_pages(keep, p_lo), n_seen = n_kept + pos / PAGE - p_lo + 1;
+    const int i_first = split * chunk_pages, i_last = min((split + 1) * chunk_pages, n_seen) - 1;
+    if (i_first > i_last) return;                                  // there is no such chunk
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    for (int idx = threadIdx.x; idx < 16 * CH; idx += 128) {
+        const int r = idx / CH, c = idx % CH;
+        const bool v = r < n_here;
+        cp16(Qs + r * LD + c * 8, v ? q + ((size_t)b * nh + h0 + r) * HD + c * 8 : q, v);
+    }
+    const int* row_of_table = table + (size_t)b * table_stride;
+    auto load = [&](int stage, int i) {
+        int page = row_of_table[page_at(i, n_kept, p_lo)];
+        if (page < 0 || page >= n_pages) { if (lane == 0) ik_set_status(status, IK_STATUS_READ_NO_PAGE); page = 0; }
+        const size_t first = ((size_t)page * nkv + kvh) * PAGE + warp * MINE;
+        const int at = (stage * PAGE + warp * MINE) * LD;
+        #pragma unroll
+        for (int idx = lane; idx < MINE * CH; idx += 32) {
+            const int r = idx / CH, c = idx % CH;
+            cp16(Ks + at + r * LD + c * 8, k_pages + (first + r) * HD + c * 8, true);
+            if (!ONE_ROW) cp16(Vs + at + r * LD + c * 8, v_pages + (first + r) * HD + c * 8, true);
+        }
+        if (ONE_ROW && lane < MINE / 4) cp16(Cs + stage * PAGE + warp * MINE + lane * 4, key_scales + first + lane * 4, true);
+    };
+    cp_commit();
+    #pragma unroll
+    for (int s = 0; s < NS; s++) {
+        if (i_first + s <= i_last) load(s, i_first + s);
+        cp_commit();
+    }
+    float slope[NT][2];
+    #pragma unroll
+    for (int n = 0; n < NT; n++)
+        #pragma unroll
+        for (int e = 0; e < 2; e++) slope[n][e] = SLOPES && slopes && n * 8 + 2 * t + e < n_here ? slopes[h0 + n * 8 + 2 * t + e] * 1.4426950408889634f : 0.f;
+    cp_wait<NS>();
+    __syncthreads();                                               // the queries are there
+    uint32_t qf[NT][HD / 16][2];
+    #pragma unroll
+    for (int n = 0; n < NT; n++)
+        #pragma unroll
+        for (int ks = 0; ks < HD / 16; ks++) {
+            const uint32_t a = (uint32_t)__cvta_generic_to_shared(Qs + (n * 8 + (lane & 7)) * LD + ks * 16 + ((lane >> 3) & 1) * 8);
+            asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n" : "=r"(qf[n][ks][0]), "=r"(qf[n][ks][1]) : "r"(a));
+        }
+    float o[NT][HD / 16][4], m_i[NT][2], l_i[NT][2];
+    #pragma unroll
+    for (int n = 0; n < NT; n++) {
+        #pragma unroll
+        for (int d = 0; d < HD / 16; d++)
+            #pragma unroll
+            for (int e = 0; e < 4; e++) o[n][d][e] = 0.f;
+        m_i[n][0] = m_i[n][1] = -INFINITY;
+        l_i[n][0] = l_i[n][1] = 0.f;
+    }
+    for (int i = i_first; i <= i_last; i++) {
+        const int stage = (i - i_first) % NS, j_base = page_at(i, n_kept, p_lo) * PAGE + warp * MINE;
+        cp_wait<NS - 1>();
+        __syncwarp();
+        const bf16* ks_ = Ks + (stage * PAGE + warp * MINE) * LD;
+        const bf16* vs_ = Vs + (stage * PAGE + warp * MINE) * LD;
+        float s[NT][4];
+        #pragma unroll
+        for (int n = 0; n < NT; n++)
+            #pragma unroll
+            for (int e = 0; e < 4; e++) s[n][e] = 0.f;
+        #pragma unroll
+        for (int ks = 0; ks < HD / 16; ks++) {
+            uint32_t a[4];
+            ldsm4(a, ks_ + ((lane & 7) + ((lane >> 3) & 1) * 8) * LD + ks * 16 + (lane >> 4) * 8);
+            #pragma unroll
+            for (int n = 0; n < NT; n++) mma(s[n], a, qf[n][ks][0], qf[n][ks][1]);
+        }
+        bool ok[2];
+        float ksc[2];
+        #pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int j = j_base + g + 8 * r;
+            ok[r] = j <= pos && (j >= j0 || j < keep);
+            ksc[r] = ONE_ROW ? Cs[stage * PAGE + warp * MINE + g + 8 * r] : 1.f;
+        }
+        uint32_t pb[NT][2];
+        #pragma unroll
+        for (int n = 0; n < NT; n++) {
+            float p[4], alpha[2];
+            #pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const float v = ik_score(s[n][e], ksc[e >> 1], scale_log2e, cap_log2e, slope[n][e & 1], pos - (j_base + g + 8 * (e >> 1)));
+                p[e] = ok[e >> 1] ? v : -INFINITY;
+            }
+            #pragma unroll
+            for (int x = 0; x < 2; x++) {
+                float mx = fmaxf(p[x], p[2 + x]);
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
+                const float m_new = fmaxf(m_i[n][x], mx), m_use = m_new == -INFINITY ? 0.f : m_new;
+                alpha[x] = ik_ex2(m_i[n][x] - m_use);
+                m_i[n][x] = m_new;
+                p[x] = ik_ex2(p[x] - m_use);
+                p[2 + x] = ik_ex2(p[2 + x] - m_use);
+                l_i[n][x] = fmaf(l_i[n][x], alpha[x], p[x] + p[2 + x]);
+            }
+            #pragma unroll
+            for (int d = 0; d < HD / 16; d++) { o[n][d][0] *= alpha[0]; o[n][d][1] *= alpha[1]; o[n][d][2] *= alpha[0]; o[n][d][3] *= alpha[1]; }
+            #pragma unroll
+            for (int r = 0; r < 2; r++) {
+                const uint32_t w = pack_bf16(p[2 * r], p[2 * r + 1]);
+                asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;\n" : "=r"(pb[n][r]) : "r"(w));
+            }
+        }
+        #pragma unroll
+        for (int d = 0; d < HD / 16; d++) {
+            uint32_t a[4];
+            ldsm4t(a, vs_ + ((lane & 7) + (lane >> 4) * 8) * LD + d * 16 + ((lane >> 3) & 1) * 8);
+            #pragma unroll
+            for (int n = 0; n < NT; n++) mma(o[n][d], a, pb[n][0], pb[n][1]);
+        }
+        __syncwarp();                                               // the warp is done with this stage
+        if (i + NS <= i_last) load(stage, i + NS);
+        cp_commit();
+    }
+    cp_wait<0>();
+    ik_pdl_launch_dependents();                                     // every key and value of this block has been read
+    __syncthreads();
+    float* sm_o = (float*)Ks;                         // [4][16][HD]
+    float* sm_ml = sm_o + 4 * 16 * HD;                // [4][16][2]
+    #pragma unroll
+    for (int n = 0; n < NT; n++)
+        #pragma unroll
+        for (int x = 0; x < 2; x++) {
+            float l = l_i[n][x];
+            #pragma unroll
+            for (int y = 4; y < 32; y <<= 1) l += __shfl_xor_sync(0xffffffffu, l, y);
+            const int row = warp * 16 + n * 8 + 2 * t + x;
+            #pragma unroll
+            for (int d = 0; d < HD / 16; d++) {
+                sm_o[row * HD + d * 16 + g] = o[n][d][x];
+                sm_o[row * HD + d * 16 + g + 8] = o[n][d][2 + x];
+            }
+            if (g == 0) { sm_ml[row * 2] = m_i[n][x]; sm_ml[row * 2 + 1] = l; }
+        }
+    __syncthreads();
+    for (int idx = threadIdx.x; idx < n_here * HD; idx += 128) {
+        const int hh = idx / HD, x = idx % HD;
+        float mm = -INFINITY;
+        #pragma unroll
+        for (int w = 0; w < 4; w++) mm = fmaxf(mm, sm_ml[(w * 16 + hh) * 2]);
+        const float m_use = mm == -INFINITY ? 0.f : mm;
+        float acc = 0.f, ll = 0.f;
+        #pragma unroll
+        for (int w = 0; w < 4; w++) {
+            const float a = exp2f(sm_ml[(w * 16 + hh) * 2] - m_use);
+            acc += sm_o[(w * 16 + hh) * HD + x] * a;
+            ll += sm_ml[(w * 16 + hh) * 2 + 1] * a;
+        }
+        const size_t slot = ((size_t)b * nh + h0 + hh) * n_splits + split;
+        part_o[slot * HD + x] = acc;
+        if (x == 0) { part_ml[slot * 2] = mm; part_ml[slot * 2 + 1] = ll; }
+    }
+}
+#endif
 
 // Merges the partials of each (sequence, head) in chunk order and writes the normalised output.
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
@@ -995,19 +1173,28 @@ IK_EXPORT int ik_attn_decode(const void* q, const void* k_pages, const void* v_p
     // the ring's space is also where the warps' partial results meet at the end
     const size_t merge_bytes = (size_t)4 * 16 * (HD + 2) * sizeof(float);
     const size_t smem = q_bytes + (ns * stage_bytes > merge_bytes ? ns * stage_bytes : merge_bytes);
+#if IK_SLOPES || IK_ONE_ROW
+#define IK_DEC_KERNEL(NS_) (G <= 8 ? attn_decode_keys_kernel<NS_, 1> : attn_decode_keys_kernel<NS_, 2>)
+#define IK_DEC_OPTIONS key_scales, slopes, far,
+#else
+#define IK_DEC_KERNEL(NS_) attn_decode_kernel<NS_>
+#define IK_DEC_OPTIONS
+#endif
 #define IK_DEC(NS_)                                                                                                  \
     {                                                                                                                \
-        auto kern = attn_decode_kernel<NS_>;                                                                         \
+        auto kern = IK_DEC_KERNEL(NS_);                                                                              \
         if (smem > 48 * 1024) {                                                                                      \
             cudaError_t e0 = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
             if (e0 != cudaSuccess) return (int)e0;                                                                   \
         }                                                                                                            \
         IK_RETURN_IF_ERROR(ik_launch(kern, grid, 128, smem, stream, (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, part_o, part_ml, \
-                                          kv_lens, table, table_stride, nh, nkv, sc_a, sc_b, window, keep, \
-                                          key_scales, slopes, far, n_pages, chunk_pages, n_splits, status));                                   \
+                                          kv_lens, table, table_stride, nh, nkv, sc_a, sc_b, window, keep, IK_DEC_OPTIONS \
+                                          n_pages, chunk_pages, n_splits, status));                                   \
     }
     if (ns == 2) IK_DEC(2) else if (ns == 3) IK_DEC(3) else IK_DEC(4)
 #undef IK_DEC
+#undef IK_DEC_KERNEL
+#undef IK_DEC_OPTIONS
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
     dim3 grid2(B, nh);

@@ -18,6 +18,9 @@ from .ops import KernelError, _check, _ptr, _stream, sm_count
 _vp, _i, _f = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
 _modules: Dict[tuple, ctypes.CDLL] = {}
 
+# Modules with options, measured on B200 (head sizes 64 and 128, contexts 2k-8k, batches 8-64): a ring of 60 KB a block leaves room for
+# enough blocks per SM; where heads stop early the blocks of a sequence are unequal, and chunks of at most 8 pages even them out.
+OPTION_RING_KB, REACH_CHUNK_PAGES = 60, 8
 DECODE_CHUNK_PAGES = 4        # default: a decode block covers 4 pages = 256 keys; chunks start at multiples of that
 
 
@@ -155,7 +158,12 @@ def attend(q, k_pages, v_pages, ctx, table, n_heads: int, scale: float, window: 
     if ctx.is_decode:
         # from the bound, not from this step's longest sequence: a captured graph is replayed for other lengths
         chunk = decode_chunk_pages(ctx.n_seqs, n_heads, nkv, seen_pages(ctx.kv_len_bound, window, keep, page_size) * page_size, page_size)
+        options = {}
+        if key_scales is not None or slopes is not None:
+            options["ring_kb"] = OPTION_RING_KB
+        if reach is not None:
+            chunk = min(chunk, REACH_CHUNK_PAGES)
         return decode(q, k_pages, v_pages, ctx.kv_lens, table, ctx.n_seqs, ctx.kv_len_bound, n_heads, scale, window,
-                      status, chunk_pages=chunk, work=work, softcap=softcap, sink=sink, keep=keep, key_scales=key_scales, slopes=slopes, reach=reach)
+                      status, chunk_pages=chunk, work=work, **options, softcap=softcap, sink=sink, keep=keep, key_scales=key_scales, slopes=slopes, reach=reach)
     return prefill(q, k_pages, v_pages, ctx.cu_seqlens, ctx.kv_lens, table, ctx.n_seqs, ctx.max_new, n_heads, scale,
                    window, status, work=work, softcap=softcap, sink=sink, keep=keep, key_scales=key_scales, slopes=slopes, reach=reach)

@@ -140,6 +140,7 @@ _SIGNATURES = {
     "ik_token_shift": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _u64, _i, _i, _i, _i, _i, _vp],
     "ik_row_decay": [_i, _vp, _i, _i, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
     "ik_lowrank_decay": [_vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _f, _i, _vp],
+    "ik_gla_decode": [_vp, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _vp, _vp, _vp, _vp, _f, _f, _vp, _i, _i, _i, _i, _vp],
     "ik_gla_places": [_i, _i],
     "ik_gla_chunks": [_vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _f, _f, _vp, _i, _i, _i, _i, _i, _vp],
     "ik_dynamic_tanh": [_vp, _vp, _vp, _vp, _f, _vp, _i, _i, _i, _vp],
@@ -1624,6 +1625,27 @@ def gla_chunks(p: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, 
     if st == -2:
         return None
     _check(st, "gla_chunks", kernels=3)
+    return out
+
+
+def gla_decode(p: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, a_off: int, a2: torch.Tensor, a2_bias: torch.Tensor, power: float,
+               state: torch.Tensor, ctx, n_heads: int, dk: int, dv: int, norm_w: torch.Tensor, eps: float, scale: float) -> Optional[torch.Tensor]:
+    """One token per sequence: ``lowrank_decay``, ``row_decay("plain", ...)`` and the head's norm and silu gate as one kernel.  Returns
+    bfloat16 [T, heads * dv], or None when the kernel does not take these sizes."""
+    _need(p, "p", torch.float32, contiguous=False)
+    for name, t in (("a2", a2), ("a2_bias", a2_bias), ("state", state), ("norm_w", norm_w)):
+        _need(t, name, torch.float32)
+    T, H, rank = p.shape[0], n_heads, a2.shape[0]
+    if p.stride(1) != 1 or T != ctx.n_seqs or a2.shape[1] != H * dk or a2_bias.numel() != H * dk or tuple(state.shape[1:]) != (2, H, dv, dk) \
+            or norm_w.numel() != dv or max(q_off + H * dk, k_off + H * dk, v_off + H * dv, g_off + H * dv, a_off + rank) > p.shape[1]:
+        raise KernelError("gla_decode: the sizes do not fit together")
+    out = torch.empty((T, H * dv), dtype=torch.bfloat16, device=p.device)
+    _work(f"gla_decode {T}x{H}x{dk}x{dv}", 8 * T * H * dk * dv + T * H * ((2 * dk + 2 * dv) * 4 + 2 * dv) + 4 * rank * H * dk, 6 * T * H * dk * dv)
+    st = lib().ik_gla_decode(_ptr(p), p.stride(0), q_off, k_off, v_off, g_off, a_off, rank, _ptr(a2), _ptr(a2_bias), power, _ptr(state), _ptr(ctx.slots),
+                             _ptr(ctx.kv_lens), _ptr(norm_w), eps, scale, _ptr(out), T, H, dk, dv, _stream())
+    if st == -2:
+        return None
+    _check(st, "gla_decode")
     return out
 
 

@@ -14,8 +14,8 @@ position the state belongs to, as the other recurrences do, so that a decode ste
 [q | k | v | g | Wa1 x] in float; the decay's second factor, the sigmoid and the root are one kernel on its last columns.  Decays, the
 state, its sums and the norm are float32 on both paths; only the products' operands are 16-bit on the bfloat16 path.
 
-A prompt on the bfloat16 path runs recurrence, norm and gate by chunks of 64 tokens on the tensor cores (``csrc/gla_chunk.cu``); single
-tokens, a few at a time, the float32 path and sizes that kernel does not take run the recurrence token by token.
+A prompt on the bfloat16 path runs recurrence, norm and gate by chunks of 64 tokens on the tensor cores (``csrc/gla_chunk.cu``), a decode
+step runs everything between the products as one kernel (``csrc/gla_decode.cu``); a few tokens at a time, the float32 path and sizes that kernel does not take run the recurrence token by token.
 """
 from __future__ import annotations
 
@@ -80,7 +80,10 @@ class GatedLinearAttention:
         p = torch.empty((T, -(-n // 4) * 4), dtype=torch.float32, device=x.device)[:, :n]
         self.in_proj(x, out=p)                                                # [T, q | k | v | g | a1]
         mid = None
-        if rt.dtype == "bfloat16" and ctx.max_new >= CHUNKED_FROM:
+        if rt.dtype == "bfloat16" and ctx.is_decode:
+            mid = ops.gla_decode(p, 0, self.k_off, self.v_off, self.g_off, self.a_off, self.a2, self.a2_bias, self.power, cache.state(STATE), ctx, H, dk,
+                                 dv, self.norm_w, self.norm_eps, self.scale)
+        elif rt.dtype == "bfloat16" and ctx.max_new >= CHUNKED_FROM:
             decay = ops.lowrank_decay(p, self.a_off, self.a2, self.a2_bias, self.power, log2=True)
             mid = ops.gla_chunks(p, 0, self.k_off, self.v_off, self.g_off, decay, cache.state(STATE), ctx, H, dk, dv, self.norm_w, self.norm_eps,
                                  self.scale)

@@ -320,6 +320,39 @@ def test_gated_linear_attention_kernels(H, K, V, strong):
             at += n
 
 
+@pytest.mark.parametrize("H,K,V,rank", [(4, 24, 40, 7), (3, 80, 16, 16), (1, 16, 32, 1), (2, 64, 128, 16), (2, 200, 8, 33), (2, 300, 24, 5), (16, 48, 64, 64), (1, 4, 300, 3),
+                                        (2, 128, 256, 16)])
+def test_the_decode_kernel_with_its_decay_norm_and_gate(H, K, V, rank):
+    """Token by token from position 0 in slots with leftovers; running a step twice changes nothing (a captured graph does)."""
+    from ithaca_b200.csrc import ops
+    n, slots, scale, eps = 12, [2, 0], K ** -0.5, 1e-5
+    g = torch.Generator().manual_seed(K)
+    a_off = 4 + 2 * H * K + 2 * H * V
+    rows = [torch.randn(n, a_off + rank + 2, generator=g) for _ in slots]
+    a2, b2, nw = torch.randn(rank, H * K, generator=g) * rank ** -0.5, torch.randn(H * K, generator=g) * 3, 1 + 0.3 * torch.randn(V, generator=g)
+    state = torch.randn(3, 2, H, V, K, device=DEV)
+    want = []
+    for b in range(2):
+        log2 = torch.log2(P.channel_decay(rows[b][:, a_off:a_off + rank].double() @ a2.double() + b2.double(), 3.0))
+        o, S, gate = _gla_plain(rows[b][:, :a_off], log2, H, K, V, scale, None)
+        want.append(((P.rms(o, eps) * nw.double()).reshape(n, H * V) * P.silu(gate), S))
+    for i in range(n):
+        p = torch.stack([r[i] for r in rows]).to(DEV)
+        for _ in range(2):
+            y = ops.gla_decode(p, 4, 4 + H * K, 4 + 2 * H * K, 4 + 2 * H * K + H * V, a_off, a2.to(DEV), b2.to(DEV), 1 / 3.0, state, _ctx([i, i], [i + 1, i + 1], slots),
+                               H, K, V, nw.to(DEV), eps, scale)
+        for b in range(2):
+            assert rel_err(y[b].float().cpu().numpy(), want[b][0][i].numpy()) < 6e-3, (i, b)
+    for b in range(2):
+        assert rel_err(state[slots[b], (n - 1) & 1].cpu().transpose(1, 2).numpy(), want[b][1].numpy()) < 1e-5
+
+
+def test_the_decode_kernel_declines_odd_key_sizes():
+    from ithaca_b200.csrc import ops
+    z = lambda *s: torch.zeros(*s, device=DEV)
+    assert ops.gla_decode(z(1, 24), 0, 6, 12, 16, 20, z(1, 6), z(6), 1.0, z(1, 2, 1, 4, 6), _ctx([0], [1], [0]), 1, 6, 4, z(4), 1e-6, 1.0) is None
+
+
 @pytest.mark.parametrize("strong", [0.05, 1.0])
 def test_long_prompts_in_chunks_against_token_by_token(strong):
     """Prompts of several chunks with a ragged end, three sequences, a portion behind each, many heads at once; the states of
