@@ -59,13 +59,15 @@ __global__ void decay_rows_kernel(const float* __restrict__ x, int ldx, const fl
 // A decay whose logit is a projection of a low-rank factor that lies in columns of a wider product:
 //   z[t, c] = sum_r w[r, c] p[t, off + r] + bias[c],   out[t, c] = sigmoid(z)^power = exp(power * log sigmoid(z)), or its log2.
 // w is stored [rank, C] (a factor's weights of neighbouring channels lie together).  A block takes TOK tokens and 256 channels; the
-// factors of its tokens go through shared memory, RC at a time, and a weight that is read serves all of its tokens.
+// factors of its tokens go through shared memory, RC at a time, and a weight that is read serves all of its tokens.  The logarithm
+// to base 2 is formed with the hardware's exponential and logarithm: log sigmoid(z) is small where they are inexact, and its
+// absolute error, a few 2^-24, is what rounding the decay itself to float would leave.
 constexpr int LR_RC = 64;
 template <int TOK>
 __global__ void __launch_bounds__(256)
 lowrank_decay_kernel(const float* __restrict__ p, int ldp, int off, int rank, const float* __restrict__ w, const float* __restrict__ bias,
                      float* __restrict__ out, int T, int C, float power, int log2_form) {
-    __shared__ float low[TOK][LR_RC];
+    __shared__ __align__(16) float low[TOK][LR_RC];
     ik_pdl_wait();
     IK_AFTER_WAIT(p);
     ik_pdl_launch_dependents();
@@ -74,19 +76,24 @@ lowrank_decay_kernel(const float* __restrict__ p, int ldp, int off, int rank, co
     #pragma unroll
     for (int i = 0; i < TOK; i++) acc[i] = 0.f;
     for (int r0 = 0; r0 < rank; r0 += LR_RC) {
-        const int n = min(LR_RC, rank - r0);
+        const int n = min(LR_RC, rank - r0), n4 = (n + 3) / 4;
         __syncthreads();
-        for (int f = threadIdx.x; f < TOK * n; f += 256) {
-            const int i = f / n, r = f - i * n;
-            low[i][r] = t0 + i < T ? p[(size_t)(t0 + i) * ldp + off + r0 + r] : 0.f;
+        for (int f = threadIdx.x; f < TOK * 4 * n4; f += 256) {
+            const int i = f / (4 * n4), r = f - i * 4 * n4;
+            low[i][r] = t0 + i < T && r < n ? p[(size_t)(t0 + i) * ldp + off + r0 + r] : 0.f;
         }
         __syncthreads();
         if (c < C) {
-            #pragma unroll 4
-            for (int r = 0; r < n; r++) {
-                const float wv = w[(size_t)(r0 + r) * C + c];
+            #pragma unroll 2
+            for (int r4 = 0; r4 < n4; r4++) {
+                float wv[4];
                 #pragma unroll
-                for (int i = 0; i < TOK; i++) acc[i] = fmaf(wv, low[i][r], acc[i]);
+                for (int j = 0; j < 4; j++) wv[j] = 4 * r4 + j < n ? w[(size_t)(r0 + 4 * r4 + j) * C + c] : 0.f;
+                #pragma unroll
+                for (int i = 0; i < TOK; i++) {
+                    const float4 l = *reinterpret_cast<const float4*>(&low[i][4 * r4]);
+                    acc[i] = fmaf(wv[3], l.w, fmaf(wv[2], l.z, fmaf(wv[1], l.y, fmaf(wv[0], l.x, acc[i]))));
+                }
             }
         }
     }
@@ -95,9 +102,9 @@ lowrank_decay_kernel(const float* __restrict__ p, int ldp, int off, int rank, co
     #pragma unroll
     for (int i = 0; i < TOK; i++) {
         if (t0 + i >= T) break;
-        const float z = acc[i] + b, tail = log1pf(expf(-fabsf(z)));
-        const float l = power * ((z < 0.f ? z : 0.f) - tail);
-        out[(size_t)(t0 + i) * C + c] = log2_form ? l * 1.4426950408889634f : expf(l);
+        const float z = acc[i] + b, down = z < 0.f ? z : 0.f;
+        out[(size_t)(t0 + i) * C + c] = log2_form ? power * (down * 1.4426950408889634f - __log2f(1.0f + __expf(-fabsf(z))))
+                                                  : expf(power * (down - log1pf(expf(-fabsf(z)))));
     }
 }
 

@@ -72,9 +72,10 @@ class Attention:
         d, nh, nkv, hd = spec["hidden_size"], spec["n_heads"], spec["n_kv_heads"], spec["head_dim"]
         w = spec.weights
         hdv = spec.get("v_head_dim") or hd
-        out = {w["q"]: TensorReq((nh * hd, d)), w["k"]: TensorReq((nkv * hd, d)), w["o"]: TensorReq((d, nh * hdv))}
+        out = {w["q"]: TensorReq((nh * hd, d)), w["k"]: TensorReq((nkv * hd, d))}
         if spec.get("values") != "keys":
             out[w["v"]] = TensorReq((nkv * hdv, d))
+        out[w["o"]] = TensorReq((d, nh * hdv))
         if spec.get("qk_norm") in ("head", "projection"):
             per_head = spec.get("qk_norm") == "head"
             out[w["q_norm"]] = TensorReq((hd if per_head else nh * hd,), init="ones")
